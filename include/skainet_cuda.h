@@ -61,6 +61,9 @@ extern "C" {
 #define SKN_TYPE_IQ4_NL 20 /* 32 weights, 18 bytes: d, 16 nibble bytes indexing the 16-entry IQ4 codebook */
 #define SKN_TYPE_IQ4_XS 23 /* 256 weights, 136 bytes: d, 16 scale high bits, 4 scale nibble bytes, 128 codebook nibbles */
 
+/* Dense weights (skn_tensor_upload_dense): bf16, two bytes per weight */
+#define SKN_TYPE_BF16 30
+
 typedef struct skn_ctx skn_ctx;
 typedef struct skn_tensor skn_tensor;
 typedef struct skn_kvcache skn_kvcache;
@@ -154,6 +157,13 @@ int32_t skn_tensor_upload_quant_shard(skn_ctx *ctx, int32_t ggml_type, int64_t n
                                       int64_t row_begin, int64_t row_count, int64_t col_begin,
                                       int64_t col_count, skn_tensor **out);
 
+/* Upload a dense [n_rows, n_cols] weight of bf16 values (type SKN_TYPE_BF16), n_bytes = n_rows * n_cols * 2.  The
+ * device rows are zero-padded to 16 bytes.  The result is multiplied by skn_matmul[_dev] (bf16 operands and fp32
+ * accumulation from SKN_OPT_PREFILL_MIN_M rows on, fp32 products of fp32 activations below) and taken by the decoders
+ * over dense weights; the block-quantized entry points answer SKN_ERR_TYPE for it. */
+int32_t skn_tensor_upload_dense(skn_ctx *ctx, int32_t type, int64_t n_rows, int64_t n_cols, const void *host, int64_t n_bytes,
+                                skn_tensor **out);
+
 int32_t skn_tensor_destroy(skn_tensor *t);
 
 /* shape / type / device layout of a tensor (any out pointer may be NULL):
@@ -237,8 +247,18 @@ int32_t skn_kv_create(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int32_t h
 #define SKN_KV_F32 0
 #define SKN_KV_F16 1
 #define SKN_KV_Q8_0 2
+#define SKN_KV_BF16 3 /* position-addressed caches only (skn_kv_create_by_position) */
 int32_t skn_kv_create_typed(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int32_t head_dim, int32_t capacity,
                             int32_t kv_dtype, skn_kvcache **out);
+/* A position-addressed cache: the token at position p of sequence b occupies slot p % capacity of
+ * K [batch][n_kv_heads][capacity][k_dim rounded up to 16] and V (v_dim likewise), fp32 or bf16 (SKN_KV_F32 /
+ * SKN_KV_BF16), k_dim and v_dim up to SKN_ATTN_MAX_DIM.  It does not count tokens: its owner passes the positions, so
+ * a freed sequence needs no clearing, and attention that never looks further back than a chunk needs no more slots
+ * than a chunk and one step's tokens.  Served by skn_chunk_attn and the decoders over dense weights; the ring
+ * operations below (append, load, gather, skn_attn_*) refuse it with SKN_ERR_BAD_HANDLE. */
+#define SKN_ATTN_MAX_DIM 512
+int32_t skn_kv_create_by_position(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int32_t k_dim, int32_t v_dim, int32_t capacity,
+                                  int32_t kv_dtype, skn_kvcache **out);
 /* element type of the cache (what k_dev / v_dev of skn_kv_info point at) */
 int32_t skn_kv_dtype(const skn_kvcache *kv, int32_t *kv_dtype);
 int32_t skn_kv_destroy(skn_kvcache *kv);
@@ -391,6 +411,105 @@ int32_t skn_llama_forward(skn_llama *m, const int32_t *tokens_host, int32_t T, i
 int32_t skn_llama_forward_dev(skn_llama *m, const int32_t *tokens_dev, int32_t T);
 /* tokens cached per sequence so far as counted by the host-side calls (-1 on a bad handle) */
 int32_t skn_llama_position(const skn_llama *m);
+
+/* ---- Token mixers of decoders over dense weights ------------------------------------------------
+ * No counterpart in the reference (no attention, no recurrence).  Host-pointer forms of the mechanisms
+ * that skn_lugasun_* runs on the device; each advances `n_seqs` sequences (slots seq0 ..) by T tokens,
+ * pos_host[s] tokens having come before.  Raw heads are [n_seqs][T][heads][dim] fp32. */
+typedef struct skn_state skn_state;
+
+/* Softmax attention with per-head RMS norm of q and k, rotation of the first rot_dims dimensions of q
+ * and k (dimension i pairs with i + rot_dims / 2, angle pos * rot_base^(-2 i / rot_dims)), scores
+ * scale * (q . k) optionally capped to softcap * tanh(score / softcap), and visibility of the earlier
+ * keys of the query's own chunk of `chunk` positions (counted from position 0). */
+typedef struct skn_attn_spec {
+    int32_t heads, kv_heads, dim, vdim;
+    int32_t rot_dims;    /* 0: no rotation */
+    int32_t chunk;       /* 0: every earlier key is visible */
+    double rot_base;
+    float scale, softcap; /* softcap 0: none */
+    float eps;           /* of the q / k norms */
+    int32_t reserved;
+} skn_attn_spec;
+/* Linear attention with one decay per head: S <- decay S + k v^T, o = S^T q, with q and k rotated as
+ * above and k divided by sqrt(dim); each head's o is divided by its root mean square and multiplied by
+ * silu(g).  `decay` is a host array of `heads` values. */
+typedef struct skn_retention_spec {
+    int32_t heads, dim, vdim;
+    int32_t rot_dims;
+    double rot_base;
+    const double *decay;
+    float eps;
+    int32_t reserved;
+} skn_retention_spec;
+
+/* recurrent state of `slots` sequences, fp32 [heads][k_dim][v_dim] each; a sequence at position 0 starts from zero */
+int32_t skn_state_create(skn_ctx *ctx, int32_t slots, int32_t heads, int32_t k_dim, int32_t v_dim, skn_state **out);
+int32_t skn_state_destroy(skn_state *s);
+int32_t skn_state_read(skn_state *s, int32_t slot, float *out_host);
+/* out [n_seqs][T][heads][vdim]; the new keys and values enter the cache.  q_gain, k_gain [dim]: gains of the norms, or
+ * both NULL for no norm. */
+int32_t skn_chunk_attn(skn_kvcache *kv, const skn_attn_spec *spec, int32_t seq0, int32_t n_seqs, int32_t T, const int32_t *pos_host,
+                       int32_t max_ctx, const float *q_gain_host, const float *k_gain_host, const float *q_host, const float *k_host,
+                       const float *v_host, float *out_host);
+int32_t skn_retention(skn_state *s, const skn_retention_spec *spec, int32_t seq0, int32_t n_seqs, int32_t T, const int32_t *pos_host,
+                      int32_t max_ctx, const float *q_host, const float *k_host, const float *v_host, const float *g_host, float *out_host);
+
+/* ---- Lugasun decoder ----------------------------------------------------------------------------
+ * Embedding -> layers -> RMS norm -> logits over the embedding table.  A layer adds to the residual stream (fp32):
+ * a mixer (chunked attention and retention side by side on the same normalised input, each with its own weight
+ * in the sum), an optional squared-relu feed-forward, and an optional token side input (a gate times a row of a
+ * second embedding table, projected and normalised).  Layers loop_start .. loop_stop - 1 run loop_times
+ * times in a row with a cache and a state per pass, each pass starting from loop_in [x; embedding].
+ * Weights are dense bf16; matrix products run on bf16 operands with fp32 accumulation (SKN_LUGASUN_BF16)
+ * or in fp32 throughout (SKN_LUGASUN_F32).  The decoder keeps max_seqs sequences of any lengths; a step
+ * advances a contiguous range of them by the same number of tokens. */
+typedef struct skn_lugasun skn_lugasun;
+#define SKN_LUGASUN_F32 0
+#define SKN_LUGASUN_BF16 1
+typedef struct skn_lugasun_layer {
+    skn_attn_spec left;
+    skn_retention_spec right;
+    float left_scale, right_scale;
+    int32_t ff;          /* 0: no feed-forward */
+    int32_t reserved;
+} skn_lugasun_layer;
+typedef struct skn_lugasun_spec {
+    int32_t n_layers, width, vocab;
+    int32_t side_dim;    /* 0: no token side input */
+    int32_t loop_start, loop_stop, loop_times; /* loop_times 0: no loop */
+    float eps;
+    const skn_lugasun_layer *layers;
+} skn_lugasun_spec;
+/* Weights of one layer, borrowed (they must outlive the decoder); gains are host vectors, copied.
+ * w_in: [left q | left k | left v | right q | right k | right v | right g] stacked by rows, [.., width];
+ * w_out: [left o | right o] side by side, [width, left heads * vdim + right heads * vdim]. */
+typedef struct skn_lugasun_weights {
+    const skn_tensor *w_in, *w_out, *up, *down, *side_gate, *side_proj;
+    const float *norm1, *norm2, *q_gain, *k_gain, *side_norm;
+} skn_lugasun_weights;
+int32_t skn_lugasun_create(skn_ctx *ctx, const skn_lugasun_spec *spec, int32_t max_seqs, int32_t max_tokens, int32_t max_ctx,
+                           int32_t dtype, skn_lugasun **out);
+int32_t skn_lugasun_destroy(skn_lugasun *m);
+int32_t skn_lugasun_set_layer(skn_lugasun *m, int32_t layer, const skn_lugasun_weights *w);
+/* loop_in and side_embed may be NULL when the model has no loop / no side input */
+int32_t skn_lugasun_set_head(skn_lugasun *m, const skn_tensor *embed, const float *final_norm_host, const skn_tensor *loop_in,
+                             const skn_tensor *side_embed);
+/* forget the tokens of sequence seq (-1: of all) */
+int32_t skn_lugasun_reset(skn_lugasun *m, int32_t seq);
+int32_t skn_lugasun_position(const skn_lugasun *m, int32_t seq);
+/* One step: T new tokens for each of the sequences seq0 .. seq0 + n_seqs - 1 (n_seqs * T <= max_tokens);
+ * tokens [n_seqs][T], NULL with T == 1 feeds back the greedy ids of those sequences.  want_rows: the
+ * n_want rows (s * T + t, any order) whose logits [n_want][vocab] are returned; next_host [n_seqs]: the
+ * greedy token after each sequence's last position.  With neither the output layer is skipped. */
+int32_t skn_lugasun_forward(skn_lugasun *m, int32_t seq0, int32_t n_seqs, const int32_t *tokens_host, int32_t T, int32_t n_want,
+                            const int32_t *want_rows_host, float *logits_host, int32_t *next_host);
+/* Enqueue only; head != 0 computes logits and greedy ids of every sequence's last position.  A single-token step
+ * with tokens_dev == NULL may be captured into a CUDA graph; replays advance the device positions but not
+ * skn_lugasun_position, and a step past max_ctx is reported by skn_sync as SKN_ERR_SHAPE. */
+int32_t skn_lugasun_forward_dev(skn_lugasun *m, int32_t seq0, int32_t n_seqs, const int32_t *tokens_dev, int32_t T, int32_t head);
+/* residual stream after every layer run of the last step: [layer runs][rows][width], recorded while `on` */
+int32_t skn_lugasun_trace(skn_lugasun *m, int32_t on, int32_t rows, float *out_host);
 
 /* ---- GGUF container --------------------------------------------------------------------------
  * Memory-mapped GGUF v2 / v3 reader with 64-bit offsets; tensor data is handed out as pointers

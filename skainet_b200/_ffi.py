@@ -16,6 +16,34 @@ LIB_PATH = os.environ.get("SKAINET_CUDA_LIB") or os.path.join(_HERE, "libskainet
 c_i32, c_i64, c_vp = ctypes.c_int32, ctypes.c_int64, ctypes.c_void_p
 P = ctypes.POINTER
 
+
+
+class AttnSpec(ctypes.Structure):
+    _fields_ = [("heads", c_i32), ("kv_heads", c_i32), ("dim", c_i32), ("vdim", c_i32), ("rot_dims", c_i32), ("chunk", c_i32),
+                ("rot_base", ctypes.c_double), ("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("eps", ctypes.c_float),
+                ("reserved", c_i32)]
+
+
+class RetentionSpec(ctypes.Structure):
+    _fields_ = [("heads", c_i32), ("dim", c_i32), ("vdim", c_i32), ("rot_dims", c_i32), ("rot_base", ctypes.c_double),
+                ("decay", P(ctypes.c_double)), ("eps", ctypes.c_float), ("reserved", c_i32)]
+
+
+class LugasunLayer(ctypes.Structure):
+    _fields_ = [("left", AttnSpec), ("right", RetentionSpec), ("left_scale", ctypes.c_float), ("right_scale", ctypes.c_float),
+                ("ff", c_i32), ("reserved", c_i32)]
+
+
+class LugasunSpec(ctypes.Structure):
+    _fields_ = [("n_layers", c_i32), ("width", c_i32), ("vocab", c_i32), ("side_dim", c_i32), ("loop_start", c_i32),
+                ("loop_stop", c_i32), ("loop_times", c_i32), ("eps", ctypes.c_float), ("layers", P(LugasunLayer))]
+
+
+class LugasunWeights(ctypes.Structure):
+    _fields_ = [(n, c_vp) for n in ("w_in", "w_out", "up", "down", "side_gate", "side_proj", "norm1", "norm2", "q_gain", "k_gain",
+                                    "side_norm")]
+
+
 # name -> (restype, argtypes)
 SIGNATURES = {
     "skn_version": (c_i32, []),
@@ -77,6 +105,22 @@ SIGNATURES = {
     "skn_llama_forward": (c_i32, [c_vp, c_vp, c_i32, c_vp, c_vp]),
     "skn_llama_forward_dev": (c_i32, [c_vp, c_vp, c_i32]),
     "skn_llama_position": (c_i32, [c_vp]),
+    "skn_tensor_upload_dense": (c_i32, [c_vp, c_i32, c_i64, c_i64, c_vp, c_i64, P(c_vp)]),
+    "skn_kv_create_by_position": (c_i32, [c_vp, c_i32, c_i32, c_i32, c_i32, c_i32, c_i32, P(c_vp)]),
+    "skn_state_create": (c_i32, [c_vp, c_i32, c_i32, c_i32, c_i32, P(c_vp)]),
+    "skn_state_destroy": (c_i32, [c_vp]),
+    "skn_state_read": (c_i32, [c_vp, c_i32, c_vp]),
+    "skn_chunk_attn": (c_i32, [c_vp, P(AttnSpec), c_i32, c_i32, c_i32, c_vp, c_i32, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp]),
+    "skn_retention": (c_i32, [c_vp, P(RetentionSpec), c_i32, c_i32, c_i32, c_vp, c_i32, c_vp, c_vp, c_vp, c_vp, c_vp]),
+    "skn_lugasun_create": (c_i32, [c_vp, P(LugasunSpec), c_i32, c_i32, c_i32, c_i32, P(c_vp)]),
+    "skn_lugasun_destroy": (c_i32, [c_vp]),
+    "skn_lugasun_set_layer": (c_i32, [c_vp, c_i32, P(LugasunWeights)]),
+    "skn_lugasun_set_head": (c_i32, [c_vp, c_vp, c_vp, c_vp, c_vp]),
+    "skn_lugasun_reset": (c_i32, [c_vp, c_i32]),
+    "skn_lugasun_position": (c_i32, [c_vp, c_i32]),
+    "skn_lugasun_forward": (c_i32, [c_vp, c_i32, c_i32, c_vp, c_i32, c_i32, c_vp, c_vp, c_vp]),
+    "skn_lugasun_forward_dev": (c_i32, [c_vp, c_i32, c_i32, c_vp, c_i32, c_i32]),
+    "skn_lugasun_trace": (c_i32, [c_vp, c_i32, c_i32, c_vp]),
     "skn_gguf_open": (c_i32, [ctypes.c_char_p, P(c_vp)]),
     "skn_gguf_close": (c_i32, [c_vp]),
     "skn_gguf_counts": (c_i32, [c_vp, P(c_i32), P(c_i64), P(c_i64), P(c_i64), P(c_i64)]),
@@ -88,22 +132,35 @@ SIGNATURES = {
 }
 
 _lib = None
+_path = None
 
 
 class LibraryMissing(RuntimeError):
     pass
 
 
+def use(path: str):
+    """Load this build instead of the default one: a library that holds the entry points of one model family
+    (build.build_family).  Entry points it does not have raise AttributeError when called."""
+    global _path
+    if _lib is not None and _path != path:
+        raise RuntimeError("a library is loaded already")
+    _path = path
+
+
 def lib() -> ctypes.CDLL:
     """Load the shared library (once).  Raises LibraryMissing if it has not been built."""
-    global _lib
+    global _lib, _path
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
+        path = _path or LIB_PATH
+        if not os.path.exists(path):
             raise LibraryMissing(
-                f"{LIB_PATH} is missing: build it with `python -m skainet_b200.build` "
+                f"{path} is missing: build it with `python -m skainet_b200.build` "
                 "(there is no fallback implementation)")
-        L = ctypes.CDLL(LIB_PATH)
+        L = ctypes.CDLL(path)
         for name, (res, args) in SIGNATURES.items():
+            if _path is not None and not hasattr(L, name):
+                continue                 # a one-family build
             fn = getattr(L, name)  # AttributeError if the symbol is not exported
             fn.restype = res
             fn.argtypes = args

@@ -1,6 +1,9 @@
 """Builds libskainet_cuda.so in-tree with nvcc for sm_100a (cross-compiles without a GPU).
 
     python -m skainet_b200.build [--force] [--verbose]
+
+`build` makes the whole library; `build_family` compiles only what one model family runs (FAMILIES), for a
+program that serves a single model from a fresh checkout.
 """
 from __future__ import annotations
 
@@ -27,24 +30,41 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found")
 
 
-def sources() -> list[str]:
-    return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
+# translation units of a model family (the entry points of the others are absent from its library)
+FAMILIES = {"lugasun": ["skn_core.cu", "skn_kv_cache.cu", "skn_dense.cu", "skn_rows.cu", "skn_mixers.cu", "skn_glue.cu", "skn_lugasun.cu"]}
 
 
-def _deps_mtime() -> float:
-    files = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(ROOT, "include", "skainet_cuda.h")]
-    return max(os.path.getmtime(f) for f in files)
+def sources(family: str | None = None) -> list[str]:
+    return sorted(os.path.join(CSRC, f) for f in (FAMILIES[family] if family else os.listdir(CSRC)) if f.endswith(".cu"))
+
+
+def _deps_mtime(family: str | None = None) -> float:
+    files = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if not f.endswith(".cu")] + sources(family)
+    return max(os.path.getmtime(f) for f in files + [os.path.join(ROOT, "include", "skainet_cuda.h")])
+
+
+def _fresh(lib: str, family: str | None = None) -> bool:
+    return os.path.exists(lib) and os.path.getmtime(lib) >= _deps_mtime(family)
+
+
+def build_family(family: str) -> str:
+    """Path of a library with this family's entry points: the whole library when it is built, else a smaller one."""
+    return LIB if _fresh(LIB) else _build(os.path.join(HERE, f"libskainet_{family}.so"), family)
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and os.path.exists(LIB) and os.path.getmtime(LIB) >= _deps_mtime():
+    return _build(LIB, None, force, verbose)
+
+
+def _build(LIB: str, family: str | None, force: bool = False, verbose: bool = False) -> str:
+    if not force and _fresh(LIB, family):
         return LIB
     nvcc = _nvcc()
     os.makedirs(OBJ_DIR, exist_ok=True)
     hdr_mtime = max(os.path.getmtime(os.path.join(CSRC, f)) for f in os.listdir(CSRC) if not f.endswith(".cu"))
     hdr_mtime = max(hdr_mtime, os.path.getmtime(os.path.join(ROOT, "include", "skainet_cuda.h")))
     objs, procs = [], []
-    for src in sources():
+    for src in sources(family):
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
         objs.append(obj)
         if not force and os.path.exists(obj) and os.path.getmtime(obj) >= max(os.path.getmtime(src), hdr_mtime):

@@ -11,6 +11,7 @@
 #define SKN_MAGIC_CTX 0x736b6e63u     // 'sknc'
 #define SKN_MAGIC_TENSOR 0x736b6e74u  // 'sknt'
 #define SKN_MAGIC_KV 0x736b6e6bu      // 'sknk'
+#define SKN_MAGIC_STATE 0x736b6e73u   // 'skns'
 
 // cached launch geometry of the streaming matvec (state: 0 = not planned yet,
 // 1 = valid, -1 = shape not covered by the streaming kernel)
@@ -126,11 +127,35 @@ struct skn_order_guard {
     skn_order_guard &operator=(const skn_order_guard &) = delete;
 };
 
-// error plumbing (skn_api.cu)
+struct skn_kvcache {
+    uint32_t magic;
+    skn_ctx *ctx;
+    int32_t batch, n_kv_heads, head_dim, capacity;
+    int32_t dtype;               // SKN_KV_*: element type of d_k / d_v
+    // position-addressed caches (skn_kv_create_by_position): position p of a sequence lives in slot p % capacity, rows
+    // are k_pitch / v_pitch elements apart, and the owner keeps the lengths (d_len counts nothing)
+    bool by_position;
+    int32_t v_dim, k_pitch, v_pitch;
+    void *d_k, *d_v;
+    int32_t *d_len, *d_start;
+    unsigned *d_tickets;         // [batch][n_kv_heads], zero between launches: split-attention merge tickets
+};
+
+// Recurrent state of linear-attention heads, [slots][heads][k_dim][v_pitch] fp32.  A sequence at position 0 starts
+// from zero whatever its slot held before.
+struct skn_state {
+    uint32_t magic;
+    skn_ctx *ctx;
+    int32_t slots, heads, k_dim, v_dim, v_pitch;
+    float *d;
+};
+
+// error plumbing (skn_core.cu)
 int32_t skn_fail(skn_ctx *ctx, int32_t code, const char *fmt, ...);
 int32_t skn_check_cuda(skn_ctx *ctx, cudaError_t e, const char *what);
 bool skn_ctx_ok(const skn_ctx *ctx);
 bool skn_tensor_ok(const skn_tensor *t);
+bool skn_kv_ok(const skn_kvcache *kv);
 int32_t skn_stage_reserve(skn_ctx *ctx, void **buf, size_t *cap, size_t need);
 int32_t skn_status_check(skn_ctx *ctx);
 

@@ -30,21 +30,12 @@
 #include <stdlib.h>
 #include <new>
 
-struct skn_kvcache {
-    uint32_t magic;
-    skn_ctx *ctx;
-    int32_t batch, n_kv_heads, head_dim, capacity;
-    int32_t dtype;               // SKN_KV_F32, SKN_KV_F16 or SKN_KV_Q8_0: element type of d_k / d_v
-    void *d_k, *d_v;
-    int32_t *d_len, *d_start;
-    unsigned *d_tickets;         // [batch][n_kv_heads], zero between launches: split-attention merge tickets
-};
-
 constexpr int ATT_CHUNK = 256;   // cached tokens per CTA (64 when the grid would otherwise leave SMs idle)
 constexpr int ATT_WARPS = 4;
 constexpr int ATT_MERGE_MAX_SPLITS = 64;   // most splits the in-kernel merge handles (its weights reuse the score buffer)
 
-static bool kv_ok(const skn_kvcache *kv) { return kv && kv->magic == SKN_MAGIC_KV && skn_ctx_ok(kv->ctx); }
+// the ring operations of this file: equal key and value widths, counted by the cache itself (not the position-addressed caches)
+static bool kv_ok(const skn_kvcache *kv) { return skn_kv_ok(kv) && !kv->by_position; }
 
 // Cache element types: fp32, or fp16 (half the attention traffic; values are rounded to nearest
 // even on their way in and widened to fp32 on their way out, all arithmetic stays fp32).
@@ -1056,77 +1047,6 @@ static cudaError_t dispatch_attn(const skn_kvcache *kv, int G, const float *q, f
 // ----------------------------------------------------------------------------------------
 extern "C" {
 
-int32_t skn_kv_create(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int32_t head_dim, int32_t capacity,
-                      skn_kvcache **out) {
-    return skn_kv_create_typed(ctx, batch, n_kv_heads, head_dim, capacity, SKN_KV_F32, out);
-}
-
-int32_t skn_kv_create_typed(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int32_t head_dim, int32_t capacity,
-                            int32_t kv_dtype, skn_kvcache **out) {
-    if (!skn_ctx_ok(ctx)) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "bad context handle");
-    SKN_ENTER(ctx);
-    if (!out) return skn_fail(ctx, SKN_ERR_ARG, "out is NULL");
-    *out = nullptr;
-    if (kv_dtype != SKN_KV_F32 && kv_dtype != SKN_KV_F16 && kv_dtype != SKN_KV_Q8_0)
-        return skn_fail(ctx, SKN_ERR_TYPE, "cache element type %d is none of fp32, fp16, Q8_0", kv_dtype);
-    if (batch < 1 || n_kv_heads < 1 || capacity < 1) return skn_fail(ctx, SKN_ERR_ARG, "batch, heads and capacity must be positive");
-    if (head_dim != 64 && head_dim != 128) return skn_fail(ctx, SKN_ERR_SHAPE, "head_dim must be 64 or 128 (got %d)", head_dim);
-    skn_kvcache *kv = new (std::nothrow) skn_kvcache();
-    if (!kv) return skn_fail(ctx, SKN_ERR_OOM, "host allocation failed");
-    memset(kv, 0, sizeof(*kv));
-    kv->magic = SKN_MAGIC_KV;
-    kv->ctx = ctx;
-    kv->batch = batch; kv->n_kv_heads = n_kv_heads; kv->head_dim = head_dim; kv->capacity = capacity;
-    kv->dtype = kv_dtype;
-    // Q8_0: an int8 plane, then the fp16 scales of its 32-dim blocks
-    const size_t elems = (size_t)batch * n_kv_heads * capacity * head_dim;
-    const size_t n = kv_dtype == SKN_KV_Q8_0 ? elems + elems / 32 * 2 : elems * (kv_dtype == SKN_KV_F16 ? 2 : sizeof(float));
-    cudaError_t e = cudaSetDevice(ctx->device);
-    if (e == cudaSuccess) e = cudaMalloc((void **)&kv->d_k, n);
-    if (e == cudaSuccess) e = cudaMalloc((void **)&kv->d_v, n);
-    const size_t n_ints = (size_t)2 * batch + (size_t)batch * n_kv_heads;     // lengths, starts, merge tickets
-    if (e == cudaSuccess) e = cudaMalloc((void **)&kv->d_len, n_ints * sizeof(int32_t));
-    if (e == cudaSuccess) {
-        kv->d_start = kv->d_len + batch;
-        kv->d_tickets = reinterpret_cast<unsigned *>(kv->d_len + 2 * batch);
-        e = cudaMemsetAsync(kv->d_len, 0, n_ints * sizeof(int32_t), ctx->stream);
-    }
-    if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
-    if (e != cudaSuccess) {
-        if (kv->d_k) cudaFree(kv->d_k);
-        if (kv->d_v) cudaFree(kv->d_v);
-        if (kv->d_len) cudaFree(kv->d_len);
-        kv->magic = 0;
-        delete kv;
-        return skn_check_cuda(ctx, e, "kv cache allocation");
-    }
-    *out = kv;
-    return SKN_OK;
-}
-
-int32_t skn_kv_destroy(skn_kvcache *kv) {
-    if (!kv || kv->magic != SKN_MAGIC_KV) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "bad kv cache handle");
-    if (skn_ctx_ok(kv->ctx)) {
-        cudaSetDevice(kv->ctx->device);
-        cudaStreamSynchronize(kv->ctx->stream);
-    }
-    cudaFree(kv->d_k);
-    cudaFree(kv->d_v);
-    cudaFree(kv->d_len);
-    kv->magic = 0;
-    delete kv;
-    return SKN_OK;
-}
-
-int32_t skn_kv_reset(skn_kvcache *kv) {
-    if (!kv_ok(kv)) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "bad kv cache handle");
-    skn_ctx *ctx = kv->ctx;
-    SKN_ENTER(ctx);
-    SKN_CUDA(ctx, cudaSetDevice(ctx->device));
-    SKN_CUDA(ctx, cudaMemsetAsync(kv->d_len, 0, 2 * sizeof(int32_t) * kv->batch, ctx->stream));
-    return SKN_OK;
-}
-
 int32_t skn_kv_load(skn_kvcache *kv, const float *k_host, const float *v_host, int32_t tokens,
                     const int32_t *lens_host) {
     if (!kv_ok(kv)) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "bad kv cache handle");
@@ -1475,29 +1395,6 @@ int32_t skn_attn_decode_noalloc_dev(skn_kvcache *kv, const float *q_dev, int32_t
     }
     SKN_CUDA(ctx, dispatch_attn(kv, G, q_dev, scale, part, attn_pick_chunk(kv, n_q_heads, 1, SKN_ATTN_STATIC_SCRATCH_BYTES),
                                 out_dev, ctx->stream));
-    return SKN_OK;
-}
-
-// element type of the cache buffers (SKN_KV_F32 / SKN_KV_F16 / SKN_KV_Q8_0): what the pointers of skn_kv_info point at
-int32_t skn_kv_dtype(const skn_kvcache *kv, int32_t *kv_dtype) {
-    if (!kv_ok(kv)) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "bad kv cache handle");
-    if (!kv_dtype) return skn_fail(kv->ctx, SKN_ERR_ARG, "kv_dtype is NULL");
-    *kv_dtype = kv->dtype;
-    return SKN_OK;
-}
-
-// device pointers of the cache (for callers that fill it with their own kernels)
-int32_t skn_kv_info(const skn_kvcache *kv, int32_t *batch, int32_t *n_kv_heads, int32_t *head_dim, int32_t *capacity,
-                    void **k_dev, void **v_dev, void **len_dev, void **start_dev) {
-    if (!kv_ok(kv)) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "bad kv cache handle");
-    if (batch) *batch = kv->batch;
-    if (n_kv_heads) *n_kv_heads = kv->n_kv_heads;
-    if (head_dim) *head_dim = kv->head_dim;
-    if (capacity) *capacity = kv->capacity;
-    if (k_dev) *k_dev = kv->d_k;
-    if (v_dev) *v_dev = kv->d_v;
-    if (len_dev) *len_dev = kv->d_len;
-    if (start_dev) *start_dev = kv->d_start;
     return SKN_OK;
 }
 

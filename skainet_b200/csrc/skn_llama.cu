@@ -191,7 +191,7 @@ static int32_t upload_gain(skn_llama *m, float *dst, const float *host) {
 }
 
 static bool shape_is(const skn_tensor *t, const skn_ctx *ctx, int64_t rows, int64_t cols) {
-    return skn_tensor_ok(t) && t->ctx == ctx && t->n_rows == rows && t->n_cols == cols;
+    return skn_tensor_ok(t) && t->ctx == ctx && t->type != SKN_TYPE_BF16 && t->n_rows == rows && t->n_cols == cols;
 }
 
 extern "C" {

@@ -17,89 +17,11 @@
 // fence.proxy.async before its warp arrives on the full barrier.  All waits are bounded.
 #include "skn_blocks.cuh"
 #include "skn_ptx.cuh"
-
-#include <cuda.h>
-#include <cuda_bf16.h>
+#include "skn_tc.cuh"
 
 constexpr int TC_BM = 128, TC_BN = 128, TC_BK = 64;
 constexpr int TC_TILE_BYTES = TC_BM * TC_BK * 2;   // 16 KB, one operand tile
 constexpr int TC_THREADS = 10 * 32;   // 8 dequant warps, 1 MMA warp, 1 TMA warp
-
-// ---- tcgen05 wrappers ---------------------------------------------------------------------
-__device__ __forceinline__ void tc_alloc(uint32_t *slot_smem, uint32_t ncols) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(skn_smem_u32(slot_smem)),
-                 "r"(ncols)
-                 : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tc_dealloc(uint32_t taddr, uint32_t ncols) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_commit(uint64_t *bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(skn_smem_u32(bar))
-                 : "memory");
-}
-// D[tmem] (+)= A[smem] * B[smem]^T, 128 x N x 16, bf16 in, fp32 out
-__device__ __forceinline__ void tc_mma_bf16(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc,
-                                            uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-        ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-// 32 lanes x 32 columns of 32-bit accumulators -> 32 registers per thread
-__device__ __forceinline__ void tc_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-          "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-          "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-          "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-        : "r"(taddr)
-        : "memory");
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
-
-// 2-D tiled TMA load (no multicast) of a box at element coordinates (x = column, y = row); the
-// tensor map's 128-byte swizzle lays the box out exactly as tc_store_chunk does
-__device__ __forceinline__ void tc_tma_load_2d(void *dst_smem, const CUtensorMap *tmap, int x, int y, uint64_t *bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-        ::"r"(skn_smem_u32(dst_smem)), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(x), "r"(y), "r"(skn_smem_u32(bar))
-        : "memory");
-}
-
-// Shared-memory matrix descriptor: K-major operand, rows of 64 bf16 (128 bytes) in 8-row
-// groups of 1024 bytes, 128-byte swizzle (16-byte chunk c of row r sits at chunk c ^ (r & 7)).
-__device__ __forceinline__ uint64_t tc_smem_desc(uint32_t smem_addr) {
-    uint64_t d = 0;
-    d |= (uint64_t)((smem_addr & 0x3FFFFu) >> 4);   // start address
-    d |= (uint64_t)1 << 16;                          // leading byte offset (unused for swizzled K-major)
-    d |= (uint64_t)(1024 >> 4) << 32;                // stride byte offset: 8 rows * 128 bytes
-    d |= (uint64_t)1 << 46;                          // descriptor version of this architecture
-    d |= (uint64_t)2 << 61;                          // swizzle mode: 128 bytes
-    return d;
-}
-// Instruction descriptor: fp32 accumulator, bf16 A and B, both K-major, M x N tile
-__device__ __forceinline__ uint32_t tc_idesc(int m, int n) {
-    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
-}
-
-// store 8 consecutive bf16 (one 16-byte chunk `c` of row `r`) into a swizzled tile
-__device__ __forceinline__ void tc_store_chunk(uint8_t *tile, int r, int c, uint4 v) {
-    *reinterpret_cast<uint4 *>(tile + (r >> 3) * 1024 + (r & 7) * 128 + ((c ^ (r & 7)) << 4)) = v;
-}
-
-__device__ __forceinline__ uint32_t tc_pack_bf16(float a, float b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t *>(&h);
-}
 
 // ---- 64 weights of one row -> one 128-byte bf16 row of the operand tile ------------------------
 // Generic form (any type): two 32-weight groups through the byte-granular decoder.
@@ -537,33 +459,6 @@ skn_matmul_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, int M, int K, c
     }
 }
 
-// ---------------------------------------------------------------------------------------------
-typedef CUresult (*skn_encode_tiled_fn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *,
-                                        const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
-                                        CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-// Tensor map of the bf16 activations [M][K]: boxes of 64 columns x 128 rows, 128-byte swizzle,
-// rows past M read as zeros.
-static cudaError_t make_a_tmap(const __nv_bfloat16 *A, int M, int K, CUtensorMap *out) {
-    static skn_encode_tiled_fn encode = nullptr;
-    if (!encode) {
-        void *fn = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q);
-        if (e != cudaSuccess) return e;
-        if (!fn || q != cudaDriverEntryPointSuccess) return cudaErrorNotSupported;
-        encode = (skn_encode_tiled_fn)fn;
-    }
-    const cuuint64_t gdim[2] = {(cuuint64_t)K, (cuuint64_t)M};
-    const cuuint64_t gstride[1] = {(cuuint64_t)K * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)TC_BK, (cuuint32_t)TC_BM};
-    const cuuint32_t estr[2] = {1, 1};
-    const CUresult r = encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<__nv_bfloat16 *>(A), gdim, gstride, box,
-                              estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
-                              CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    return r == CUDA_SUCCESS ? cudaSuccess : cudaErrorInvalidValue;
-}
-
 template <int TYPE, bool DUAL>
 static cudaError_t launch_tc(const __nv_bfloat16 *A, int M, int K, const skn_tensor *w, const skn_tensor *w2,
                              const float *bias, float *out_f32, __nv_bfloat16 *out_bf16, int64_t ld_out,
@@ -580,7 +475,7 @@ static cudaError_t launch_tc(const __nv_bfloat16 *A, int M, int K, const skn_ten
         attr_done[dev & 63] = true;
     }
     CUtensorMap tmap;
-    e0 = make_a_tmap(A, M, K, &tmap);
+    e0 = skn_tmap_bf16(A, M, K, (int64_t)K * 2, TC_BM, &tmap);
     if (e0 != cudaSuccess) return e0;
     // 256-row CTAs share each dequantised weight tile between two accumulators; when that leaves
     // SMs idle (few feature tiles), 128-row CTAs double the CTA count instead

@@ -305,6 +305,41 @@ class QuantTensor:
             pass
 
 
+BF16 = 30          # type id of dense bf16 weights (SKN_TYPE_BF16)
+
+
+def to_bf16_bits(a: np.ndarray) -> np.ndarray:
+    """fp32 -> bf16 bit patterns (uint16), rounded to nearest even."""
+    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def from_bf16_bits(b: np.ndarray) -> np.ndarray:
+    return (np.ascontiguousarray(b, dtype=np.uint16).astype(np.uint32) << 16).view(np.float32)
+
+
+class DenseTensor:
+    """A [out, in] weight of bf16 values in HBM, given as bf16 bit patterns (uint16) or as fp32 (rounded)."""
+
+    def __init__(self, ctx: Context, values: np.ndarray):
+        bits = np.ascontiguousarray(values if values.dtype == np.uint16 else to_bf16_bits(values))
+        if bits.ndim != 2:
+            raise ValueError("a dense weight is a rank-2 tensor [out, in]")
+        self.ctx, self.shape, self.quant_type = ctx, Shape(*bits.shape), BF16
+        self._h = ctypes.c_void_p()
+        rc = _ffi.lib().skn_tensor_upload_dense(ctx.handle, BF16, bits.shape[0], bits.shape[1], bits.ctypes.data, bits.nbytes,
+                                                ctypes.byref(self._h))
+        if rc != SKN_OK:
+            self._h = ctypes.c_void_p()
+            _raise(ctx.handle, rc)
+
+    handle = QuantTensor.handle
+    matmul_t = QuantTensor.matmul_t
+    matmul_t_dev = QuantTensor.matmul_t_dev
+    close = QuantTensor.close
+    __del__ = QuantTensor.__del__
+
+
 def ffn_swiglu(ctx: Context, wg: QuantTensor, wu: QuantTensor, wd: QuantTensor, x: np.ndarray) -> np.ndarray:
     """(silu(x Wg^T) * (x Wu^T)) Wd^T for x [M, K] (or [K]) on the host."""
     x = np.ascontiguousarray(x, dtype=np.float32)
