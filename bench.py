@@ -869,6 +869,156 @@ def run_decode(args):
         dist.destroy_process_group()
 
 
+# --------------------------------------------------------------------------------------------
+# --workload lugasun: the Lugasun decoder beside the Llama-style decoder of the same width and size
+# --------------------------------------------------------------------------------------------
+LUGASUN_SIZES = {
+    # width: heads, kv heads, head width, retention heads, their q/k and value widths, feed-forward, side width, layers
+    1024: (8, 2, 128, 8, 64, 64, 4096, 64, 8),
+    2048: (16, 4, 128, 8, 128, 128, 8192, 64, 8),
+    4096: (32, 8, 128, 16, 128, 128, 14336, 128, 8),
+}
+LUGASUN_CHUNK, LUGASUN_VOCAB, LUGASUN_PROMPT = 1024, 32000, 2048
+
+
+def lugasun_bench_configs(width: int):
+    """(Lugasun configuration, Llama configuration with as many parameters per layer)."""
+    from skainet_b200.llama import LlamaConfig
+    from skainet_b200.lugasun import LugasunConfig
+    H, G, D, RH, RD, RV, F, S, n = LUGASUN_SIZES[width]
+    layer = {"type": "parallel", "mlp": {"ff": F, "kind": "dense"},
+             "mixer": {"left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 50.0,
+                                "mask": {"size": LUGASUN_CHUNK}, "rot": {"base": 10000.0, "dims": D}},
+                       "right": {"heads": RH, "dim": RD, "vdim": RV, "rot": {"base": 10000.0, "dims": RD},
+                                 "decay": [1.0 - 2.0 ** -(5 + 5 * h / RH) for h in range(RH)]},
+                       "left_scale": 0.5, "right_scale": 0.5}}
+    cfg = LugasunConfig.from_dict({"vocab": LUGASUN_VOCAB, "width": width, "norm": {"eps": 1e-5}, "layers": [layer] * n,
+                                   "token_side": {"dim": S}, "loop": {"start": 1, "stop": n - 1, "times": 1}})
+    per_layer = sum(int(np.prod(v)) for k, v in cfg.tensor_shapes().items() if k.startswith("l0."))
+    ffn = max(256, round((per_layer - 2 * width * (H + G) * D) / (3 * width) / 256) * 256)
+    return cfg, LlamaConfig(n_layers=n, d_model=width, n_heads=H, n_kv_heads=G, head_dim=D, ffn_dim=ffn, vocab=LUGASUN_VOCAB)
+
+
+def _random_lugasun(ctx, cfg, **kw):
+    """Random weights; the layers share one set of values in buffers of their own."""
+    from skainet_b200.lugasun import LugasunDecoder
+    from skainet_b200.tensor import to_bf16_bits
+    g, cache = np.random.default_rng(7), {}
+
+    def get(name, shape):
+        key = name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name
+        if key not in cache:
+            a = np.ones(shape, np.float32) if len(shape) == 1 else \
+                g.standard_normal(size=shape, dtype=np.float32) * np.float32((1.0 if "embed" in key else shape[1] ** -0.5))
+            cache[key] = to_bf16_bits(a)
+        return cache[key]
+    return LugasunDecoder(ctx, cfg, **kw).load(get)
+
+
+def _random_llama(ctx, cfg, batch, T, max_ctx):
+    from skainet_b200 import synth
+    from skainet_b200.llama import LlamaDecoder
+    g = synth.rng(4)
+    qd, kd = cfg.n_heads * cfg.head_dim, cfg.n_kv_heads * cfg.head_dim
+    shapes = {"wq": (qd, cfg.d_model), "wk": (kd, cfg.d_model), "wv": (kd, cfg.d_model), "wo": (cfg.d_model, qd),
+              "w_gate": (cfg.ffn_dim, cfg.d_model), "w_up": (cfg.ffn_dim, cfg.d_model), "w_down": (cfg.d_model, cfg.ffn_dim)}
+    layer = {k: synth.make_weight(g, cfg.proj_type, *shp) for k, shp in shapes.items()}
+    emb = synth.make_weight(g, cfg.head_type, cfg.vocab, cfg.d_model)
+    dec = LlamaDecoder(ctx, cfg, batch=batch, max_tokens=T, max_ctx=max_ctx, kv_dtype="f16")
+    ones = np.ones(cfg.d_model, dtype=np.float32)
+    for i in range(cfg.n_layers):
+        dec.set_layer(i, layer, ones, ones)
+    dec.set_head(emb, ones, emb)
+    return dec
+
+
+def run_lugasun(args):
+    """Prefill of a LUGASUN_PROMPT-token prompt (batch 1) and greedy decode (batch 1 and 16, one CUDA graph replay per
+    step, after the prompt) of both decoders, random weights.  Weights exceed L2 from width 2048 on."""
+    import torch
+    import skainet_b200 as skn
+    torch.cuda.set_device(0)
+    ctx = skn.Context(0)
+    stream = torch.cuda.Stream()
+    torch.cuda.set_stream(stream)
+    ctx.set_stream(stream.cuda_stream)
+    T, steps = args.prompt, max(1, min(args.steps, 128))
+    max_ctx = T + 4 * steps + 160
+    rows = []
+    sampler = ClockSampler(0)
+    sampler.start()
+    for width in ([args.width] if args.width else sorted(LUGASUN_SIZES)):
+        lcfg, mcfg = lugasun_bench_configs(width)
+        dense = sum(int(np.prod(v)) for k, v in lcfg.tensor_shapes().items() if "embed" not in k)
+        for name in ([args.only] if args.only else ["lugasun", "llama"]):
+            row = {"model": name, "width": width, "layers": len(lcfg.layers), "parameters_in_layers": dense}
+            for B in ([args.batch] if args.only else [1, 16]):
+                # decode at batch B; the prompt is timed at batch 1
+                prompt_len = T if B == 1 else 512
+                g = np.random.default_rng(3)
+                toks = torch.from_numpy(g.integers(0, LUGASUN_VOCAB, size=(B, prompt_len)).astype(np.int32)).cuda()
+                if name == "lugasun":
+                    dec = _random_lugasun(ctx, lcfg, max_seqs=B, max_tokens=max(prompt_len, B), max_ctx=max_ctx)
+
+                    def prefill():
+                        dec.reset()
+                        for b in range(B):
+                            dec.forward_dev(toks[b], prompt_len, seq=b)
+
+                    def decode():
+                        dec.forward_dev(None, 1, seq=0, n=B)
+                else:
+                    # the Llama-style decoder advances all its sequences together: its prompt tokens go in portions
+                    per = prompt_len if B == 1 else 64
+                    dec = _random_llama(ctx, mcfg, B, per, max_ctx)
+                    parts = [toks[:, i:i + per].contiguous() for i in range(0, prompt_len, per)]
+
+                    def prefill():
+                        dec.reset()
+                        for p in parts:
+                            dec.forward_dev(p, per)
+
+                    def decode():
+                        dec.forward_dev(None, 1)
+                prefill()
+                decode()
+                if B == 1 and not args.no_prefill:
+                    ms = _events_ms(torch, stream, prefill, 5, 3)
+                    row.update(prefill_tokens=T, prefill_ms=ms, prefill_tok_s=T * 1e3 / ms)
+                    prefill()
+                graph = None
+                if not args.no_graph:
+                    cap = torch.cuda.Stream()
+                    cap.wait_stream(stream)
+                    graph = torch.cuda.CUDAGraph()
+                    with torch.cuda.stream(cap):
+                        ctx.set_stream(cap.cuda_stream)
+                        with torch.cuda.graph(graph, stream=cap):
+                            decode()
+                    ctx.set_stream(stream.cuda_stream)
+                    torch.cuda.synchronize()
+                    prefill()
+                ms = _events_ms(torch, stream, graph.replay if graph else decode, steps, 3)
+                ctx.sync()
+                row[f"decode_b{B}_ms"], row[f"decode_b{B}_tok_s"] = ms, B * 1e3 / ms
+                if name == "lugasun" and B == 1:
+                    row["decode_weight_gbs"] = 2 * (dense + LUGASUN_VOCAB * width) / (ms * 1e-3) / 1e9
+                del graph
+                dec.close()
+            rows.append(row)
+    clocks = sampler.stop()
+    peak, kind = measured_peak()
+    big = [r for r in rows if r["model"] == "lugasun"] or rows
+    print(json.dumps({
+        "metric": "lugasun_decode_tok_s", "value": big[-1].get("decode_b1_tok_s", big[-1].get(f"decode_b{args.batch}_tok_s")), "unit": "tok/s",
+        "n_gpus": 1, "steps": steps, "warmup": 3, "ms_per_step": None, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": f"Lugasun (bf16) beside a Llama-style decoder (Q4_K, fp16 cache) of the same width, layers and parameters "
+                               f"per layer; {T}-token prompt, chunks of {LUGASUN_CHUNK}, vocabulary {LUGASUN_VOCAB}"},
+        "hbm_peak_gbs": peak, "peak_kind": kind, "rows": rows, "clocks": clocks}), flush=True)
+    ctx.close()
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -895,11 +1045,15 @@ def main():
     ap.add_argument("--fused-exchange", default="auto", choices=["auto", "on", "off"],
                     help="tensor-parallel decode: push partial sums from the matvec epilogue (SKN_OPT_FUSED_EXCHANGE); "
                          "auto = the library's choice (off)")
-    ap.add_argument("--workload", default="matvec", choices=["matvec", "ffn", "attn", "sweep", "decode"],
+    ap.add_argument("--workload", default="matvec", choices=["matvec", "ffn", "attn", "sweep", "decode", "lugasun"],
                     help="matvec is the headline line; the others print one secondary JSON line (1 GPU)")
+    ap.add_argument("--width", type=int, default=0, choices=[0, *LUGASUN_SIZES], help="lugasun workload: this width only")
+    ap.add_argument("--only", default="", choices=["", "lugasun", "llama"], help="lugasun workload: this decoder only, at --batch")
+    ap.add_argument("--prompt", type=int, default=LUGASUN_PROMPT, help="lugasun workload: prompt tokens")
+    ap.add_argument("--no-prefill", action="store_true", help="lugasun workload: decode only")
     args = ap.parse_args()
     if args.impl == "ours" and args.workload != "matvec":
-        return {"ffn": run_ffn, "attn": run_attn, "sweep": run_sweep, "decode": run_decode}[args.workload](args)
+        return {"ffn": run_ffn, "attn": run_attn, "sweep": run_sweep, "decode": run_decode, "lugasun": run_lugasun}[args.workload](args)
     if args.impl == "reference":
         run_reference(args)
     else:
