@@ -1,8 +1,7 @@
 // Linear layers over dense bf16 weights [out][in] (row pitch a multiple of 16 bytes, rows zero-padded to it).
 //
-//  skn_dense_matvec_kernel   1 .. 4 activation rows, HBM-bound: x (fp32) is brought into shared memory once per CTA,
-//                            with the RMS norm folded in; a warp streams two weight rows at a time.  The first
-//                            weights of every warp are in flight before the kernel waits for its predecessor.
+//  skn_dense_matvec_kernel   1 .. 4 activation rows (fp32), HBM-bound: weight rows stream through shared memory in bulk
+//                            copies, the RMS norm of x is folded in
 //  skn_dense_f32_kernel      any number of rows, fp32 products and sums on the CUDA cores (the 32-bit mode)
 //  skn_dense_tc_kernel       tcgen05: a tile is 128 weight rows (TMEM lanes) x up to 256 tokens (TMEM columns), so
 //                            the same kernel serves a batch of decode rows (narrow tiles, split-K over the SMs)
@@ -31,66 +30,182 @@ __device__ __forceinline__ void dense_store(const skn_epi &e, int64_t m, int64_t
     if (e.y16) e.y16[m * e.ld_y16 + n] = __float2bfloat16_rn(v);
 }
 
+// NC consecutive tokens m .. of weight row n: everything the epilogue reads is loaded before the first store
+template <int EPI, int NC>
+__device__ __forceinline__ void dense_store_run(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count) {
+    if (EPI == SKN_EPI_ADD) {
+        float r[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) r[c] = c < count ? e.resid[(m + c) * e.ld_resid + n] : 0.f;
+#pragma unroll
+        for (int c = 0; c < NC; ++c) v[c] += r[c];
+    }
+    if (EPI == SKN_EPI_GELU_TABLE) {
+        float r[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            int64_t id = c < count ? e.ids[m + c] : 0;
+            if (id < 0 || id >= e.table_rows) id = 0;
+            r[c] = __bfloat162float(e.table[id * e.ld_table + e.table_col + n]);
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) v[c] = dense_gelu_tanh(v[c]) * r[c];
+    }
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        if (EPI == SKN_EPI_RELU2) {
+            v[c] = fmaxf(v[c], 0.f);
+            v[c] *= v[c];
+        }
+        if (c < count) {
+            if (e.y32) e.y32[(m + c) * e.ld_y32 + n] = v[c];
+            if (e.y16) e.y16[(m + c) * e.ld_y16 + n] = __float2bfloat16_rn(v[c]);
+        }
+    }
+}
+
 __device__ __forceinline__ float bf_lo(uint32_t w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 0xFFFF0000u); }
 
 // ---- matvec ------------------------------------------------------------------------------------------------
-constexpr int MVD_THREADS = 512, MVD_WARPS = MVD_THREADS / 32, MVD_U = 4;
+// CTA b owns the weight rows [b N / grid, (b + 1) N / grid): a producer warp streams them, a few rows per bulk copy, through
+// a ring of shared-memory stages and starts before the kernel waits for its predecessor; eight warps each take an eighth of
+// the columns of every row.  Their partial sums meet in shared memory, 128 rows at a time.  One activation row lives in
+// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).
+constexpr int MVD_WARPS = 8, MVD_THREADS = (MVD_WARPS + 1) * 32, MVD_ROWS = 128;
+constexpr int MVD_RING = 96 * 1024, MVD_MAX_STAGES = 24;
+// dynamic shared memory beside the partial sums of MR rows
+constexpr int mvd_smem(int mr) { return 224 * 1024 - mr * 2 * MVD_WARPS * MVD_ROWS * 4; }
+// rows of a stage: about 16 KB of weights
+__host__ __device__ constexpr int mvd_stage_rows(int mr, int uu) { return uu == 0 ? (mr > 1 ? 2 : 1) : uu == 1 ? 4 : uu == 2 ? 2 : 1; }
 
-template <int MR, int EPI>
-__global__ void __launch_bounds__(MVD_THREADS, 1)
-skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int K, int m0, const float *__restrict__ x, int64_t ldx,
-                        const float *__restrict__ xb, int64_t ldxb, int ka, const float *__restrict__ gain, float eps, skn_epi e) {
-    extern __shared__ float xs[];                  // [MR][2 planes][K8 / 2]: quads 0 and 1 of every eight columns
-    __shared__ float red[MVD_WARPS][MR];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2;
-    const int pairs = (N + 1) / 2;
-    const int stride = gridDim.x * MVD_WARPS;
-    int pair = warp * gridDim.x + blockIdx.x;
+__device__ __forceinline__ void mvd_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-    uint4 wa[MVD_U], wb[MVD_U];
-    auto load = [&](int p, int i0) {
-        const bool two = 2 * p + 1 < N;
-        const uint4 *ra = reinterpret_cast<const uint4 *>(W + (int64_t)(2 * p) * pitch);
-        const uint4 *rb = reinterpret_cast<const uint4 *>(W + (int64_t)(2 * p + 1) * pitch);
-#pragma unroll
-        for (int u = 0; u < MVD_U; ++u) {
-            const int i = i0 + u * 32 + lane;
-            const bool in = i < nv;
-            wa[u] = in ? __ldg(ra + i) : make_uint4(0u, 0u, 0u, 0u);
-            wb[u] = in && two ? __ldg(rb + i) : make_uint4(0u, 0u, 0u, 0u);
-        }
-    };
-    if (pair < pairs) load(pair, 0);
-    skn_pdl_launch_dependents();
-    skn_pdl_wait();
-
-    float ss[MR];
-#pragma unroll
-    for (int m = 0; m < MR; ++m) {
-        ss[m] = 0.f;
-        const float *xr = x + (int64_t)(m0 + m) * ldx;
-        const float *xbr = xb ? xb + (int64_t)(m0 + m) * ldxb - ka : xr;
-        float *dst = xs + m * K8;
-#pragma unroll 4
-        for (int k = threadIdx.x; k < K8; k += MVD_THREADS) {
-            float v = 0.f;
-            if (k < K) v = __ldcg(k < ka ? xr + k : xbr + k);
-            ss[m] = fmaf(v, v, ss[m]);
-            if (gain && k < K) v *= __ldg(gain + k);
-            dst[((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] = v;
-        }
+__device__ __forceinline__ void dense_store_any(const skn_epi &e, int64_t m, int64_t n, float v) {
+    switch (e.kind) {
+    case SKN_EPI_ADD: dense_store<SKN_EPI_ADD>(e, m, n, v); break;
+    case SKN_EPI_RELU2: dense_store<SKN_EPI_RELU2>(e, m, n, v); break;
+    case SKN_EPI_GELU_TABLE: dense_store<SKN_EPI_GELU_TABLE>(e, m, n, v); break;
+    default: dense_store<SKN_EPI_STORE>(e, m, n, v); break;
     }
-    if (gain) {
-#pragma unroll
-        for (int m = 0; m < MR; ++m) {
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) ss[m] += __shfl_xor_sync(0xffffffffu, ss[m], o);
-            if (lane == 0) red[warp][m] = ss[m];
+}
+
+__device__ __forceinline__ float mvd_dot8(const uint4 &w, const float4 &lo, const float4 &hi, float a) {
+    a = fmaf(bf_lo(w.x), lo.x, a); a = fmaf(bf_hi(w.x), lo.y, a); a = fmaf(bf_lo(w.y), lo.z, a); a = fmaf(bf_hi(w.y), lo.w, a);
+    a = fmaf(bf_lo(w.z), hi.x, a); a = fmaf(bf_hi(w.z), hi.y, a); a = fmaf(bf_lo(w.w), hi.z, a); return fmaf(bf_hi(w.w), hi.w, a);
+}
+// row of the eight whose sum this lane holds after the joint reduction
+__device__ __forceinline__ int mvd_row(int lane) { return ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1); }
+
+template <int MR, int UU>
+__global__ void __launch_bounds__(MVD_THREADS, 2)
+skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int K, int m0, const float *x, int64_t ldx, const float *xb,
+                        int64_t ldxb, int ka, const float *__restrict__ gain, float eps, int stages, skn_epi e, int32_t *status) {
+    extern __shared__ __align__(128) uint8_t ring[];
+    constexpr int GR = mvd_stage_rows(MR, UU);
+    __shared__ uint64_t full_bar[MVD_MAX_STAGES], empty_bar[MVD_MAX_STAGES];
+    __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2, per = (nv + MVD_WARPS - 1) / MVD_WARPS;
+    const int r0 = (int)((int64_t)N * blockIdx.x / gridDim.x), r1 = (int)((int64_t)N * (blockIdx.x + 1) / gridDim.x);
+    const int steps = (r1 - r0 + GR - 1) / GR;
+    const size_t stage_bytes = (size_t)GR * pitch;
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < stages; ++s) {
+            skn_mbar_init(&full_bar[s], 1);
+            skn_mbar_init(&empty_bar[s], MVD_WARPS);
         }
+        skn_fence_mbar_init();
     }
     __syncthreads();
+    skn_pdl_launch_dependents();
+    if (warp == MVD_WARPS) {
+        if (lane == 0) {
+            int s = 0;
+            uint32_t phase = 1;
+            for (int i = 0; i < steps; ++i) {
+                const int row = r0 + i * GR;
+                if (!skn_mbar_wait(&empty_bar[s], phase)) {
+                    atomicExch(status, SKN_ERR_TIMEOUT);
+                    break;
+                }
+                const uint32_t bytes = (uint32_t)(min(GR, r1 - row) * pitch);
+                skn_mbar_expect_tx(&full_bar[s], bytes);
+                skn_bulk_g2s(ring + s * stage_bytes, W + (int64_t)row * pitch, bytes, &full_bar[s]);
+                if (++s == stages) {
+                    s = 0;
+                    phase ^= 1u;
+                }
+            }
+        }
+        skn_pdl_wait();
+        return;
+    }
+    skn_pdl_wait();
+
+    // this warp's columns: vectors v0 + lane + 32 u below v1
+    const int v0 = warp * per, v1 = min(nv, v0 + per);
+    float4 xr[UU > 0 ? 2 * UU : 1];
+    float *xs = reinterpret_cast<float *>(ring + stages * stage_bytes);     // UU = 0: [MR][2 planes][K8 / 2]: quads 0 and 1 of every eight columns
+    float ss[MR];
+    auto fetch = [&](int m, int k) {
+        float v = 0.f;
+        if (k < K) v = __ldcg(k < ka ? x + (int64_t)(m0 + m) * ldx + k : xb + (int64_t)(m0 + m) * ldxb + k - ka);
+        return v;
+    };
+    if constexpr (UU > 0) {
+        // rows that are whole aligned vectors (the usual case) are read 16 bytes at a time
+        const bool vec = K % 8 == 0 && ka % 8 == 0 && ldx % 4 == 0 && ldxb % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xb)) & 15) == 0;
+        float q = 0.f;
+#pragma unroll
+        for (int u = 0; u < UU; ++u) {
+            const int i = v0 + u * 32 + lane;
+            float f[8];
+            const int k = i * 8;
+            if (vec && i < v1) {
+                const float *p = k < ka ? x + (int64_t)m0 * ldx + k : xb + (int64_t)m0 * ldxb + k - ka;
+                *reinterpret_cast<float4 *>(f) = __ldcg(reinterpret_cast<const float4 *>(p));
+                *reinterpret_cast<float4 *>(f + 4) = __ldcg(reinterpret_cast<const float4 *>(p + 4));
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) f[j] = i < v1 ? fetch(0, k + j) : 0.f;
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) q = fmaf(f[j], f[j], q);
+            if (gain && i < v1) {
+                if (vec) {
+                    const float4 g0 = __ldg(reinterpret_cast<const float4 *>(gain + k)), g1 = __ldg(reinterpret_cast<const float4 *>(gain + k + 4));
+                    f[0] *= g0.x; f[1] *= g0.y; f[2] *= g0.z; f[3] *= g0.w;
+                    f[4] *= g1.x; f[5] *= g1.y; f[6] *= g1.z; f[7] *= g1.w;
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 8; ++j)
+                        if (k + j < K) f[j] *= __ldg(gain + k + j);
+                }
+            }
+            xr[2 * u] = make_float4(f[0], f[1], f[2], f[3]);
+            xr[2 * u + 1] = make_float4(f[4], f[5], f[6], f[7]);
+        }
+        ss[0] = q;
+    } else {
+#pragma unroll
+        for (int m = 0; m < MR; ++m) {
+            ss[m] = 0.f;
+            for (int k = threadIdx.x; k < K8; k += MVD_WARPS * 32) {
+                float v = fetch(m, k);
+                ss[m] = fmaf(v, v, ss[m]);
+                if (gain && k < K) v *= __ldg(gain + k);
+                xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] = v;
+            }
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < MR; ++m) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) ss[m] += __shfl_xor_sync(0xffffffffu, ss[m], o);
+        if (lane == 0) red[warp][m] = ss[m];
+    }
+    mvd_barrier();
     float rs[MR];
 #pragma unroll
     for (int m = 0; m < MR; ++m) {
@@ -103,97 +218,140 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
         }
     }
 
-    float a0[MR], a1[MR];
+    // eight rows at a time: their sums are reduced across the warp together (9 shuffles for 8 rows)
+    bool ok = true;
+    int buf = 0, filled = 0, base = r0;            // rows base .. base + filled - 1 have partial sums in part[buf]
+    int s = 0;
+    uint32_t phase = 0;
+    const uint4 *w = reinterpret_cast<const uint4 *>(ring);
+    for (int g0 = 0; g0 < r1 - r0; g0 += 8) {
+        float acc[MR][8];
 #pragma unroll
-    for (int m = 0; m < MR; ++m) a0[m] = a1[m] = 0.f;
-    int i0 = 0;
-    while (pair < pairs) {
+        for (int m = 0; m < MR; ++m)
 #pragma unroll
-        for (int u = 0; u < MVD_U; ++u) {
-            const int i = i0 + u * 32 + lane;
-            if (i < nv) {
-                const uint4 p = wa[u], q = wb[u];
+            for (int j = 0; j < 8; ++j) acc[m][j] = 0.f;
+        const int rows = min(8, r1 - r0 - g0);
 #pragma unroll
-                for (int m = 0; m < MR; ++m) {
-                    const float4 lo = *reinterpret_cast<const float4 *>(xs + m * K8 + i * 4);
-                    const float4 hi = *reinterpret_cast<const float4 *>(xs + m * K8 + half + i * 4);
-                    float s = a0[m], t = a1[m];
-                    s = fmaf(bf_lo(p.x), lo.x, s); s = fmaf(bf_hi(p.x), lo.y, s); s = fmaf(bf_lo(p.y), lo.z, s); s = fmaf(bf_hi(p.y), lo.w, s);
-                    s = fmaf(bf_lo(p.z), hi.x, s); s = fmaf(bf_hi(p.z), hi.y, s); s = fmaf(bf_lo(p.w), hi.z, s); s = fmaf(bf_hi(p.w), hi.w, s);
-                    t = fmaf(bf_lo(q.x), lo.x, t); t = fmaf(bf_hi(q.x), lo.y, t); t = fmaf(bf_lo(q.y), lo.z, t); t = fmaf(bf_hi(q.y), lo.w, t);
-                    t = fmaf(bf_lo(q.z), hi.x, t); t = fmaf(bf_hi(q.z), hi.y, t); t = fmaf(bf_lo(q.w), hi.z, t); t = fmaf(bf_hi(q.w), hi.w, t);
-                    a0[m] = s;
-                    a1[m] = t;
+        for (int j0 = 0; j0 < 8; j0 += GR) {
+            if (j0 < rows) {
+                if (ok && !skn_mbar_wait(&full_bar[s], phase)) {
+                    if (lane == 0) atomicExch(status, SKN_ERR_TIMEOUT);
+                    ok = false;
+                }
+                // (rows past the CTA's last one are old bytes of the ring: multiplied, never stored)
+                if constexpr (UU > 0) {
+                    float odd[GR] = {};            // two chains
+#pragma unroll
+                    for (int u = 0; u < UU; ++u) {
+                        const int c = v0 + u * 32 + lane;
+                        if (c < v1) {
+#pragma unroll
+                            for (int j = 0; j < GR; ++j) {
+                                float &t = (u & 1) ? odd[j] : acc[0][j0 + j];
+                                t = mvd_dot8(w[j * nv + c], xr[2 * u], xr[2 * u + 1], t);
+                            }
+                        }
+                    }
+#pragma unroll
+                    for (int j = 0; j < GR; ++j) acc[0][j0 + j] += odd[j];
+                } else {
+                    for (int c = v0 + lane; c < v1; c += 32) {
+                        uint4 p[GR];
+#pragma unroll
+                        for (int j = 0; j < GR; ++j) p[j] = w[j * nv + c];
+#pragma unroll
+                        for (int m = 0; m < MR; ++m) {
+                            const float4 lo = *reinterpret_cast<const float4 *>(xs + m * K8 + c * 4), hi = *reinterpret_cast<const float4 *>(xs + m * K8 + half + c * 4);
+#pragma unroll
+                            for (int j = 0; j < GR; ++j) acc[m][j0 + j] = mvd_dot8(p[j], lo, hi, acc[m][j0 + j]);
+                        }
+                    }
+                }
+                __syncwarp();
+                if (lane == 0) skn_mbar_arrive(&empty_bar[s]);
+                if (++s == stages) {
+                    s = 0;
+                    phase ^= 1u;
+                    w = reinterpret_cast<const uint4 *>(ring);
+                } else {
+                    w += GR * nv;
                 }
             }
         }
-        const int done = pair;
-        i0 += 32 * MVD_U;
-        const bool last = i0 >= nv;
-        if (last) {
-            i0 = 0;
-            pair += stride;
-        }
-        if (pair < pairs) load(pair, i0);
-        if (last) {
-            float mine = 0.f;
 #pragma unroll
-            for (int m = 0; m < MR; ++m) {
+        for (int m = 0; m < MR; ++m) {
 #pragma unroll
-                for (int o = 16; o > 0; o >>= 1) {
-                    a0[m] += __shfl_xor_sync(0xffffffffu, a0[m], o);
-                    a1[m] += __shfl_xor_sync(0xffffffffu, a1[m], o);
+            for (int o = 16, n = 4; o >= 4; o >>= 1, n >>= 1)
+#pragma unroll
+                for (int j = 0; j < n; ++j) {
+                    const bool up = lane & o;
+                    const float mine = up ? acc[m][j + n] : acc[m][j], other = up ? acc[m][j] : acc[m][j + n];
+                    acc[m][j] = mine + __shfl_xor_sync(0xffffffffu, other, o);
                 }
-                if (lane == 2 * m) mine = a0[m] * rs[m];
-                if (lane == 2 * m + 1) mine = a1[m] * rs[m];
-                a0[m] = a1[m] = 0.f;
+            float t = acc[m][0];
+            t += __shfl_xor_sync(0xffffffffu, t, 2);
+            t += __shfl_xor_sync(0xffffffffu, t, 1);
+            if ((lane & 3) == 0) part[buf][m][warp][filled + mvd_row(lane)] = t * rs[m];
+        }
+        filled += rows;
+        if (filled + 8 > MVD_ROWS || g0 + 8 >= r1 - r0) {
+            mvd_barrier();
+            for (int j = threadIdx.x; j < filled * MR; j += MVD_WARPS * 32) {
+                const int m = j / filled, r = j % filled;
+                float t = 0.f;
+#pragma unroll
+                for (int w8 = 0; w8 < MVD_WARPS; ++w8) t += part[buf][m][w8][r];
+                dense_store_any(e, m0 + m, base + r, t);
             }
-            const int n = 2 * done + (lane & 1);
-            if (lane < 2 * MR && n < N) dense_store<EPI>(e, m0 + (lane >> 1), n, mine);
+            base += filled;
+            filled = 0;
+            buf ^= 1;                              // the other half is free: every warp has passed the barrier of its readers
         }
     }
 }
 
-template <int MR, int EPI>
+template <int MR, int UU>
 static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int m0, cudaStream_t st) {
-    auto kern = skn_dense_matvec_kernel<MR, EPI>;
-    const int K8 = (int)(l.w->pitch / 2);
-    const size_t smem = (size_t)MR * K8 * sizeof(float);
+    auto kern = skn_dense_matvec_kernel<MR, UU>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
-        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, mvd_smem(MR));
         if (e != cudaSuccess) return e;
         attr_done[ctx->device & 63] = true;
     }
-    const int pairs = (int)((l.w->n_rows + 1) / 2);
-    int grid = (pairs + MVD_WARPS - 1) / MVD_WARPS;
-    // few rows: one warp per CTA has work, so that every SM takes part
-    if (grid < ctx->sm_count) grid = pairs < ctx->sm_count ? pairs : ctx->sm_count;
-    if (grid > ctx->sm_count) grid = ctx->sm_count;
-    const int K = (int)l.w->n_cols;
-    return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), smem, st, 1, (const uint8_t *)l.w->d_blocks, l.w->pitch, (int)l.w->n_rows, K,
-                          m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, l.gain, l.eps, l.epi);
-}
-
-template <int MR>
-static cudaError_t dispatch_mvd(skn_ctx *ctx, const skn_linear &l, int m0, cudaStream_t st) {
-    switch (l.epi.kind) {
-    case SKN_EPI_STORE: return launch_mvd<MR, SKN_EPI_STORE>(ctx, l, m0, st);
-    case SKN_EPI_ADD: return launch_mvd<MR, SKN_EPI_ADD>(ctx, l, m0, st);
-    case SKN_EPI_RELU2: return launch_mvd<MR, SKN_EPI_RELU2>(ctx, l, m0, st);
-    case SKN_EPI_GELU_TABLE: return launch_mvd<MR, SKN_EPI_GELU_TABLE>(ctx, l, m0, st);
-    }
-    return cudaErrorInvalidValue;
+    const int64_t pitch = l.w->pitch;
+    const int N = (int)l.w->n_rows, K = (int)l.w->n_cols, rows = mvd_stage_rows(MR, UU);
+    const size_t xbytes = UU > 0 ? 0 : (size_t)MR * pitch * 2;
+    size_t room = mvd_smem(MR) - xbytes;
+    if (room > (size_t)MVD_RING) room = MVD_RING;
+    int stages = (int)(room / (rows * pitch));
+    if (stages < 1) return cudaErrorNotSupported;
+    if (stages > MVD_MAX_STAGES) stages = MVD_MAX_STAGES;
+    const int grid = N < ctx->sm_count ? N : ctx->sm_count;
+    return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks, pitch,
+                          N, K, m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, l.gain, l.eps, stages, l.epi, ctx->d_status);
 }
 
 cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStream_t st) {
-    const size_t row = (size_t)l.w->pitch * 2;            // one activation row in shared memory
-    int fit = (int)((size_t)200 * 1024 / row);
-    if (fit < 1) return cudaErrorNotSupported;
+    const int64_t pitch = l.w->pitch;
+    if (pitch * 3 > mvd_smem(1)) return cudaErrorNotSupported;       // one stage and one activation row must fit
+    const int uu = (int)(((pitch / 16 + MVD_WARPS - 1) / MVD_WARPS + 31) / 32);
     for (int m0 = 0; m0 < l.M;) {
         const int left = l.M - m0;
-        int mr = left >= 4 && fit >= 4 ? 4 : left >= 2 && fit >= 2 ? 2 : 1;
-        const cudaError_t e = mr == 4 ? dispatch_mvd<4>(ctx, l, m0, st) : mr == 2 ? dispatch_mvd<2>(ctx, l, m0, st) : dispatch_mvd<1>(ctx, l, m0, st);
+        cudaError_t e;
+        int mr = 1;
+        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0>(ctx, l, m0, st); }
+        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0>(ctx, l, m0, st); }
+        else switch (uu) {
+            case 1: e = launch_mvd<1, 1>(ctx, l, m0, st); break;
+            case 2: e = launch_mvd<1, 2>(ctx, l, m0, st); break;
+            case 3: e = launch_mvd<1, 3>(ctx, l, m0, st); break;
+            case 4: e = launch_mvd<1, 4>(ctx, l, m0, st); break;
+            case 5: e = launch_mvd<1, 5>(ctx, l, m0, st); break;
+            case 6: e = launch_mvd<1, 6>(ctx, l, m0, st); break;
+            case 7: e = launch_mvd<1, 7>(ctx, l, m0, st); break;
+            default: e = launch_mvd<1, 0>(ctx, l, m0, st); break;
+        }
         if (e != cudaSuccess) return e;
         m0 += mr;
     }
@@ -307,6 +465,16 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     tc_fence_after();
     const uint32_t tmem = tmem_slot;
     skn_pdl_launch_dependents();
+    // the weights depend on no kernel before this one: the first unit's first stages are requested ahead of the wait
+    int early = 0;
+    if (warp == 5 && lane == 0 && (int)blockIdx.x < units) {
+        const int sp = (blockIdx.x / mt) % splits, n0 = (blockIdx.x / mt / splits) * DTC_BM;
+        const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
+        for (; early < stages && early < ke - kb; ++early) {
+            skn_mbar_expect_tx(&full_bar[early], (uint32_t)stage_bytes);
+            tc_tma_load_2d(smem + (size_t)early * stage_bytes, &tmap_w, (kb + early) * DTC_BK, n0, &full_bar[early]);
+        }
+    }
     skn_pdl_wait();
 
     if (warp == 5) {
@@ -318,14 +486,16 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
                 for (int k = kb; k < ke; ++k, ++it) {
                     const int s = it % stages;
-                    if (!skn_mbar_wait(&empty_bar[s], ((uint32_t)(it / stages) & 1u) ^ 1u)) {
-                        atomicExch(status, SKN_ERR_TIMEOUT);
-                        ok = false;
-                        break;
-                    }
                     uint8_t *a = smem + (size_t)s * stage_bytes;
-                    skn_mbar_expect_tx(&full_bar[s], (uint32_t)stage_bytes);
-                    tc_tma_load_2d(a, &tmap_w, k * DTC_BK, n0, &full_bar[s]);
+                    if (it >= early) {
+                        if (!skn_mbar_wait(&empty_bar[s], ((uint32_t)(it / stages) & 1u) ^ 1u)) {
+                            atomicExch(status, SKN_ERR_TIMEOUT);
+                            ok = false;
+                            break;
+                        }
+                        skn_mbar_expect_tx(&full_bar[s], (uint32_t)stage_bytes);
+                        tc_tma_load_2d(a, &tmap_w, k * DTC_BK, n0, &full_bar[s]);
+                    }
                     tc_tma_load_2d(a + DTC_A_BYTES, &tmap_x, k * DTC_BK, m0, &full_bar[s]);
                 }
             }
@@ -391,14 +561,10 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 tc_ld32(src + c0, acc);
                 if (splits == 1) {
                     if (n < N && ok) {
-                        if (cols - c0 >= 32) {
+                        float v[32];
 #pragma unroll
-                            for (int c = 0; c < 32; ++c) dense_store<EPI>(e, m0 + c0 + c, n, __uint_as_float(acc[c]));
-                        } else {
-#pragma unroll
-                            for (int c = 0; c < 32; ++c)
-                                if (c0 + c < cols) dense_store<EPI>(e, m0 + c0 + c, n, __uint_as_float(acc[c]));
-                        }
+                        for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
+                        dense_store_run<EPI, 32>(e, m0 + c0, n, v, cols - c0);
                     }
                 } else {
 #pragma unroll
@@ -417,10 +583,15 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 dtc_barrier_epilogue();
                 if (last_flag) {
                     __threadfence();
-                    for (int c = 0; c < cols; ++c) {
-                        float v = 0.f;
-                        for (int s = 0; s < splits; ++s) v += __ldcg(pbase + ((size_t)s * NT + c) * DTC_BM);
-                        if (n < N && ok) dense_store<EPI>(e, m0 + c, n, v);
+                    for (int c0 = 0; c0 < cols; c0 += 16) {
+                        float v[16];
+#pragma unroll
+                        for (int c = 0; c < 16; ++c) v[c] = 0.f;
+#pragma unroll 2
+                        for (int s = 0; s < splits; ++s)
+#pragma unroll
+                            for (int c = 0; c < 16; ++c) v[c] += __ldcg(pbase + ((size_t)s * NT + c0 + c) * DTC_BM);
+                        if (n < N && ok) dense_store_run<EPI, 16>(e, m0 + c0, n, v, cols - c0);
                     }
                     if (threadIdx.x == 0) tickets[tidx] = 0;
                 }
@@ -448,21 +619,45 @@ static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense
     }
     const int N = (int)l.w->n_rows, K = (int)l.w->n_cols, M = l.M, sms = ctx->sm_count;
     const int nt = (N + DTC_BM - 1) / DTC_BM;
-    // token tile: the narrowest that covers M, at most 256; halved while that leaves SMs without a tile
+    const int ksteps = (K + DTC_BK - 1) / DTC_BK;
+    // token tile: the narrowest that covers M; beyond that, of the widths whose operands the shared memory feeds at full
+    // rate, the one with the least time in waves (a wave of narrower tiles costs less, but loads more per product)
     int NT = 16;
-    while (NT < 256 && NT < M) NT *= 2;
-    while (NT > 64 && nt * ((M + NT - 1) / NT) < sms) NT /= 2;
-    const int mt = (M + NT - 1) / NT, ksteps = (K + DTC_BK - 1) / DTC_BK;
+    if (M <= 128) {
+        while (NT < M) NT *= 2;
+    } else {
+        const int width[3] = {256, 192, 128};
+        const double rate[3] = {1.0, 1.03, 1.12};
+        double best = 1e30;
+        for (int i = 0; i < 3; ++i) {
+            const int64_t tiles = (int64_t)nt * ((M + width[i] - 1) / width[i]);
+            const double cost = (double)((tiles + sms - 1) / sms) * (width[i] + 8) * rate[i];
+            if (cost < best) {
+                best = cost;
+                NT = width[i];
+            }
+        }
+    }
+    while (NT > 64 && nt * ((M + NT - 1) / NT) * 2 <= sms) NT = NT == 192 ? 128 : NT / 2;
+    const int mt = (M + NT - 1) / NT;
+    // K splits that even out the load of the SMs (the tiles of a decode-size step are fewer than the SMs, or not many more)
     int splits = 1;
-    if (mt * nt < sms && mt * nt <= SKN_DENSE_MAX_TILES) {
-        splits = sms / (mt * nt);
-        if (splits > ksteps / 4) splits = ksteps / 4;                // at least four K steps each
-        if (splits > 16) splits = 16;
-        while (splits > 1 && (size_t)mt * nt * splits * NT * DTC_BM > SKN_DENSE_WS_FLOATS) --splits;
-        if (splits < 1) splits = 1;
+    if (mt * nt < 2 * sms && mt * nt <= SKN_DENSE_MAX_TILES) {
+        double best = 1e30;
+        for (int s = 1; s <= 16 && (s == 1 || s <= ksteps / 4); ++s) {
+            if (s > 1 && (size_t)mt * nt * s * NT * DTC_BM > SKN_DENSE_WS_FLOATS) break;
+            const int64_t waves = ((int64_t)mt * nt * s + sms - 1) / sms;
+            // per unit: its K steps, a fixed cost, and the partial sums that go out and come back
+            const double cost = waves * ((double)ksteps / s + 2.0 + (s > 1 ? NT / 16.0 : 0.0)) + (s > 1 ? s * NT / 32.0 : 0.0);
+            if (cost < best * 0.97) {
+                best = cost;
+                splits = s;
+            }
+        }
     }
     const int stage_bytes = DTC_A_BYTES + NT * DTC_BK * 2;
-    int stages = DTC_SMEM / stage_bytes;
+    // narrow tiles leave room for the CTA of the next launch, which then requests its weights early
+    int stages = (NT <= 64 ? DTC_SMEM / 2 : DTC_SMEM) / stage_bytes;
     if (stages > DTC_MAX_STAGES) stages = DTC_MAX_STAGES;
     CUtensorMap tw, tx;
     cudaError_t e = skn_tmap_bf16(l.w->d_blocks, N, K, l.w->pitch, DTC_BM, &tw);

@@ -81,6 +81,7 @@ cudaError_t skn_launch_rows_to_bf16(const float *in, int64_t ld, int M, int D, _
 cudaError_t skn_launch_concat_bf16(const float *a, const float *b, int64_t ld, int M, int D, __nv_bfloat16 *out, int64_t ldo, cudaStream_t st);
 // Token side input of a few rows in one launch (a cluster of 8 CTAs per row):
 //   g = gelu_tanh(Wg x) * table[id][col ..], y = Wp g, x += y / sqrt(mean(y^2) + eps) * gain
+bool skn_token_side_fits(const skn_tensor *wg, const skn_tensor *wp);
 cudaError_t skn_launch_token_side(const skn_tensor *wg, const skn_tensor *wp, const skn_tensor *table, int64_t col, const int32_t *ids,
                                   float *x, int64_t ldx, int M, const float *gain, float eps, cudaStream_t st);
 

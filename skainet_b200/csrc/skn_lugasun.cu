@@ -1,7 +1,7 @@
 // The Lugasun decoder over dense bf16 weights: one step is a fixed sequence of launches on the context's stream, all
 // with programmatic dependent launch and capturable in a CUDA graph.  Three routes share the buffers and the mixers:
 //
-//   few rows (<= SKN_MATVEC_ROWS)   fp32 activations: norm + joint projection | attention + state update | output
+//   few rows                        fp32 activations: norm + joint projection | attention + state update | output
 //                                   projection + residual | norm + up + relu^2 | down + residual | token side input
 //   bf16, more rows                 tcgen05 products of bf16 rows; relu^2, the residual sum and the side gate in their
 //                                   epilogues, norms as row kernels (the side input's norm joins the next layer's)
@@ -35,6 +35,8 @@ struct Rot {
     float2 *table;
 };
 
+constexpr int BF16_MATVEC_ROWS = 2;
+constexpr int SIDE_ROWS = 16;                    // rows whose token side input takes one launch
 constexpr int HEAD_ROWS = 64;                    // rows of logits computed at a time
 
 inline int64_t up8(int64_t n) { return (n + 7) / 8 * 8; }
@@ -191,8 +193,13 @@ static bool dense_is(const skn_tensor *t, const skn_ctx *ctx, int64_t rows, int6
     return skn_tensor_ok(t) && t->ctx == ctx && t->type == SKN_TYPE_BF16 && t->n_rows == rows && t->n_cols == cols;
 }
 
-// one row of x in the matvec kernel's shared memory
-static bool fits_matvec(const skn_tensor *t) { return !t || t->pitch * 2 <= 200 * 1024; }
+// a weight row and one activation row in the matvec kernel's shared memory
+static bool fits_matvec(const skn_tensor *t) { return !t || t->pitch <= 64 * 1024; }
+
+// rows of a step that take the matvec route; with bf16 operands the tensor-core kernel is faster beyond BF16_MATVEC_ROWS
+static bool is_few(const skn_lugasun *m, int rows) {
+    return m->matvec_ok && rows <= (m->dtype == SKN_LUGASUN_F32 ? SKN_MATVEC_ROWS : BF16_MATVEC_ROWS);
+}
 
 // The three routes of a linear layer.  in32 / in16: the same rows in either form (in16 only where bf16 rows run).
 static cudaError_t linear(skn_lugasun *m, bool few, const skn_tensor *w, int M, const float *in32, int64_t ld32, const __nv_bfloat16 *in16,
@@ -226,7 +233,7 @@ static int32_t run_layers(skn_lugasun *m, const skn_step &st, const int32_t *ids
     cudaStream_t s = ctx->stream;
     const skn_lugasun_spec &sp = m->spec;
     const int M = st.n_seqs * st.T, W = sp.width;
-    const bool few = M <= SKN_MATVEC_ROWS && m->matvec_ok, f32 = m->dtype == SKN_LUGASUN_F32, rows32 = few || f32;
+    const bool f32 = m->dtype == SKN_LUGASUN_F32, few = is_few(m, M), rows32 = few || f32;
     const int64_t ldw = m->ldw;
     m->x = m->xa;
     m->xalt = m->xb;
@@ -284,7 +291,8 @@ static int32_t run_layers(skn_lugasun *m, const skn_step &st, const int32_t *ids
         }
         SKN_CUDA(ctx, st.T == 1 ? skn_launch_mix_decode(ctx, st, &aa, &rr, s) : skn_launch_mix_prefill(ctx, st, &aa, &rr, s));
         // output projection into the residual stream (the side gate takes x as bf16 rows on the tensor-core route)
-        const bool side = sp.side_dim > 0, raw = side && !rows32;
+        const bool side = sp.side_dim > 0, side_once = side && M <= SIDE_ROWS && skn_token_side_fits(l.w.side_gate, l.w.side_proj);
+        const bool raw = side && !rows32 && !side_once;
         skn_epi eo = to_rows(SKN_EPI_ADD, m->x, ldw, raw && !l.spec.ff ? m->x16 : nullptr, ldw);
         eo.resid = m->x; eo.ld_resid = ldw;
         SKN_CUDA(ctx, linear(m, few, l.w.w_out, M, m->mix32, m->ldm, m->mix16, m->ldm, nullptr, eo));
@@ -301,9 +309,9 @@ static int32_t run_layers(skn_lugasun *m, const skn_step &st, const int32_t *ids
         h_ready = false;
         if (side) {
             const int64_t col = (int64_t)m->runs[run] * sp.side_dim;
-            cudaError_t e = cudaErrorNotSupported;
-            if (few) e = skn_launch_token_side(l.w.side_gate, l.w.side_proj, m->side_embed, col, ids, m->x, ldw, M, l.side_norm, sp.eps, s);
-            if (e == cudaErrorNotSupported) {
+            if (side_once) {
+                SKN_CUDA(ctx, skn_launch_token_side(l.w.side_gate, l.w.side_proj, m->side_embed, col, ids, m->x, ldw, M, l.side_norm, sp.eps, s));
+            } else {
                 skn_epi eg = to_rows(SKN_EPI_GELU_TABLE, rows32 ? m->g32 : nullptr, m->lds, rows32 ? nullptr : m->g16, m->lds);
                 eg.table = reinterpret_cast<const __nv_bfloat16 *>(m->side_embed->d_blocks);
                 eg.ld_table = m->side_embed->pitch / 2; eg.table_rows = m->side_embed->n_rows; eg.table_col = col; eg.ids = ids;
@@ -311,10 +319,9 @@ static int32_t run_layers(skn_lugasun *m, const skn_step &st, const int32_t *ids
                 SKN_CUDA(ctx, linear(m, few, l.w.side_proj, M, m->g32, m->lds, m->g16, m->lds, nullptr, to_rows(SKN_EPI_STORE, m->y32, ldw, nullptr, 0)));
                 // y joins the residual stream in the pass that takes the next run's first norm
                 h_ready = !few && run + 1 < m->runs.size() && !m->pass_start[run + 1];
-                e = skn_launch_norm_rows(m->x, ldw, M, W, sp.eps, m->y32, ldw, l.side_norm, h_ready ? m->layers[m->runs[run + 1]].norm1 : nullptr, hout,
-                                         nullptr, 0, nullptr, s);
+                SKN_CUDA(ctx, skn_launch_norm_rows(m->x, ldw, M, W, sp.eps, m->y32, ldw, l.side_norm, h_ready ? m->layers[m->runs[run + 1]].norm1 : nullptr,
+                                                   hout, nullptr, 0, nullptr, s));
             }
-            SKN_CUDA(ctx, e);
         }
         if (m->tracing) {
             const size_t at = m->trace.size();
@@ -329,7 +336,7 @@ static int32_t run_layers(skn_lugasun *m, const skn_step &st, const int32_t *ids
 // logits of n rows of the residual stream (rows: device list, NULL for the first n) into m->logits
 static int32_t run_head(skn_lugasun *m, int n, const int32_t *rows) {
     skn_ctx *ctx = m->ctx;
-    const bool few = n <= SKN_MATVEC_ROWS && m->matvec_ok, rows32 = few || m->dtype == SKN_LUGASUN_F32;
+    const bool few = is_few(m, n), rows32 = few || m->dtype == SKN_LUGASUN_F32;
     const skn_rows_out hout = rows32 ? skn_rows_out{m->h32, m->ldw, nullptr, 0} : skn_rows_out{nullptr, 0, m->h16, m->ldw};
     const bool fold = few && !rows;
     if (!fold)

@@ -69,10 +69,78 @@ skn_norm_rows_kernel(float *x, int64_t ldx, int D, float eps, const float *add, 
     }
 }
 
+// The same for widths that are multiples of four: the row stays in registers, NV vectors per thread.
+template <int NV>
+__global__ void __launch_bounds__(256)
+skn_norm_rows_vec_kernel(float *x, int64_t ldx, int D, float eps, const float *add, int64_t ld_add, const float *__restrict__ add_gain,
+                         const float *__restrict__ gain, skn_rows_out out, __nv_bfloat16 *raw16, int64_t ld_raw16, const int32_t *rows) {
+    __shared__ float red[8];
+    skn_pdl_launch_dependents();
+    skn_pdl_wait();
+    const int64_t m = blockIdx.x, src = rows ? rows[m] : m;
+    float *xr = x + src * ldx;
+    float4 v[NV];
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+        const int i = (u * 256 + threadIdx.x) * 4;
+        v[u] = i < D ? *reinterpret_cast<const float4 *>(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (add) {
+        float4 a[NV];
+        float ss = 0.f;
+#pragma unroll
+        for (int u = 0; u < NV; ++u) {
+            const int i = (u * 256 + threadIdx.x) * 4;
+            a[u] = i < D ? *reinterpret_cast<const float4 *>(add + m * ld_add + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss += a[u].x * a[u].x + a[u].y * a[u].y + a[u].z * a[u].z + a[u].w * a[u].w;
+        }
+        const float r = 1.f / sqrtf(row_block_sum(ss, red) / (float)D + eps);
+#pragma unroll
+        for (int u = 0; u < NV; ++u) {
+            const int i = (u * 256 + threadIdx.x) * 4;
+            if (i < D) {
+                const float4 g = __ldg(reinterpret_cast<const float4 *>(add_gain + i));
+                v[u].x += a[u].x * r * g.x; v[u].y += a[u].y * r * g.y; v[u].z += a[u].z * r * g.z; v[u].w += a[u].w * r * g.w;
+                *reinterpret_cast<float4 *>(xr + i) = v[u];
+            }
+        }
+    }
+    auto put16 = [&](__nv_bfloat16 *p, float4 f) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(f.x, f.y), b = __floats2bfloat162_rn(f.z, f.w);
+        uint2 w;
+        w.x = *reinterpret_cast<const uint32_t *>(&a);
+        w.y = *reinterpret_cast<const uint32_t *>(&b);
+        *reinterpret_cast<uint2 *>(p) = w;
+    };
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+        const int i = (u * 256 + threadIdx.x) * 4;
+        if (raw16 && i < D) put16(raw16 + m * ld_raw16 + i, v[u]);
+        ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+    }
+    if (!gain) return;
+    const float r = 1.f / sqrtf(row_block_sum(ss, red) / (float)D + eps);
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+        const int i = (u * 256 + threadIdx.x) * 4;
+        if (i >= D) continue;
+        const float4 g = __ldg(reinterpret_cast<const float4 *>(gain + i));
+        const float4 f = make_float4(v[u].x * r * g.x, v[u].y * r * g.y, v[u].z * r * g.z, v[u].w * r * g.w);
+        if (out.y32) *reinterpret_cast<float4 *>(out.y32 + m * out.ld32 + i) = f;
+        if (out.y16) put16(out.y16 + m * out.ld16 + i, f);
+    }
+}
+
 cudaError_t skn_launch_norm_rows(float *x, int64_t ldx, int M, int D, float eps, const float *add, int64_t ld_add,
                                  const float *add_gain, const float *gain, const skn_rows_out &out, __nv_bfloat16 *raw16,
                                  int64_t ld_raw16, const int32_t *rows, cudaStream_t st) {
     if (M == 0) return cudaSuccess;
+    if (D % 4 == 0 && D <= 8192 && ldx % 4 == 0 && ld_add % 4 == 0 && out.ld32 % 4 == 0 && out.ld16 % 4 == 0 && ld_raw16 % 4 == 0) {
+#define NORM_CASE(NV) skn_launch_pdl(skn_norm_rows_vec_kernel<NV>, dim3(M), dim3(256), 0, st, 1, x, ldx, D, eps, add, ld_add, add_gain, gain, out, raw16, ld_raw16, rows)
+        return D <= 1024 ? NORM_CASE(1) : D <= 2048 ? NORM_CASE(2) : D <= 4096 ? NORM_CASE(4) : NORM_CASE(8);
+#undef NORM_CASE
+    }
     return skn_launch_pdl(skn_norm_rows_kernel, dim3(M), dim3(256), 0, st, 1, x, ldx, D, eps, add, ld_add, add_gain, gain, out, raw16, ld_raw16, rows);
 }
 
@@ -99,20 +167,27 @@ cudaError_t skn_launch_rows_to_bf16(const float *in, int64_t ld, int M, int D, _
 // ---- token side input, a few rows -------------------------------------------------------------------------------
 // The cluster of 8 CTAs owns one row: CTA r computes the gate rows r, r + 8, ... and shares them through distributed
 // shared memory, then its eighth of the projection's rows; the sum of squares meets the same way.
-constexpr int SIDE_CLUSTER = 8, SIDE_THREADS = 256;
+constexpr int SIDE_CLUSTER = 8, SIDE_THREADS = 512;
+
+__device__ __forceinline__ void prefetch_l2(const void *p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 __global__ void __launch_bounds__(SIDE_THREADS)
 skn_token_side_kernel(const uint8_t *__restrict__ wg, int64_t pitch_g, const uint8_t *__restrict__ wp, int64_t pitch_p,
                       const uint8_t *__restrict__ table, int64_t pitch_t, int64_t table_rows, int64_t col, const int32_t *ids, float *x,
                       int64_t ldx, int D, int S, const float *__restrict__ gain, float eps) {
     extern __shared__ float sm[];                      // x row (padded to 8), then g [S padded to 8], then y [rows of this CTA]
-    __shared__ float red[8], part[SIDE_CLUSTER];
+    __shared__ float red[SIDE_THREADS / 32], part[SIDE_CLUSTER];
     cg::cluster_group cl = cg::this_cluster();
     const int rank = (int)cl.block_rank(), m = blockIdx.x / SIDE_CLUSTER;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int D8 = (int)(pitch_g / 2), S8 = (int)(pitch_p / 2);
     float *xs = sm, *gs = sm + D8, *ys = gs + S8;
     skn_pdl_launch_dependents();
+    // this CTA's weights are on their way into L2 while the kernel before still runs
+    const int per = (D + SIDE_CLUSTER - 1) / SIDE_CLUSTER, n0 = rank * per, n1 = min(D, n0 + per);
+    for (int j = rank + SIDE_CLUSTER * warp; j < S; j += SIDE_CLUSTER * (SIDE_THREADS / 32))
+        for (int64_t i = (int64_t)lane * 128; i < pitch_g; i += 32 * 128) prefetch_l2(wg + (int64_t)j * pitch_g + i);
+    for (int64_t i = n0 * pitch_p + (int64_t)threadIdx.x * 128; i < n1 * pitch_p; i += SIDE_THREADS * 128) prefetch_l2(wp + i);
     skn_pdl_wait();
     float *xr = x + (int64_t)m * ldx;
     for (int i = threadIdx.x; i < D8; i += SIDE_THREADS) xs[i] = i < D ? __ldcg(xr + i) : 0.f;
@@ -125,7 +200,7 @@ skn_token_side_kernel(const uint8_t *__restrict__ wg, int64_t pitch_g, const uin
     for (int j = rank + SIDE_CLUSTER * warp; j < S; j += SIDE_CLUSTER * (SIDE_THREADS / 32)) {
         const uint4 *wr = reinterpret_cast<const uint4 *>(wg + (int64_t)j * pitch_g);
         float a = 0.f;
-#pragma unroll 4
+#pragma unroll 8
         for (int i = lane; i < D8 / 8; i += 32) {
             const uint4 w = __ldg(wr + i);
             const float4 lo = *reinterpret_cast<const float4 *>(xs + i * 8), hi = *reinterpret_cast<const float4 *>(xs + i * 8 + 4);
@@ -138,12 +213,11 @@ skn_token_side_kernel(const uint8_t *__restrict__ wg, int64_t pitch_g, const uin
         if (lane < SIDE_CLUSTER) *cl.map_shared_rank(gs + j, lane) = a;
     }
     cl.sync();
-    const int per = (D + SIDE_CLUSTER - 1) / SIDE_CLUSTER, n0 = rank * per, n1 = min(D, n0 + per);
     float ss = 0.f;
     for (int n = n0 + threadIdx.x; n < n1; n += SIDE_THREADS) {
         const uint4 *wr = reinterpret_cast<const uint4 *>(wp + (int64_t)n * pitch_p);
         float a = 0.f;
-#pragma unroll 4
+#pragma unroll 8
         for (int i = 0; i < S8 / 8; ++i) {
             const uint4 w = __ldg(wr + i);
             const float4 lo = *reinterpret_cast<const float4 *>(gs + i * 8), hi = *reinterpret_cast<const float4 *>(gs + i * 8 + 4);
@@ -163,12 +237,17 @@ skn_token_side_kernel(const uint8_t *__restrict__ wg, int64_t pitch_g, const uin
     for (int n = n0 + threadIdx.x; n < n1; n += SIDE_THREADS) xr[n] = xs[n] + ys[n - n0] * r * gain[n];
 }
 
+static size_t side_smem(const skn_tensor *wg, const skn_tensor *wp) {
+    return ((size_t)wg->pitch / 2 + wp->pitch / 2 + (wg->n_cols + SIDE_CLUSTER - 1) / SIDE_CLUSTER) * sizeof(float);
+}
+bool skn_token_side_fits(const skn_tensor *wg, const skn_tensor *wp) { return side_smem(wg, wp) <= 200 * 1024; }
+
 cudaError_t skn_launch_token_side(const skn_tensor *wg, const skn_tensor *wp, const skn_tensor *table, int64_t col, const int32_t *ids,
                                   float *x, int64_t ldx, int M, const float *gain, float eps, cudaStream_t st) {
     if (M == 0) return cudaSuccess;
     const int D = (int)wg->n_cols, S = (int)wg->n_rows;
-    const size_t smem = ((size_t)wg->pitch / 2 + wp->pitch / 2 + (D + SIDE_CLUSTER - 1) / SIDE_CLUSTER) * sizeof(float);
-    if (smem > 200 * 1024) return cudaErrorNotSupported;
+    if (!skn_token_side_fits(wg, wp)) return cudaErrorNotSupported;
+    const size_t smem = side_smem(wg, wp);
     const cudaError_t e = cudaFuncSetAttribute(skn_token_side_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return e;
     return skn_launch_pdl(skn_token_side_kernel, dim3(M * SIDE_CLUSTER), dim3(SIDE_THREADS), smem, st, SIDE_CLUSTER, (const uint8_t *)wg->d_blocks,

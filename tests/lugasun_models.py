@@ -48,12 +48,16 @@ def getter(bits):
     return get
 
 
-def error(got, want):
-    """Worst row: root mean square difference of mean-free logits over the root mean square of the wanted ones."""
+def errors(got, want):
+    """Per row: root mean square difference of mean-free logits over the root mean square of the wanted ones."""
     d = np.asarray(got, np.float64) - want
     d -= d.mean(-1, keepdims=True)
     w = want - want.mean(-1, keepdims=True)
-    return float((np.sqrt((d * d).mean(-1)) / np.sqrt((w * w).mean())).max())
+    return np.sqrt((d * d).mean(-1)) / np.sqrt((w * w).mean())
+
+
+def error(got, want):
+    return float(errors(got, want).max())
 
 
 TOL = {"float32": 3e-5, "bfloat16": 4e-2}
