@@ -440,7 +440,7 @@ typedef struct skn_retention_spec {
     double rot_base;
     const double *decay;
     float eps;
-    int32_t reserved;
+    int32_t exact;       /* many-token steps: 1 = fp32 products only, 0 = tensor cores with two-term tf32 operands */
 } skn_retention_spec;
 
 /* recurrent state of `slots` sequences, fp32 [heads][k_dim][v_dim] each; a sequence at position 0 starts from zero */

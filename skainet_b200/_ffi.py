@@ -26,7 +26,7 @@ class AttnSpec(ctypes.Structure):
 
 class RetentionSpec(ctypes.Structure):
     _fields_ = [("heads", c_i32), ("dim", c_i32), ("vdim", c_i32), ("rot_dims", c_i32), ("rot_base", ctypes.c_double),
-                ("decay", P(ctypes.c_double)), ("eps", ctypes.c_float), ("reserved", c_i32)]
+                ("decay", P(ctypes.c_double)), ("eps", ctypes.c_float), ("exact", c_i32)]
 
 
 class LugasunLayer(ctypes.Structure):

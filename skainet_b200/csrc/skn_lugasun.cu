@@ -280,6 +280,7 @@ static int32_t run_layers(skn_lugasun *m, const skn_step &st, const int32_t *ids
         rr.q = m->proj + (int64_t)a.heads * a.dim + (int64_t)a.kv_heads * (a.dim + a.vdim);
         rr.k = rr.q + (int64_t)r.heads * r.dim; rr.v = rr.k + (int64_t)r.heads * r.dim; rr.g = rr.v + (int64_t)r.heads * r.vdim; rr.ld = m->ldp;
         rr.out_scale = l.spec.right_scale;
+        rr.exact = f32;
         rr.chunks = m->ret_chunks;
         const int64_t rc0 = (int64_t)a.heads * a.vdim;
         if (rows32) {

@@ -8,8 +8,8 @@
 //  skn_attn_tc_kernel      64 queries of one head: scores and products on the tensor cores (bf16 operands, fp32 sums);
 //                          the weights enter the second product as two bf16 terms, so they keep 16 bits
 //  skn_attn_rows_kernel    the split kernel on prepared keys (fp32 cache, or head widths beyond the tensor-core form)
-//  skn_ret_*_kernel        retention in chunks of 64 tokens, all fp32: what each chunk adds to the state, the states
-//                          at the chunk starts, and the outputs
+//  skn_ret_*_kernel        retention in chunks of 64 tokens: what each chunk adds to the state, the states at the chunk
+//                          starts, and the outputs; on the CUDA cores (fp32 decoder) or the tensor cores (two-term tf32)
 #include "skn_mixers.cuh"
 #include "skn_ptx.cuh"
 
@@ -433,7 +433,8 @@ skn_head_prep_kernel(skn_attn_args a, skn_ret_args r, skn_step st, prep_args p, 
 }
 
 // ---- attention on the tensor cores ---------------------------------------------------------------------------------
-constexpr int ATQ = 64, ATK = 64;      // queries and keys of a tile
+constexpr int ATQ = 64, ATK = 32;      // queries and keys of a tile
+constexpr int AT_THREADS = ATQ * 2;    // a warp owns 16 queries
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
@@ -461,7 +462,7 @@ __device__ __forceinline__ float tanh_exp(float y) {
 }
 
 template <int DV>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(AT_THREADS, DV <= 128 ? 3 : 1)
 skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict__ kc_, const __nv_bfloat16 *__restrict__ vc_, int G, int cap, int vdim,
                    int kp, int vp) {
     extern __shared__ __align__(16) uint8_t smb[];
@@ -478,27 +479,26 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
     const size_t head_rows = ((size_t)slot * G + g) * cap;
     const __nv_bfloat16 *kc = kc_ + head_rows * kp, *vc = vc_ + head_rows * vp;
 
+    const int slot0 = lo % cap;
+    const bool idle = warp * 16 >= nq;                                   // none of this warp's queries exist
+    // four threads per key row (two per query row), every fourth 16-byte piece each
+    const int cr = tid >> 2, cc = tid & 3;
     auto load_tile = [&](int t, int buf) {
-        const int j0 = lo + t * ATK;
-        const int kch = kp / 8, vch = DV / 8;
-        for (int i = tid; i < ATK * kch; i += 128) {
-            const int r = i / kch, c = i % kch, j = j0 + r;
-            cp_async16(skn_smem_u32(K + ((size_t)buf * ATK + r) * ks + c * 8), kc + (size_t)((j <= pl ? j : pl) % cap) * kp + c * 8, j <= pl);
-        }
-        for (int i = tid; i < ATK * vch; i += 128) {
-            const int r = i / vch, c = i % vch, j = j0 + r;
-            const bool in = j <= pl && c * 8 < vp;
-            cp_async16(skn_smem_u32(V + ((size_t)buf * ATK + r) * vs + c * 8), vc + (size_t)((j <= pl ? j : pl) % cap) * vp + (c * 8 < vp ? c * 8 : 0), in);
-        }
+        const int j = lo + t * ATK + cr;
+        const bool in = j <= pl;
+        int sl = slot0 + t * ATK + cr;
+        if (sl >= cap) sl %= cap;
+        const __nv_bfloat16 *kr = kc + (size_t)sl * kp, *vr = vc + (size_t)sl * vp;
+        const uint32_t kd = skn_smem_u32(K + ((size_t)buf * ATK + cr) * ks), vd = skn_smem_u32(V + ((size_t)buf * ATK + cr) * vs);
+        for (int c = cc * 8; c < kp; c += 32) cp_async16(kd + c * 2, kr + c, in);
+#pragma unroll
+        for (int c = cc * 8; c < DV; c += 32) cp_async16(vd + c * 2, vr + (c < vp ? c : 0), in && c < vp);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     {
-        const int kch = kp / 8;
-        const __nv_bfloat16 *q = a.q16 + (((int64_t)seq * st.T + t0) * a.heads + h) * kp;
-        for (int i = tid; i < ATQ * kch; i += 128) {
-            const int r = i / kch, c = i % kch;
-            cp_async16(skn_smem_u32(Q + (size_t)r * ks + c * 8), q + (int64_t)(r < nq ? r : 0) * a.heads * kp + c * 8, r < nq);
-        }
+        const int r = tid >> 1;
+        const __nv_bfloat16 *q = a.q16 + (((int64_t)seq * st.T + t0 + (r < nq ? r : 0)) * a.heads + h) * kp;
+        for (int c = (tid & 1) * 8; c < kp; c += 16) cp_async16(skn_smem_u32(Q + (size_t)r * ks + c), q + c, r < nq);
     }
     load_tile(0, 0);
 
@@ -511,6 +511,7 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
     int qlo[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) qlo[i] = a.chunk > 0 ? qi[i] / a.chunk * a.chunk : 0;
+    const int w0 = pf + warp * 16, wlo = a.chunk > 0 ? w0 / a.chunk * a.chunk : 0, whi = a.chunk > 0 ? (w0 + 15) / a.chunk * a.chunk : 0;
     const float L2E = 1.4426950408889634f;
     const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
 
@@ -519,30 +520,36 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         if (t + 1 < tiles) load_tile(t + 1, buf ^ 1);
-        float s[8][4];
+        const int j0 = lo + t * ATK;
+        // tiles that none of the warp's queries sees: past its last query, or in an earlier chunk than its first
+        if (idle || j0 > w0 + 15 || j0 + ATK <= wlo) {
+            __syncthreads();
+            continue;
+        }
+        const bool masked = j0 + ATK - 1 > w0 || j0 < whi;               // some pair of this tile is invisible
+        float s[ATK / 8][4];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+        for (int i = 0; i < ATK / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
         const __nv_bfloat16 *Kb = K + (size_t)buf * ATK * ks, *Vb = V + (size_t)buf * ATK * vs;
         for (int kk = 0; kk < kp; kk += 16) {
             uint32_t af[4];
             ldsm4(af, skn_smem_u32(Q + (size_t)(warp * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8));
 #pragma unroll
-            for (int n = 0; n < 4; ++n) {
+            for (int n = 0; n < ATK / 16; ++n) {
                 uint32_t bf[4];
                 ldsm4(bf, skn_smem_u32(Kb + (size_t)(n * 16 + (lane & 7) + ((lane >> 4) << 3)) * ks + kk + ((lane >> 3) & 1) * 8));
                 mma_bf16(s[2 * n], af, bf[0], bf[1]);
                 mma_bf16(s[2 * n + 1], af, bf[2], bf[3]);
             }
         }
-        const int j0 = lo + t * ATK;
         float mx[2] = {mrow[0], mrow[1]};
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < ATK / 8; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int i = e >> 1, j = j0 + n * 8 + (lane & 3) * 2 + (e & 1);
                 float v = a.softcap > 0.f ? a.softcap * tanh_exp(s[n][e] * inv_cap) : s[n][e] * a.scale;
-                v = (j <= qi[i] && j >= qlo[i]) ? v * L2E : -INFINITY;
+                v = !masked || (j <= qi[i] && j >= qlo[i]) ? v * L2E : -INFINITY;
                 s[n][e] = v;
                 mx[i] = fmaxf(mx[i], v);
             }
@@ -557,7 +564,7 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
             lrow[i] *= corr[i];
         }
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < ATK / 8; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 s[n][e] = exp2f(s[n][e] - base[e >> 1]);
@@ -569,7 +576,7 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
             o[i][2] *= corr[1]; o[i][3] *= corr[1];
         }
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
+        for (int kk = 0; kk < ATK / 16; ++kk) {
             uint32_t hi[4], lw[4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
@@ -618,7 +625,7 @@ static cudaError_t launch_attn_tc(const skn_step &s, const skn_attn_args &a, cud
     const size_t smem = ((size_t)(ATQ + 2 * ATK) * (kp + 8) + (size_t)2 * ATK * (DV + 8)) * 2;
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return e;
-    return skn_launch_pdl(kern, dim3((s.T + ATQ - 1) / ATQ, a.heads, s.n_seqs), dim3(128), smem, st, 1, a, s, (const __nv_bfloat16 *)a.kv->d_k,
+    return skn_launch_pdl(kern, dim3((s.T + ATQ - 1) / ATQ, a.heads, s.n_seqs), dim3(AT_THREADS), smem, st, 1, a, s, (const __nv_bfloat16 *)a.kv->d_k,
                           (const __nv_bfloat16 *)a.kv->d_v, a.kv->n_kv_heads, a.kv->capacity, a.kv->v_dim, kp, a.kv->v_pitch);
 }
 
@@ -674,13 +681,13 @@ skn_ret_scan_kernel(skn_ret_args r, skn_step st, float *S, int H, int dk, int vp
     float4 *sp = reinterpret_cast<float4 *>(S) + (size_t)slot * per + i;
     float4 s = st.pos[slot] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
     const float full = pw[RC], tail = pw[T - (nchunks - 1) * RC];
-    for (int c0 = 0; c0 < nchunks; c0 += 4) {
-        float4 a[4];
+    for (int c0 = 0; c0 < nchunks; c0 += 8) {
+        float4 a[8];
 #pragma unroll
-        for (int u = 0; u < 4; ++u)
+        for (int u = 0; u < 8; ++u)
             if (c0 + u < nchunks) a[u] = __ldcg(p + (size_t)(c0 + u) * per);
 #pragma unroll
-        for (int u = 0; u < 4; ++u)
+        for (int u = 0; u < 8; ++u)
             if (c0 + u < nchunks) {
                 __stcg(p + (size_t)(c0 + u) * per, s);
                 const float d = c0 + u == nchunks - 1 ? tail : full;
@@ -688,6 +695,20 @@ skn_ret_scan_kernel(skn_ret_args r, skn_step st, float *S, int H, int dk, int vp
             }
     }
     *sp = s;
+}
+
+// rows of O (shared): divided by their root mean square, gated, scaled, stored
+__device__ __forceinline__ void ret_finish(const skn_ret_args &r, const float *O, int os, int64_t row0, int L, int h, int dv) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int t = warp; t < L; t += 8) {
+        float ss = 0.f;
+        for (int d = lane; d < dv; d += 32) ss = fmaf(O[t * os + d], O[t * os + d], ss);
+        const float rs = r.out_scale / sqrtf(warp_sum(ss) / (float)dv + r.eps);
+        for (int d = lane; d < dv; d += 32) {
+            const float g = __ldcg(r.g + (row0 + t) * r.ld + (int64_t)h * dv + d);
+            put_out(r.out, row0 + t, (int64_t)h * dv + d, O[t * os + d] * rs * (g / (1.f + expf(-g))));
+        }
+    }
 }
 
 // outputs of one chunk: o_i = sum_{j <= i} decay^(i - j) (q_i . k_j) v_j + decay^(i + 1) S^T q_i, then normalised and gated.
@@ -781,16 +802,173 @@ skn_ret_out_kernel(skn_ret_args r, int T, int H, int dk, int dv, int vp, int nch
             for (int y = 0; y < 4; ++y) O[(ti + x) * os + v0 + tj + y] = fmaf(pw[ti + x + 1], p[x][y], o[x][y]);
     }
     __syncthreads();
-    const int warp = tid >> 5, lane = tid & 31;
-    for (int t = warp; t < L; t += 8) {
-        float ss = 0.f;
-        for (int d = lane; d < dv; d += 32) ss = fmaf(O[t * os + d], O[t * os + d], ss);
-        const float rs = r.out_scale / sqrtf(warp_sum(ss) / (float)dv + r.eps);
-        for (int d = lane; d < dv; d += 32) {
-            const float g = __ldcg(r.g + (row0 + t) * r.ld + (int64_t)h * dv + d);
-            put_out(r.out, row0 + t, (int64_t)h * dv + d, O[t * os + d] * rs * (g / (1.f + expf(-g))));
+    ret_finish(r, O, os, row0, L, h, dv);
+}
+
+// ---- retention chunks on the tensor cores -----------------------------------------------------------------------------
+// Every fp32 operand enters as the sum of two tf32 terms and three products are formed (the lowest is below fp32
+// rounding), summed in fp32: the results carry fp32 accuracy.  Fragments are read from fp32 rows in shared memory; row
+// strides are 4 (rows along M or N) or 8 (rows along K) banks off a multiple of 32, which keeps the reads conflict-free.
+__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+struct TwoTerm { uint32_t hi, lo; };
+__device__ __forceinline__ TwoTerm two_term(float x) {
+    TwoTerm t;
+    t.hi = __float_as_uint(x) & 0xFFFFE000u;
+    t.lo = __float_as_uint(x - __uint_as_float(t.hi)) & 0xFFFFE000u;
+    return t;
+}
+// c[n] += A (16 x 8 at rows m, column step k) times B (8 x 8 NT): at(row, k) and bt(k, col) read shared memory
+template <int NT, class AT, class BT>
+__device__ __forceinline__ void mma_two_term(float (&c)[NT][4], int k, AT at, BT bt) {
+    const int g = (threadIdx.x & 31) >> 2, t = threadIdx.x & 3;
+    uint32_t ah[4], al[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const TwoTerm x = two_term(at(g + (i & 1) * 8, k + t + (i >> 1) * 4));
+        ah[i] = x.hi;
+        al[i] = x.lo;
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+        const TwoTerm b0 = two_term(bt(k + t, n * 8 + g)), b1 = two_term(bt(k + t + 4, n * 8 + g));
+        mma_tf32(c[n], al, b0.hi, b1.hi);
+        mma_tf32(c[n], ah, b0.lo, b1.lo);
+        mma_tf32(c[n], ah, b0.hi, b1.hi);
+    }
+}
+
+constexpr int RT2 = 128;              // columns of a tile
+constexpr int RKS = RT2 + 8;          // row stride of operands whose rows run along K
+
+// the chunk sums of skn_ret_chunk_kernel, in 128 x 128 tiles; a warp owns 16 rows
+__global__ void __launch_bounds__(256)
+skn_ret_chunk_tc_kernel(skn_ret_args r, int T, int H, int dk, int dv, int vp, int nchunks, int vtiles) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float pw[RC + 1];
+    float *Ks = sm, *Vs = sm + RC * RKS;
+    skn_pdl_launch_dependents();
+    skn_pdl_wait();
+    const int c = blockIdx.x, h = blockIdx.y % H, seq = blockIdx.y / H, i0 = (blockIdx.z / vtiles) * RT2, j0 = (blockIdx.z % vtiles) * RT2;
+    const int t0 = c * RC, L = min(RC, T - t0), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int64_t row0 = (int64_t)seq * T + t0;
+    const float *k = r.k + row0 * r.ld + (int64_t)h * dk + i0, *v = r.v + row0 * r.ld + (int64_t)h * dv + j0;
+    if (tid <= RC) pw[tid] = r.powers[(size_t)h * (RC + 1) + tid];
+    __syncthreads();
+#pragma unroll 8
+    for (int i = tid; i < RC * RT2; i += 256) {
+        const int t = i / RT2, d = i % RT2;
+        Ks[t * RKS + d] = t < L && i0 + d < dk ? __ldcg(k + (int64_t)t * r.ld + d) * pw[L - 1 - t] : 0.f;
+        Vs[t * RKS + d] = t < L && j0 + d < dv ? __ldcg(v + (int64_t)t * r.ld + d) : 0.f;
+    }
+    __syncthreads();
+    float acc[RT2 / 8][4] = {};
+    if (i0 + warp * 16 < dk)
+        for (int kk = 0; kk < RC; kk += 8)
+            mma_two_term(acc, kk, [&](int m, int x) { return Ks[x * RKS + warp * 16 + m]; }, [&](int x, int n) { return Vs[x * RKS + n]; });
+    float *out = r.chunks + ((((size_t)seq * nchunks + c) * H + h) * dk) * vp;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int row = i0 + warp * 16 + (lane >> 2) + e * 8;
+        if (row >= dk) continue;
+#pragma unroll
+        for (int n = 0; n < RT2 / 8; ++n) {
+            const int col = j0 + n * 8 + (lane & 3) * 2;
+            if (col < vp) *reinterpret_cast<float2 *>(out + (size_t)row * vp + col) = make_float2(acc[n][2 * e], acc[n][2 * e + 1]);
         }
     }
+}
+
+// the chunk outputs of skn_ret_out_kernel; warp w owns tokens 16 (w & 3) .. and one half of the columns
+// smem (floats): q [RC][dkp + 4] | A [RC][RC + 4] | max(k [RC][dkp + 4], b [32][RKS] and o [RC][vw + 4])
+static size_t ret_out_tc_smem(int dk, int dv) {
+    const size_t qk = (size_t)RC * ((dk + 31) / 32 * 32 + 4), bo = 32 * RKS + (size_t)RC * ((dv + RT2 - 1) / RT2 * RT2 + 4);
+    return (qk + RC * (RC + 4) + (qk > bo ? qk : bo)) * sizeof(float);
+}
+
+__global__ void __launch_bounds__(256, 2)
+skn_ret_out_tc_kernel(skn_ret_args r, int T, int H, int dk, int dv, int vp, int nchunks) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float pw[RC + 1];
+    const int dkp = (dk + 31) / 32 * 32, qs = dkp + 4, vw = (dv + RT2 - 1) / RT2 * RT2, os = vw + 4;
+    constexpr int AS = RC + 4;
+    float *Q = sm, *A = Q + RC * qs, *Kb = A + RC * AS, *B = Kb, *O = Kb + 32 * RKS;
+    skn_pdl_launch_dependents();
+    skn_pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, t0 = c * RC, L = min(RC, T - t0);
+    const int64_t row0 = (int64_t)seq * T + t0;
+    const float *q = r.q + row0 * r.ld + (int64_t)h * dk, *k = r.k + row0 * r.ld + (int64_t)h * dk, *v = r.v + row0 * r.ld + (int64_t)h * dv;
+    if (tid <= RC) pw[tid] = r.powers[(size_t)h * (RC + 1) + tid];
+    for (int d0 = 0; d0 < dkp; d0 += 32)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int t = warp + i * 8, d = d0 + lane;
+            const bool in = t < L && d < dk;
+            Q[t * qs + d] = in ? __ldcg(q + (int64_t)t * r.ld + d) : 0.f;
+            Kb[t * qs + d] = in ? __ldcg(k + (int64_t)t * r.ld + d) : 0.f;
+        }
+    __syncthreads();
+    const int m0 = (warp & 3) * 16, half = warp >> 2, g = lane >> 2, t = lane & 3;
+    {
+        float acc[RC / 16][4] = {};
+        const int n0 = half * (RC / 2);
+        if (n0 <= m0 + 15)                         // else every pair of this tile lies in the future
+            for (int kk = 0; kk < dkp; kk += 8)
+                mma_two_term(acc, kk, [&](int m, int x) { return Q[(m0 + m) * qs + x]; }, [&](int x, int n) { return Kb[(n0 + n) * qs + x]; });
+#pragma unroll
+        for (int n = 0; n < RC / 16; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = m0 + g + (e >> 1) * 8, j = n0 + n * 8 + t * 2 + (e & 1);
+                A[i * AS + j] = j <= i ? acc[n][e] * pw[i - j] : 0.f;
+            }
+    }
+    const float *S = r.chunks + ((((size_t)seq * nchunks + c) * H + h) * dk) * vp;
+    constexpr int NT = RT2 / 16;
+    for (int v0 = 0; v0 < vw; v0 += RT2) {
+        float o[NT][4] = {};
+        const int c0 = half * (RT2 / 2);
+        // tiles of 32 rows: the state's first, then the chunk's values
+        const int stiles = dkp / 32, tiles = stiles + (L + 31) / 32;
+        float pre[16];
+        auto fetch = [&](int x) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                const int row = (x < stiles ? x : x - stiles) * 32 + (tid >> 7) + i * 2, col = v0 + (tid & 127);
+                if (x < stiles) pre[i] = row < dk && col < vp ? __ldcg(S + (size_t)row * vp + col) : 0.f;
+                else pre[i] = row < L && col < dv ? __ldcg(v + (int64_t)row * r.ld + col) : 0.f;
+            }
+        };
+        fetch(0);
+        for (int x = 0; x < tiles; ++x) {
+            __syncthreads();                       // the tile before (or k) is done with
+#pragma unroll
+            for (int i = 0; i < 16; ++i) B[((tid >> 7) + i * 2) * RKS + (tid & 127)] = pre[i];
+            __syncthreads();
+            if (x + 1 < tiles) fetch(x + 1);
+            if (x == stiles)
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) o[n][e] *= pw[m0 + g + (e >> 1) * 8 + 1];
+            const float *a = x < stiles ? Q + x * 32 : A + (x - stiles) * 32;
+            const int lda = x < stiles ? qs : AS;
+            if (x < stiles || (x - stiles) * 32 <= m0 + 15)
+#pragma unroll
+                for (int kk = 0; kk < 32; kk += 8)
+                    mma_two_term(o, kk, [&](int m, int y) { return a[(m0 + m) * lda + y]; }, [&](int y, int n) { return B[y * RKS + c0 + n]; });
+        }
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+                *reinterpret_cast<float2 *>(O + (m0 + g + e * 8) * os + v0 + c0 + n * 8 + t * 2) = make_float2(o[n][2 * e], o[n][2 * e + 1]);
+    }
+    __syncthreads();
+    ret_finish(r, O, os, row0, L, h, dv);
 }
 
 template <class CT>
@@ -831,15 +1009,30 @@ cudaError_t skn_launch_mix_prefill(skn_ctx *, const skn_step &s, const skn_attn_
     }
     if (r) {
         const int H = r->state->heads, dk = r->state->k_dim, dv = r->state->v_dim, vp = r->state->v_pitch;
-        const int nchunks = (s.T + RC - 1) / RC, kt = (dk + 63) / 64, vt = (dv + 63) / 64;
-        e = skn_launch_pdl(skn_ret_chunk_kernel, dim3(nchunks, H * s.n_seqs, kt * vt), dim3(256), 0, st, 1, *r, s.T, H, dk, dv, vp, nchunks, vt);
+        const int nchunks = (s.T + RC - 1) / RC;
+        const bool tc = !r->exact && ret_out_tc_smem(dk, dv) <= 200 * 1024;
+        const int tile = tc ? RT2 : 64, kt = (dk + tile - 1) / tile, vt = (dv + tile - 1) / tile;
+        const dim3 cgrid(nchunks, H * s.n_seqs, kt * vt), ogrid(nchunks, H, s.n_seqs);
+        if (tc) {
+            e = cudaFuncSetAttribute(skn_ret_chunk_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * RC * RKS * 4);
+            if (e != cudaSuccess) return e;
+            e = skn_launch_pdl(skn_ret_chunk_tc_kernel, cgrid, dim3(256), (size_t)2 * RC * RKS * 4, st, 1, *r, s.T, H, dk, dv, vp, nchunks, vt);
+        } else {
+            e = skn_launch_pdl(skn_ret_chunk_kernel, cgrid, dim3(256), 0, st, 1, *r, s.T, H, dk, dv, vp, nchunks, vt);
+        }
         if (e != cudaSuccess) return e;
         const int64_t per = (int64_t)H * dk * (vp / 4);
         e = skn_launch_pdl(skn_ret_scan_kernel, dim3((unsigned)((per + 127) / 128), s.n_seqs), dim3(128), 0, st, 1, *r, s, r->state->d, H, dk, vp, nchunks);
         if (e != cudaSuccess) return e;
-        e = cudaFuncSetAttribute(skn_ret_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        if (e != cudaSuccess) return e;
-        e = skn_launch_pdl(skn_ret_out_kernel, dim3(nchunks, H, s.n_seqs), dim3(256), ret_out_smem(dv), st, 1, *r, s.T, H, dk, dv, vp, nchunks);
+        if (tc) {
+            e = cudaFuncSetAttribute(skn_ret_out_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+            if (e != cudaSuccess) return e;
+            e = skn_launch_pdl(skn_ret_out_tc_kernel, ogrid, dim3(256), ret_out_tc_smem(dk, dv), st, 1, *r, s.T, H, dk, dv, vp, nchunks);
+        } else {
+            e = cudaFuncSetAttribute(skn_ret_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+            if (e != cudaSuccess) return e;
+            e = skn_launch_pdl(skn_ret_out_kernel, ogrid, dim3(256), ret_out_smem(dv), st, 1, *r, s.T, H, dk, dv, vp, nchunks);
+        }
     }
     return e;
 }
@@ -1035,7 +1228,7 @@ int32_t skn_retention(skn_state *s, const skn_retention_spec *spec, int32_t seq0
     skn_ret_args x = {};
     x.state = s; x.eps = spec->eps; x.rot = skn_rot{rot, half, half}; x.k_scale = (float)(1.0 / sqrt((double)D)); x.powers = pw;
     x.q = rows; x.k = rows + w[0]; x.v = rows + 2 * w[0]; x.g = rows + 2 * w[0] + w[2]; x.ld = ld;
-    x.out_scale = 1.f; x.out = skn_rows_out{out, (int64_t)H * V, nullptr, 0}; x.chunks = chunks;
+    x.out_scale = 1.f; x.out = skn_rows_out{out, (int64_t)H * V, nullptr, 0}; x.exact = spec->exact != 0; x.chunks = chunks;
     SKN_CUDA(ctx, T == 1 ? skn_launch_mix_decode(ctx, st, nullptr, &x, ctx->stream) : skn_launch_mix_prefill(ctx, st, nullptr, &x, ctx->stream));
     SKN_CUDA(ctx, cudaMemcpyAsync(out_host, out, (size_t)M * H * V * 4, cudaMemcpyDeviceToHost, ctx->stream));
     return skn_sync(ctx);

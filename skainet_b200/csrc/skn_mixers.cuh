@@ -46,6 +46,7 @@ struct skn_ret_args {
     int64_t ld;
     float out_scale;
     skn_rows_out out;
+    bool exact;                     // fp32 products only (no tensor cores)
     float *chunks;                  // [n_seqs][ceil(T / SKN_RET_CHUNK)][heads][k_dim][v_pitch] floats
 };
 constexpr int SKN_RET_CHUNK = 64;

@@ -79,8 +79,9 @@ class RecurrentState:
         return self._h
 
     def retain(self, q, k, v, g, pos, decay, *, seq: int = 0, rot_dims: int = 0, rot_base: float = 10000.0, eps: float = 1e-5,
-               max_ctx: int = 1 << 20) -> np.ndarray:
-        """q, k [n, T, heads, dim], v, g [n, T, heads, vdim]; returns the normalised, gated outputs [n, T, heads, vdim]."""
+               max_ctx: int = 1 << 20, exact: bool = False) -> np.ndarray:
+        """q, k [n, T, heads, dim], v, g [n, T, heads, vdim]; returns the normalised, gated outputs [n, T, heads, vdim].
+        exact: fp32 products only."""
         n, T, H, D = np.shape(q)
         q, k = _rows(q, n, T, self.heads, self.dim), _rows(k, n, T, self.heads, self.dim)
         v, g = _rows(v, n, T, self.heads, self.vdim), _rows(g, n, T, self.heads, self.vdim)
@@ -88,7 +89,7 @@ class RecurrentState:
         if len(decay) != self.heads:
             raise ValueError("Shapes do not align.")
         d = (ctypes.c_double * self.heads)(*[float(x) for x in decay])
-        spec = _ffi.RetentionSpec(H, D, self.vdim, rot_dims, rot_base, ctypes.cast(d, _ffi.P(ctypes.c_double)), eps, 0)
+        spec = _ffi.RetentionSpec(H, D, self.vdim, rot_dims, rot_base, ctypes.cast(d, _ffi.P(ctypes.c_double)), eps, int(exact))
         out = np.empty((n, T, H, self.vdim), dtype=np.float32)
         _check(self.ctx.handle, _ffi.lib().skn_retention(self._h, ctypes.byref(spec), seq, n, T, pos.ctypes.data, max_ctx, q.ctypes.data,
                                                         k.ctypes.data, v.ctypes.data, g.ctypes.data, out.ctypes.data))

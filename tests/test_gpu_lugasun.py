@@ -192,8 +192,9 @@ def retention_reference(q, k, v, gate, decay, rot, eps):
     return plain.rms_unit(o, eps) * plain.silu(gate), S
 
 
-@pytest.mark.parametrize("H,D,V", [(2, 32, 32), (3, 24, 40), (1, 128, 128), (2, 20, 13), (1, 70, 260), (5, 8, 64)])
-def test_retention(ctx, H, D, V):
+@pytest.mark.parametrize("exact", [False, True])
+@pytest.mark.parametrize("H,D,V", [(2, 32, 32), (3, 24, 40), (1, 128, 128), (2, 20, 13), (1, 70, 260), (5, 8, 64), (1, 200, 136)])
+def test_retention(ctx, H, D, V, exact):
     g = np.random.default_rng(D + V)
     T, rot, decay = 200, {"dims": D // 4 * 2, "base": 90.0}, [0.999, 0.5, 0.97, 1.0, 0.9][:H]
     q, k, v, gate = (g.standard_normal((T, H, d)).astype(np.float32) for d in (D, D, V, V))
@@ -202,7 +203,7 @@ def test_retention(ctx, H, D, V):
         st = RecurrentState(ctx, 1, H, D, V)
         out, at = [], 0
         for n in cuts:
-            out.append(st.retain(*(a[None, at:at + n] for a in (q, k, v, gate)), [at], decay, rot_dims=rot["dims"], rot_base=rot["base"])[0])
+            out.append(st.retain(*(a[None, at:at + n] for a in (q, k, v, gate)), [at], decay, rot_dims=rot["dims"], rot_base=rot["base"], exact=exact)[0])
             at += n
         assert rel(np.concatenate(out), want) < 2e-5, cuts
         assert rel(st.read(0), S) < 2e-5, cuts
