@@ -97,7 +97,7 @@ static inline cudaError_t skn_launch_pdl(void (*kern)(KArgs...), dim3 grid, dim3
     cudaLaunchAttribute attr[2];
     int n = 0;
     attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[n++].val.programmaticStreamSerializationAllowed = 1;
+    attr[n++].val.programmaticStreamSerializationAllowed = skn_tune_int("SKN_PDL", 1);
     if (cluster > 1) {
         attr[n].id = cudaLaunchAttributeClusterDimension;
         attr[n].val.clusterDim.x = cluster;

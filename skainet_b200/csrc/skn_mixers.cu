@@ -89,10 +89,11 @@ __device__ __forceinline__ void put_out(const skn_rows_out &o, int64_t m, int64_
 }
 
 // ---- attention over a split of the keys ---------------------------------------------------------------------------
-// smem (floats): q [RT][kp] | key [kp] | value [vp] | weights [RT][KS] | red [MIX_THREADS][RT * VE]
+// smem (floats): q [RT][kp] | key [kp] | value [vp] | weights [RT][KS] | red [partial sums][RT][vp]
 template <class CT, int RT>
 static size_t attn_split_smem(int kp, int vp) {
-    return ((size_t)RT * kp + kp + vp + RT * KS + (size_t)MIX_THREADS * RT * CacheVec<CT>::N) * sizeof(float);
+    const int ng = vp / CacheVec<CT>::N, parts = ng <= 32 && 32 % ng == 0 ? MIX_THREADS / 32 : MIX_THREADS / ng;
+    return ((size_t)RT * kp + kp + vp + RT * KS + (size_t)parts * RT * vp) * sizeof(float);
 }
 
 template <class CT, int RT, bool APPEND>
@@ -114,6 +115,14 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
     float *qs = sm, *kn = qs + RT * kp, *vn = kn + kp, *ws = vn + vp, *red = ws + RT * KS;
     const size_t head_rows = ((size_t)slot * G + g) * cap;
     CT *kc = const_cast<CT *>(kc_) + head_rows * kp, *vc = const_cast<CT *>(vc_) + head_rows * vp;
+    // keys and values on their way into L2 while the query is prepared: two threads per key
+    const int key = tid >> 1, half = tid & 1;
+    const int kslot = (j0 + key) % cap;
+    if (key < nk) {
+        const char *kr = reinterpret_cast<const char *>(kc + (size_t)kslot * kp), *vr = reinterpret_cast<const char *>(vc + (size_t)kslot * vp);
+        for (int i = half * 128; i < (int)(kp * sizeof(CT)); i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(kr + i));
+        for (int i = half * 128; i < (int)(vp * sizeof(CT)); i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(vr + i));
+    }
 
     for (int i = warp; i < RT + 2; i += MIX_THREADS / 32) {
         if (i < RT) {
@@ -136,13 +145,12 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
     __syncthreads();
 
     // scores: two threads per key, each takes every other vector of the row
-    const int key = tid >> 1, half = tid & 1;
     const bool valid = key < nk, own = newest && key == nk - 1;
     float s[RT];
 #pragma unroll
     for (int r = 0; r < RT; ++r) s[r] = 0.f;
     if (valid) {
-        const CT *kr = kc + (size_t)((j0 + key) % cap) * kp;
+        const CT *kr = kc + (size_t)kslot * kp;
 #pragma unroll 4
         for (int u = half; u < kp / VE; u += 2) {
             float kv[VE];
@@ -198,13 +206,16 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
 #pragma unroll
         for (int e = 0; e < VE; ++e) acc[r][e] = 0.f;
     if (kk < kl) {
+        const int first = j0 % cap;
 #pragma unroll 4
         for (int j = kk; j < nk; j += kl) {
             float vv[VE];
+            int sl = first + j;
+            if (sl >= cap) sl -= cap;              // (a cache holds at least the keys that one query sees)
             if (newest && j == nk - 1) {
 #pragma unroll
                 for (int e = 0; e < VE; ++e) vv[e] = vn[cg_ * VE + e];
-            } else CacheVec<CT>::load(vc + (size_t)((j0 + j) % cap) * vp + cg_ * VE, vv);
+            } else CacheVec<CT>::load(vc + (size_t)sl * vp + cg_ * VE, vv);
 #pragma unroll
             for (int r = 0; r < RT; ++r) {
                 const float w = ws[r * KS + j];
@@ -212,13 +223,25 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
                 for (int e = 0; e < VE; ++e) acc[r][e] = fmaf(w, vv[e], acc[r][e]);
             }
         }
+    }
+    // a column vector's partial sums: first across the lanes of a warp that hold the same columns, then across the warps
+    const bool fold = ng <= 32 && 32 % ng == 0;
+    if (fold) {
+        for (int o = ng; o < 32; o <<= 1)
+#pragma unroll
+            for (int r = 0; r < RT; ++r)
+#pragma unroll
+                for (int e = 0; e < VE; ++e) acc[r][e] += __shfl_xor_sync(0xffffffffu, acc[r][e], o);
+    }
+    const int part = fold ? warp : kk;
+    if (kk < kl && (!fold || lane < ng)) {
 #pragma unroll
         for (int r = 0; r < RT; ++r)
 #pragma unroll
-            for (int e = 0; e < VE; ++e) red[((size_t)kk * RT + r) * vp + cg_ * VE + e] = acc[r][e];
+            for (int e = 0; e < VE; ++e) red[((size_t)part * RT + r) * vp + cg_ * VE + e] = acc[r][e];
     }
     __syncthreads();
-    const int nk_l = min(kl, nk);
+    const int nk_l = fold ? MIX_THREADS / 32 : min(kl, nk);
     for (int i = tid; i < nh * vdim; i += MIX_THREADS) {
         const int r = i / vdim, c = i % vdim;
         float o = 0.f;
@@ -239,19 +262,30 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
     __syncthreads();
     if (!s_last) return;
     __threadfence();
+    // weight of every split (in place of the scores): exp(max - top) / sum
+    for (int r = warp; r < nh; r += MIX_THREADS / 32) {
+        const float *rec = a.scratch + ((size_t)m * a.heads + h0 + r) * max_splits * (vdim + 2);
+        float top = -INFINITY;
+        for (int x = lane; x < live; x += 32) top = fmaxf(top, __ldcg(rec + (size_t)x * (vdim + 2)));
+        top = warp_max(top);
+        float den = 0.f;
+        for (int x = lane; x < live; x += 32) den += expf(__ldcg(rec + (size_t)x * (vdim + 2)) - top) * __ldcg(rec + (size_t)x * (vdim + 2) + 1);
+        den = warp_sum(den);
+        for (int x = lane; x < live; x += 32)
+            if (x < KS) ws[r * KS + x] = expf(__ldcg(rec + (size_t)x * (vdim + 2)) - top) / den;
+        if (lane == 0) { s_max[r] = top; s_sum[r] = den; }
+    }
+    __syncthreads();
     for (int i = tid; i < nh * vdim; i += MIX_THREADS) {
         const int r = i / vdim, c = i % vdim;
         const float *rec = a.scratch + ((size_t)m * a.heads + h0 + r) * max_splits * (vdim + 2);
-        float top = -INFINITY;
-        for (int x = 0; x < live; ++x) top = fmaxf(top, __ldcg(rec + (size_t)x * (vdim + 2)));
-        float num = 0.f, den = 0.f;
+        float num = 0.f;
+#pragma unroll 8
         for (int x = 0; x < live; ++x) {
-            const float *q = rec + (size_t)x * (vdim + 2);
-            const float f = expf(__ldcg(q) - top);
-            den = fmaf(f, __ldcg(q + 1), den);
-            num = fmaf(f, __ldcg(q + 2 + c), num);
+            const float f = x < KS ? ws[r * KS + x] : expf(__ldcg(rec + (size_t)x * (vdim + 2)) - s_max[r]) / s_sum[r];
+            num = fmaf(f, __ldcg(rec + (size_t)x * (vdim + 2) + 2 + c), num);
         }
-        put_out(a.out, m, (int64_t)(h0 + r) * vdim + c, num / den * a.out_scale);
+        put_out(a.out, m, (int64_t)(h0 + r) * vdim + c, num * a.out_scale);
     }
     if (tid == 0) *ticket = 0;
 }
@@ -321,11 +355,12 @@ __device__ void ret_step(const skn_ret_args &r, const skn_step &st, float *__res
 }
 
 template <class CT, int RT>
-__global__ void __launch_bounds__(MIX_THREADS)
+__global__ void __launch_bounds__(MIX_THREADS, 4)
 skn_mix_decode_kernel(skn_attn_args a, skn_ret_args r, skn_step st, const CT *kc, const CT *vc, int G, int cap, int dim, int vdim, int kp,
                       int vp, int max_splits, int n_attn, float *S, int RH, int rdk, int rdv, int rvp) {
     extern __shared__ __align__(16) float sm[];
-    skn_pdl_launch_dependents();
+    // the next launch starts only when this one's CTAs end (no early trigger): the weights it would stream meanwhile make
+    // every step of this chain of dependent loads wait longer
     skn_pdl_wait();
     const int m = blockIdx.y, b = blockIdx.x;
     if (b < n_attn) attn_split<CT, RT, true>(a, st, kc, vc, G, cap, dim, vdim, kp, vp, b % max_splits, max_splits, b / max_splits, m, sm);

@@ -182,7 +182,6 @@ skn_token_side_kernel(const uint8_t *__restrict__ wg, int64_t pitch_g, const uin
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int D8 = (int)(pitch_g / 2), S8 = (int)(pitch_p / 2);
     float *xs = sm, *gs = sm + D8, *ys = gs + S8;
-    skn_pdl_launch_dependents();
     // this CTA's weights are on their way into L2 while the kernel before still runs
     const int per = (D + SIDE_CLUSTER - 1) / SIDE_CLUSTER, n0 = rank * per, n1 = min(D, n0 + per);
     for (int j = rank + SIDE_CLUSTER * warp; j < S; j += SIDE_CLUSTER * (SIDE_THREADS / 32))
