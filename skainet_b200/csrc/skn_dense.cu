@@ -118,7 +118,6 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
         skn_fence_mbar_init();
     }
     __syncthreads();
-    skn_pdl_launch_dependents();
     if (warp == MVD_WARPS) {
         if (lane == 0) {
             int s = 0;
@@ -231,6 +230,8 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
 #pragma unroll
             for (int j = 0; j < 8; ++j) acc[m][j] = 0.f;
         const int rows = min(8, r1 - r0 - g0);
+        // the next launch comes in under the last rows: earlier, its own stream of weights delays this one's
+        if (g0 + 16 >= r1 - r0 && g0 + 8 < r1 - r0) skn_pdl_launch_dependents();
 #pragma unroll
         for (int j0 = 0; j0 < 8; j0 += GR) {
             if (j0 < rows) {
@@ -464,7 +465,6 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = tmem_slot;
-    skn_pdl_launch_dependents();
     // the weights depend on no kernel before this one: the first unit's first stages are requested ahead of the wait
     int early = 0;
     if (warp == 5 && lane == 0 && (int)blockIdx.x < units) {
@@ -499,6 +499,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                     tc_tma_load_2d(a + DTC_A_BYTES, &tmap_x, k * DTC_BK, m0, &full_bar[s]);
                 }
             }
+            skn_pdl_launch_dependents();           // every load of this CTA is on its way: the next launch may come in
             // the last copies have landed before this CTA ends: drain the stages still in flight
             for (int j = it > stages ? it - stages : 0; j < it && ok; ++j)
                 if (!skn_mbar_wait(&full_bar[j % stages], (uint32_t)(j / stages) & 1u)) {
@@ -638,7 +639,7 @@ static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense
             }
         }
     }
-    while (NT > 64 && nt * ((M + NT - 1) / NT) * 2 <= sms) NT = NT == 192 ? 128 : NT / 2;
+    while (NT > 32 && nt * ((M + NT - 1) / NT) * 2 <= sms) NT = NT == 192 ? 128 : NT / 2;
     const int mt = (M + NT - 1) / NT;
     // K splits that even out the load of the SMs (the tiles of a decode-size step are fewer than the SMs, or not many more)
     int splits = 1;
