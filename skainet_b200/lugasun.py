@@ -7,7 +7,7 @@ them by the same number of tokens."""
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass, field
+from dataclasses import dataclass
 from typing import List, Optional, Sequence
 
 import numpy as np
@@ -92,7 +92,6 @@ class LugasunConfig:
     eps: float = 1e-5
     side_dim: int = 0           # 0: no token side input
     loop: Optional[tuple] = None  # (start, stop, times)
-    extra: dict = field(default_factory=dict)
 
     @classmethod
     def from_dict(cls, d: dict) -> "LugasunConfig":
