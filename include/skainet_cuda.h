@@ -252,11 +252,13 @@ int32_t skn_kv_create_typed(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int
                             int32_t kv_dtype, skn_kvcache **out);
 /* A position-addressed cache: the token at position p of sequence b occupies slot p % capacity of
  * K [batch][n_kv_heads][capacity][k_dim rounded up to 16] and V (v_dim likewise), fp32 or bf16 (SKN_KV_F32 /
- * SKN_KV_BF16), k_dim and v_dim up to SKN_ATTN_MAX_DIM.  It does not count tokens: its owner passes the positions, so
+ * SKN_KV_BF16), k_dim and v_dim up to SKN_KV_MAX_DIM; v_dim 0 keeps no V (a latent cache, whose values are the start
+ * of its key rows).  It does not count tokens: its owner passes the positions, so
  * a freed sequence needs no clearing, and attention that never looks further back than a chunk needs no more slots
  * than a chunk and one step's tokens.  Served by skn_chunk_attn and the decoders over dense weights; the ring
  * operations below (append, load, gather, skn_attn_*) refuse it with SKN_ERR_BAD_HANDLE. */
 #define SKN_ATTN_MAX_DIM 512
+#define SKN_KV_MAX_DIM 1024
 int32_t skn_kv_create_by_position(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int32_t k_dim, int32_t v_dim, int32_t capacity,
                                   int32_t kv_dtype, skn_kvcache **out);
 /* element type of the cache (what k_dev / v_dev of skn_kv_info point at) */
@@ -414,14 +416,15 @@ int32_t skn_llama_position(const skn_llama *m);
 
 /* ---- Token mixers of decoders over dense weights ------------------------------------------------
  * No counterpart in the reference (no attention, no recurrence).  Host-pointer forms of the mechanisms
- * that skn_lugasun_* runs on the device; each advances `n_seqs` sequences (slots seq0 ..) by T tokens,
+ * that the decoders run on the device; each advances `n_seqs` sequences (slots seq0 ..) by T tokens,
  * pos_host[s] tokens having come before.  Raw heads are [n_seqs][T][heads][dim] fp32. */
 typedef struct skn_state skn_state;
 
 /* Softmax attention with per-head RMS norm of q and k, rotation of the first rot_dims dimensions of q
  * and k (dimension i pairs with i + rot_dims / 2, angle pos * rot_base^(-2 i / rot_dims)), scores
  * scale * (q . k) optionally capped to softcap * tanh(score / softcap), and visibility of the earlier
- * keys of the query's own chunk of `chunk` positions (counted from position 0). */
+ * keys of the query's own chunk of `chunk` positions (counted from position 0), or of the last `window`
+ * positions, the query's included. */
 typedef struct skn_attn_spec {
     int32_t heads, kv_heads, dim, vdim;
     int32_t rot_dims;    /* 0: no rotation */
@@ -429,7 +432,7 @@ typedef struct skn_attn_spec {
     double rot_base;
     float scale, softcap; /* softcap 0: none */
     float eps;           /* of the q / k norms */
-    int32_t reserved;
+    int32_t window;      /* 0: none */
 } skn_attn_spec;
 /* Linear attention with one decay per head: S <- decay S + k v^T, o = S^T q, with q and k rotated as
  * above and k divided by sqrt(dim); each head's o is divided by its root mean square and multiplied by
@@ -448,25 +451,44 @@ int32_t skn_state_create(skn_ctx *ctx, int32_t slots, int32_t heads, int32_t k_d
 int32_t skn_state_destroy(skn_state *s);
 int32_t skn_state_read(skn_state *s, int32_t slot, float *out_host);
 /* out [n_seqs][T][heads][vdim]; the new keys and values enter the cache.  q_gain, k_gain [dim]: gains of the norms, or
- * both NULL for no norm. */
+ * both NULL for no norm.  sink [heads] or NULL: a score that joins each head's softmax denominator, without a value. */
 int32_t skn_chunk_attn(skn_kvcache *kv, const skn_attn_spec *spec, int32_t seq0, int32_t n_seqs, int32_t T, const int32_t *pos_host,
                        int32_t max_ctx, const float *q_gain_host, const float *k_gain_host, const float *q_host, const float *k_host,
-                       const float *v_host, float *out_host);
+                       const float *v_host, const float *sink_host, float *out_host);
 int32_t skn_retention(skn_state *s, const skn_retention_spec *spec, int32_t seq0, int32_t n_seqs, int32_t T, const int32_t *pos_host,
                       int32_t max_ctx, const float *q_host, const float *k_host, const float *v_host, const float *g_host, float *out_host);
 
-/* ---- Lugasun decoder ----------------------------------------------------------------------------
- * Embedding -> layers -> RMS norm -> logits over the embedding table.  A layer adds to the residual stream (fp32):
- * a mixer (chunked attention and retention side by side on the same normalised input, each with its own weight
- * in the sum), an optional squared-relu feed-forward, and an optional token side input (a gate times a row of a
- * second embedding table, projected and normalised).  Layers loop_start .. loop_stop - 1 run loop_times
- * times in a row with a cache and a state per pass, each pass starting from loop_in [x; embedding].
- * Weights are dense bf16; matrix products run on bf16 operands with fp32 accumulation (SKN_LUGASUN_BF16)
- * or in fp32 throughout (SKN_LUGASUN_F32).  The decoder keeps max_seqs sequences of any lengths; a step
- * advances a contiguous range of them by the same number of tokens. */
-typedef struct skn_lugasun skn_lugasun;
-#define SKN_LUGASUN_F32 0
-#define SKN_LUGASUN_BF16 1
+/* ---- Decoders over dense weights ------------------------------------------------------------------
+ * Embedding -> layers -> RMS norm -> logits over the embedding table, the residual stream in fp32.  Weights are dense
+ * bf16; matrix products run on bf16 operands with fp32 accumulation (SKN_DECODER_BF16) or in fp32 throughout
+ * (SKN_DECODER_F32).  Layers loop_start .. loop_stop - 1 may run loop_times times in a row, with a cache or state per
+ * pass.  A decoder keeps max_seqs sequences of any lengths; a step advances a contiguous range of them by the same number
+ * of tokens.  The models (skn_lugasun_create, skn_tutezen_create) differ in their layers; every other call serves all. */
+typedef struct skn_decoder skn_decoder;
+#define SKN_DECODER_F32 0
+#define SKN_DECODER_BF16 1
+int32_t skn_decoder_destroy(skn_decoder *m);
+/* forget the tokens of sequence seq (-1: of all) */
+int32_t skn_decoder_reset(skn_decoder *m, int32_t seq);
+int32_t skn_decoder_position(const skn_decoder *m, int32_t seq);
+/* One step: T new tokens for each of the sequences seq0 .. seq0 + n_seqs - 1 (n_seqs * T <= max_tokens);
+ * tokens [n_seqs][T], NULL with T == 1 feeds back the greedy ids of those sequences.  want_rows: the
+ * n_want rows (s * T + t, any order) whose logits [n_want][vocab] are returned; next_host [n_seqs]: the
+ * greedy token after each sequence's last position.  With neither the output layer is skipped. */
+int32_t skn_decoder_forward(skn_decoder *m, int32_t seq0, int32_t n_seqs, const int32_t *tokens_host, int32_t T, int32_t n_want,
+                            const int32_t *want_rows_host, float *logits_host, int32_t *next_host);
+/* Enqueue only; head != 0 computes logits and greedy ids of every sequence's last position.  A single-token step
+ * with tokens_dev == NULL may be captured into a CUDA graph; replays advance the device positions but not
+ * skn_decoder_position, and a step past max_ctx is reported by skn_sync as SKN_ERR_SHAPE. */
+int32_t skn_decoder_forward_dev(skn_decoder *m, int32_t seq0, int32_t n_seqs, const int32_t *tokens_dev, int32_t T, int32_t head);
+/* residual stream after every layer run of the last step: [layer runs][rows][width], recorded while `on` */
+int32_t skn_decoder_trace(skn_decoder *m, int32_t on, int32_t rows, float *out_host);
+
+/* ---- Lugasun ---------------------------------------------------------------------------------------
+ * A layer adds to the residual stream: a mixer (chunked attention and retention side by side on the same normalised
+ * input, each with its own weight in the sum), an optional squared-relu feed-forward, and an optional token side input (a
+ * gate times a row of a second embedding table, projected and normalised).  Each pass of the loop starts from
+ * loop_in [x; embedding]. */
 typedef struct skn_lugasun_layer {
     skn_attn_spec left;
     skn_retention_spec right;
@@ -489,27 +511,71 @@ typedef struct skn_lugasun_weights {
     const float *norm1, *norm2, *q_gain, *k_gain, *side_norm;
 } skn_lugasun_weights;
 int32_t skn_lugasun_create(skn_ctx *ctx, const skn_lugasun_spec *spec, int32_t max_seqs, int32_t max_tokens, int32_t max_ctx,
-                           int32_t dtype, skn_lugasun **out);
-int32_t skn_lugasun_destroy(skn_lugasun *m);
-int32_t skn_lugasun_set_layer(skn_lugasun *m, int32_t layer, const skn_lugasun_weights *w);
+                           int32_t dtype, skn_decoder **out);
+int32_t skn_lugasun_set_layer(skn_decoder *m, int32_t layer, const skn_lugasun_weights *w);
 /* loop_in and side_embed may be NULL when the model has no loop / no side input */
-int32_t skn_lugasun_set_head(skn_lugasun *m, const skn_tensor *embed, const float *final_norm_host, const skn_tensor *loop_in,
+int32_t skn_lugasun_set_head(skn_decoder *m, const skn_tensor *embed, const float *final_norm_host, const skn_tensor *loop_in,
                              const skn_tensor *side_embed);
-/* forget the tokens of sequence seq (-1: of all) */
-int32_t skn_lugasun_reset(skn_lugasun *m, int32_t seq);
-int32_t skn_lugasun_position(const skn_lugasun *m, int32_t seq);
-/* One step: T new tokens for each of the sequences seq0 .. seq0 + n_seqs - 1 (n_seqs * T <= max_tokens);
- * tokens [n_seqs][T], NULL with T == 1 feeds back the greedy ids of those sequences.  want_rows: the
- * n_want rows (s * T + t, any order) whose logits [n_want][vocab] are returned; next_host [n_seqs]: the
- * greedy token after each sequence's last position.  With neither the output layer is skipped. */
-int32_t skn_lugasun_forward(skn_lugasun *m, int32_t seq0, int32_t n_seqs, const int32_t *tokens_host, int32_t T, int32_t n_want,
-                            const int32_t *want_rows_host, float *logits_host, int32_t *next_host);
-/* Enqueue only; head != 0 computes logits and greedy ids of every sequence's last position.  A single-token step
- * with tokens_dev == NULL may be captured into a CUDA graph; replays advance the device positions but not
- * skn_lugasun_position, and a step past max_ctx is reported by skn_sync as SKN_ERR_SHAPE. */
-int32_t skn_lugasun_forward_dev(skn_lugasun *m, int32_t seq0, int32_t n_seqs, const int32_t *tokens_dev, int32_t T, int32_t head);
-/* residual stream after every layer run of the last step: [layer runs][rows][width], recorded while `on` */
-int32_t skn_lugasun_trace(skn_lugasun *m, int32_t on, int32_t rows, float *out_host);
+
+/* ---- Tutezen ---------------------------------------------------------------------------------------
+ * Parallel layers: x <- x + residual_mult * (mixer(h) + feed-forward(h)) with one norm, h = norm(x).  The mixer is a
+ * selective state space (skn_ssm_spec) or latent attention (skn_latent_spec); the feed-forward is absent, dense (tanh gelu)
+ * or a mixture of experts (gated, silu) with an optional shared expert.  Before pass t of the loop x takes
+ * loop_step[t], and from the second pass on the embedding output again.
+ *
+ * Head and latent widths are padded to multiples of 8 with zero weights, written ~ below: ~n is n rounded up. */
+/* y_t = S_t^T C_t + D x_t, S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T per head, x, B, C out of a causal
+ * convolution of `taps` taps with silu, dt_t = softplus; head h reads B and C of group h / (heads / groups).  y times
+ * silu(z) is RMS-normed in norm_groups parts. */
+typedef struct skn_ssm_spec {
+    int32_t heads, vdim, state, groups, taps, norm_groups;
+    float eps;
+    int32_t reserved;
+} skn_ssm_spec;
+/* Queries and keys / values go through latents of q_rank and kv_rank (RMS-normed); a key is [dim from the latent |
+ * rot_dim rotated, shared by the heads], adjacent dimensions of the rotated part forming pairs (the first rot_dims turn).  Only the
+ * latent and the rotated key part are cached.  Query i sees keys j with 0 <= i - j < window (0: all earlier ones); one learned score
+ * per head joins the softmax denominator; the heads are multiplied by a sigmoid gate. */
+typedef struct skn_latent_spec {
+    int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank, rot_dims, window;
+    double rot_base;
+    float scale, eps;
+} skn_latent_spec;
+#define SKN_MIXER_SSM 0
+#define SKN_MIXER_LATENT 1
+typedef struct skn_tutezen_layer {
+    int32_t mixer;       /* SKN_MIXER_* */
+    int32_t ff;          /* width of a dense feed-forward (0: none, or a mixture) */
+    int32_t experts, top, expert_ff, shared_ff; /* experts 0: no mixture; shared_ff 0: no shared expert */
+    skn_ssm_spec ssm;
+    skn_latent_spec latent;
+} skn_tutezen_layer;
+typedef struct skn_tutezen_spec {
+    int32_t n_layers, width, vocab;
+    int32_t loop_start, loop_stop, loop_times; /* loop_times 0: no loop */
+    float eps, residual_mult;
+    const skn_tutezen_layer *layers;
+} skn_tutezen_spec;
+/* Weights of one layer, borrowed (they must outlive the decoder); float vectors are host arrays, copied.
+ * w_in [.., width], everything that reads h, stacked by rows:
+ *   state space: z [heads][~vdim] | x [heads][~vdim] | B [groups][~state] | C [groups][~state] | dt [~heads]
+ *   latent: dq [~q_rank] | dkv [~kv_rank] | rotated key [rp] | g [heads][~vdim]; rp: rot_dim padded so that ~dim + rp is a
+ *     multiple of 16
+ *   then router [~experts], then dense up [~ff] or shared expert [~shared_ff][gate, up] (pairs of rows)
+ * w_out [width, mixer heads * ~vdim + ~ff or ~shared_ff]: o and down side by side.
+ * latent: uq [heads * (~dim + rp), q_rank]; ukv [uk: heads * ~dim | uv: heads * ~vdim, kv_rank].
+ * experts: e_in [experts * ~expert_ff * 2, width], rows of an expert in pairs (gate, up); e_out [experts * width, ~expert_ff].
+ * conv [channels][taps], conv_b [channels]: channels as in w_in (x | B | C); dt_bias, a_log, d, sink [heads];
+ * out_norm [heads][~vdim]; q_gain [q_rank], kv_gain [kv_rank]. */
+typedef struct skn_tutezen_weights {
+    const skn_tensor *w_in, *w_out, *uq, *ukv, *e_in, *e_out;
+    const float *norm, *conv, *conv_b, *dt_bias, *a_log, *d, *out_norm, *q_gain, *kv_gain, *sink;
+} skn_tutezen_weights;
+int32_t skn_tutezen_create(skn_ctx *ctx, const skn_tutezen_spec *spec, int32_t max_seqs, int32_t max_tokens, int32_t max_ctx,
+                           int32_t dtype, skn_decoder **out);
+int32_t skn_tutezen_set_layer(skn_decoder *m, int32_t layer, const skn_tutezen_weights *w);
+/* loop_step_host [loop_times][width], NULL without a loop */
+int32_t skn_tutezen_set_head(skn_decoder *m, const skn_tensor *embed, const float *final_norm_host, const float *loop_step_host);
 
 /* ---- GGUF container --------------------------------------------------------------------------
  * Memory-mapped GGUF v2 / v3 reader with 64-bit offsets; tensor data is handed out as pointers

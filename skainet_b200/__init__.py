@@ -13,7 +13,8 @@ from .nn import MLP, Module, QuantLinear, ReLU, load_model_weights  # noqa: E402
 
 __all__ += ["LlamaConfig", "LlamaDecoder", "MLP", "Module", "ReLU", "load_model_weights"]
 from .lugasun import LugasunConfig, LugasunDecoder  # noqa: E402
+from .tutezen import TutezenConfig, TutezenDecoder  # noqa: E402
 from .registry import ARCHITECTURES, load_model  # noqa: E402
 from .generate import generate  # noqa: E402
 
-__all__ += ["ARCHITECTURES", "LugasunConfig", "LugasunDecoder", "generate", "load_model"]
+__all__ += ["ARCHITECTURES", "LugasunConfig", "LugasunDecoder", "TutezenConfig", "TutezenDecoder", "generate", "load_model"]

@@ -21,7 +21,7 @@ P = ctypes.POINTER
 class AttnSpec(ctypes.Structure):
     _fields_ = [("heads", c_i32), ("kv_heads", c_i32), ("dim", c_i32), ("vdim", c_i32), ("rot_dims", c_i32), ("chunk", c_i32),
                 ("rot_base", ctypes.c_double), ("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("eps", ctypes.c_float),
-                ("reserved", c_i32)]
+                ("window", c_i32)]
 
 
 class RetentionSpec(ctypes.Structure):
@@ -42,6 +42,31 @@ class LugasunSpec(ctypes.Structure):
 class LugasunWeights(ctypes.Structure):
     _fields_ = [(n, c_vp) for n in ("w_in", "w_out", "up", "down", "side_gate", "side_proj", "norm1", "norm2", "q_gain", "k_gain",
                                     "side_norm")]
+
+
+class SsmSpec(ctypes.Structure):
+    _fields_ = [("heads", c_i32), ("vdim", c_i32), ("state", c_i32), ("groups", c_i32), ("taps", c_i32), ("norm_groups", c_i32),
+                ("eps", ctypes.c_float), ("reserved", c_i32)]
+
+
+class LatentSpec(ctypes.Structure):
+    _fields_ = [("heads", c_i32), ("dim", c_i32), ("rot_dim", c_i32), ("vdim", c_i32), ("q_rank", c_i32), ("kv_rank", c_i32),
+                ("rot_dims", c_i32), ("window", c_i32), ("rot_base", ctypes.c_double), ("scale", ctypes.c_float), ("eps", ctypes.c_float)]
+
+
+class TutezenLayer(ctypes.Structure):
+    _fields_ = [("mixer", c_i32), ("ff", c_i32), ("experts", c_i32), ("top", c_i32), ("expert_ff", c_i32), ("shared_ff", c_i32),
+                ("ssm", SsmSpec), ("latent", LatentSpec)]
+
+
+class TutezenSpec(ctypes.Structure):
+    _fields_ = [("n_layers", c_i32), ("width", c_i32), ("vocab", c_i32), ("loop_start", c_i32), ("loop_stop", c_i32), ("loop_times", c_i32),
+                ("eps", ctypes.c_float), ("residual_mult", ctypes.c_float), ("layers", P(TutezenLayer))]
+
+
+class TutezenWeights(ctypes.Structure):
+    _fields_ = [(n, c_vp) for n in ("w_in", "w_out", "uq", "ukv", "e_in", "e_out", "norm", "conv", "conv_b", "dt_bias", "a_log", "d",
+                                    "out_norm", "q_gain", "kv_gain", "sink")]
 
 
 # name -> (restype, argtypes)
@@ -110,17 +135,20 @@ SIGNATURES = {
     "skn_state_create": (c_i32, [c_vp, c_i32, c_i32, c_i32, c_i32, P(c_vp)]),
     "skn_state_destroy": (c_i32, [c_vp]),
     "skn_state_read": (c_i32, [c_vp, c_i32, c_vp]),
-    "skn_chunk_attn": (c_i32, [c_vp, P(AttnSpec), c_i32, c_i32, c_i32, c_vp, c_i32, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp]),
+    "skn_chunk_attn": (c_i32, [c_vp, P(AttnSpec), c_i32, c_i32, c_i32, c_vp, c_i32, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp]),
     "skn_retention": (c_i32, [c_vp, P(RetentionSpec), c_i32, c_i32, c_i32, c_vp, c_i32, c_vp, c_vp, c_vp, c_vp, c_vp]),
     "skn_lugasun_create": (c_i32, [c_vp, P(LugasunSpec), c_i32, c_i32, c_i32, c_i32, P(c_vp)]),
-    "skn_lugasun_destroy": (c_i32, [c_vp]),
     "skn_lugasun_set_layer": (c_i32, [c_vp, c_i32, P(LugasunWeights)]),
     "skn_lugasun_set_head": (c_i32, [c_vp, c_vp, c_vp, c_vp, c_vp]),
-    "skn_lugasun_reset": (c_i32, [c_vp, c_i32]),
-    "skn_lugasun_position": (c_i32, [c_vp, c_i32]),
-    "skn_lugasun_forward": (c_i32, [c_vp, c_i32, c_i32, c_vp, c_i32, c_i32, c_vp, c_vp, c_vp]),
-    "skn_lugasun_forward_dev": (c_i32, [c_vp, c_i32, c_i32, c_vp, c_i32, c_i32]),
-    "skn_lugasun_trace": (c_i32, [c_vp, c_i32, c_i32, c_vp]),
+    "skn_tutezen_create": (c_i32, [c_vp, P(TutezenSpec), c_i32, c_i32, c_i32, c_i32, P(c_vp)]),
+    "skn_tutezen_set_layer": (c_i32, [c_vp, c_i32, P(TutezenWeights)]),
+    "skn_tutezen_set_head": (c_i32, [c_vp, c_vp, c_vp, c_vp]),
+    "skn_decoder_destroy": (c_i32, [c_vp]),
+    "skn_decoder_reset": (c_i32, [c_vp, c_i32]),
+    "skn_decoder_position": (c_i32, [c_vp, c_i32]),
+    "skn_decoder_forward": (c_i32, [c_vp, c_i32, c_i32, c_vp, c_i32, c_i32, c_vp, c_vp, c_vp]),
+    "skn_decoder_forward_dev": (c_i32, [c_vp, c_i32, c_i32, c_vp, c_i32, c_i32]),
+    "skn_decoder_trace": (c_i32, [c_vp, c_i32, c_i32, c_vp]),
     "skn_gguf_open": (c_i32, [ctypes.c_char_p, P(c_vp)]),
     "skn_gguf_close": (c_i32, [c_vp]),
     "skn_gguf_counts": (c_i32, [c_vp, P(c_i32), P(c_i64), P(c_i64), P(c_i64), P(c_i64)]),

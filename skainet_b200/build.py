@@ -31,7 +31,9 @@ def _nvcc() -> str:
 
 
 # translation units of a model family (the entry points of the others are absent from its library)
-FAMILIES = {"lugasun": ["skn_core.cu", "skn_kv_cache.cu", "skn_dense.cu", "skn_rows.cu", "skn_mixers.cu", "skn_glue.cu", "skn_lugasun.cu"]}
+DENSE = ["skn_core.cu", "skn_kv_cache.cu", "skn_dense.cu", "skn_rows.cu", "skn_mixers.cu", "skn_glue.cu", "skn_decoder.cu"]
+FAMILIES = {"lugasun": DENSE + ["skn_lugasun.cu"],
+            "tutezen": DENSE + ["skn_ssm.cu", "skn_latent.cu", "skn_moe.cu", "skn_tutezen.cu"]}
 
 
 def sources(family: str | None = None) -> list[str]:

@@ -13,10 +13,21 @@
 __device__ __forceinline__ float dense_gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+// 0.5 (1 + tanh u) = 1 / (1 + exp(-2 u)); relative error a few 1e-7
+__device__ __forceinline__ float dense_gelu_exp(float z) {
+    return __fdividef(z, 1.f + __expf(fminf(-1.5957691216057308f * (z + 0.044715f * z * z * z), 80.f)));
+}
+__device__ __forceinline__ float dense_silu(float z) { return __fdividef(z, 1.f + __expf(fminf(-z, 80.f))); }
 
 template <int EPI>
 __device__ __forceinline__ void dense_store(const skn_epi &e, int64_t m, int64_t n, float v) {
-    if (EPI == SKN_EPI_ADD) v += e.resid[m * e.ld_resid + n];
+    if (EPI == SKN_EPI_ADD) v = fmaf(e.alpha, v, e.resid[m * e.ld_resid + n]);
+    if (EPI == SKN_EPI_GELU_TAIL && n >= e.n_act) {
+        v = dense_gelu_exp(v);
+        if (e.act32) e.act32[m * e.ld_act32 + n - e.n_act] = v;
+        if (e.act16) e.act16[m * e.ld_act16 + n - e.n_act] = __float2bfloat16_rn(v);
+        return;
+    }
     if (EPI == SKN_EPI_RELU2) {
         v = fmaxf(v, 0.f);
         v *= v;
@@ -30,6 +41,42 @@ __device__ __forceinline__ void dense_store(const skn_epi &e, int64_t m, int64_t
     if (e.y16) e.y16[m * e.ld_y16 + n] = __float2bfloat16_rn(v);
 }
 
+__device__ __forceinline__ void dense_put(const skn_epi &e, int64_t m, int64_t n, float v) {
+    if (e.y32) e.y32[m * e.ld_y32 + n] = v;
+    if (e.y16) e.y16[m * e.ld_y16 + n] = __float2bfloat16_rn(v);
+}
+// gate and up of an activation column
+__device__ __forceinline__ void dense_put_silu(const skn_epi &e, int64_t m, int64_t n, float gate, float up) {
+    float v = dense_silu(gate) * up;
+    if (e.act_scale) v *= e.act_scale[(n - e.n_act) / e.scale_rows];
+    const int64_t c = (n - e.n_act) >> 1;
+    if (e.act32) e.act32[m * e.ld_act32 + c] = v;
+    if (e.act16) e.act16[m * e.ld_act16 + c] = __float2bfloat16_rn(v);
+}
+// angle of the pair that row n belongs to; false: it passes unchanged
+__device__ __forceinline__ bool dense_angle(const skn_epi &e, int64_t m, int64_t n, float2 &cs) {
+    const int i = ((int)(n % e.rot_head) - e.rot_lo) >> 1;
+    if (i < 0 || i >= e.rot.half) return false;
+    cs = __ldcg(e.rot.table + m * e.rot.ld + i);
+    return true;
+}
+// weight rows n (even) and n + 1 of token m, for the epilogues that work on pairs
+template <int EPI>
+__device__ __forceinline__ void dense_store_pair(const skn_epi &e, int64_t m, int64_t n, float a, float b, bool both) {
+    if (EPI == SKN_EPI_SILU_TAIL && n >= e.n_act) {
+        if (both) dense_put_silu(e, m, n, a, b);
+        return;
+    }
+    float2 cs;
+    if (EPI == SKN_EPI_ROTATE && both && dense_angle(e, m, n, cs)) {
+        const float u = a;
+        a = u * cs.x - b * cs.y;
+        b = b * cs.x + u * cs.y;
+    }
+    dense_put(e, m, n, a);
+    if (both) dense_put(e, m, n + 1, b);
+}
+
 // NC consecutive tokens m .. of weight row n: everything the epilogue reads is loaded before the first store
 template <int EPI, int NC>
 __device__ __forceinline__ void dense_store_run(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count) {
@@ -38,7 +85,17 @@ __device__ __forceinline__ void dense_store_run(const skn_epi &e, int64_t m, int
 #pragma unroll
         for (int c = 0; c < NC; ++c) r[c] = c < count ? e.resid[(m + c) * e.ld_resid + n] : 0.f;
 #pragma unroll
-        for (int c = 0; c < NC; ++c) v[c] += r[c];
+        for (int c = 0; c < NC; ++c) v[c] = fmaf(e.alpha, v[c], r[c]);
+    }
+    if (EPI == SKN_EPI_GELU_TAIL && n >= e.n_act) {
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            if (c >= count) continue;
+            const float g = dense_gelu_exp(v[c]);
+            if (e.act32) e.act32[(m + c) * e.ld_act32 + n - e.n_act] = g;
+            if (e.act16) e.act16[(m + c) * e.ld_act16 + n - e.n_act] = __float2bfloat16_rn(g);
+        }
+        return;
     }
     if (EPI == SKN_EPI_GELU_TABLE) {
         float r[NC];
@@ -64,6 +121,59 @@ __device__ __forceinline__ void dense_store_run(const skn_epi &e, int64_t m, int
     }
 }
 
+// The same for the pair epilogues, the whole warp together: lane l holds row n = (even base) + l, `in` marks the rows that exist.
+template <int EPI, int NC>
+__device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count, bool in) {
+    const bool odd = n & 1;
+    const bool act = EPI == SKN_EPI_SILU_TAIL && n >= e.n_act;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        const float other = __shfl_xor_sync(0xffffffffu, v[c], 1);
+        if (c >= count || !in) continue;
+        if (act) {
+            if (!odd) dense_put_silu(e, m + c, n, v[c], other);
+            continue;
+        }
+        float2 cs;
+        if (EPI == SKN_EPI_ROTATE && dense_angle(e, m + c, n, cs)) v[c] = odd ? v[c] * cs.x + other * cs.y : v[c] * cs.x - other * cs.y;
+        dense_put(e, m + c, n, v[c]);
+    }
+}
+
+// experts as groups of rows: first tile of each in tiles of NT rows (start[E]: their number), by one warp
+__device__ __forceinline__ void dense_group_tiles(const int32_t *offset, int E, int NT, int *start, int *off) {
+    const int lane = threadIdx.x & 31;
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+        const int e = e0 + lane;
+        const int lo = e < E ? __ldcg(offset + e) : 0, hi = e < E ? __ldcg(offset + e + 1) : 0;
+        int t = (hi - lo + NT - 1) / NT;
+        const int own = t;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int y = __shfl_up_sync(0xffffffffu, t, o);
+            if (lane >= o) t += y;
+        }
+        if (e < E) {
+            start[e] = base + t - own;
+            off[e] = lo;
+            if (e == E - 1) off[E] = hi;
+        }
+        base += __shfl_sync(0xffffffffu, t, 31);
+    }
+    if (lane == 0) start[E] = base;
+}
+// expert of tile t
+__device__ __forceinline__ int dense_group_of(const int *start, int E, int t) {
+    int lo = 0, hi = E - 1;
+    while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (start[mid] <= t) lo = mid;
+        else hi = mid - 1;
+    }
+    return lo;
+}
+
 __device__ __forceinline__ float bf_lo(uint32_t w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 0xFFFF0000u); }
 
@@ -71,7 +181,8 @@ __device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 
 // CTA b owns the weight rows [b N / grid, (b + 1) N / grid): a producer warp streams them, a few rows per bulk copy, through
 // a ring of shared-memory stages and starts before the kernel waits for its predecessor; eight warps each take an eighth of
 // the columns of every row.  Their partial sums meet in shared memory, 128 rows at a time.  One activation row lives in
-// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).
+// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).  PICK: the weight rows, or pieces of
+// them, belong to experts that a kernel before chose, so the stream of those starts after the dependency wait.
 constexpr int MVD_WARPS = 8, MVD_THREADS = (MVD_WARPS + 1) * 32, MVD_ROWS = 128;
 constexpr int MVD_RING = 96 * 1024, MVD_MAX_STAGES = 24;
 // dynamic shared memory beside the partial sums of MR rows
@@ -86,6 +197,7 @@ __device__ __forceinline__ void dense_store_any(const skn_epi &e, int64_t m, int
     case SKN_EPI_ADD: dense_store<SKN_EPI_ADD>(e, m, n, v); break;
     case SKN_EPI_RELU2: dense_store<SKN_EPI_RELU2>(e, m, n, v); break;
     case SKN_EPI_GELU_TABLE: dense_store<SKN_EPI_GELU_TABLE>(e, m, n, v); break;
+    case SKN_EPI_GELU_TAIL: dense_store<SKN_EPI_GELU_TAIL>(e, m, n, v); break;
     default: dense_store<SKN_EPI_STORE>(e, m, n, v); break;
     }
 }
@@ -97,17 +209,33 @@ __device__ __forceinline__ float mvd_dot8(const uint4 &w, const float4 &lo, cons
 // row of the eight whose sum this lane holds after the joint reduction
 __device__ __forceinline__ int mvd_row(int lane) { return ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1); }
 
-template <int MR, int UU>
+struct mvd_pick {
+    const int32_t *expert;
+    const uint8_t *w2;                  // SKN_PICK_COLS
+    int64_t pitch1;                     // bytes of a row of w / of w2 (the joint row has `pitch` bytes)
+    int64_t pitch2;
+    int n, rows_per;
+};
+struct mvd_norm {
+    const float *gain;
+    float eps;
+    int cols, parts;                    // cols 0: the whole row
+};
+
+template <int MR, int UU, int PICK>
 __global__ void __launch_bounds__(MVD_THREADS, 2)
 skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int K, int m0, const float *x, int64_t ldx, const float *xb,
-                        int64_t ldxb, int ka, const float *__restrict__ gain, float eps, int stages, skn_epi e, int32_t *status) {
+                        int64_t ldxb, int ka, mvd_norm nm, mvd_pick pk, int stages, skn_epi e, int32_t *status) {
     extern __shared__ __align__(128) uint8_t ring[];
     constexpr int GR = mvd_stage_rows(MR, UU);
     __shared__ uint64_t full_bar[MVD_MAX_STAGES], empty_bar[MVD_MAX_STAGES];
-    __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS];
+    __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS], psum[MR][MVD_WARPS][SKN_NORM_PARTS];
+    const float *__restrict__ gain = nm.gain;
+    const bool pairs = skn_epi_pairs(e.kind), partial = gain && nm.cols > 0;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2, per = (nv + MVD_WARPS - 1) / MVD_WARPS;
-    const int r0 = (int)((int64_t)N * blockIdx.x / gridDim.x), r1 = (int)((int64_t)N * (blockIdx.x + 1) / gridDim.x);
+    const int q_rows = pairs ? 2 : 1, nq = (N + q_rows - 1) / q_rows;     // pairs of rows stay together
+    const int r0 = min(N, q_rows * (int)((int64_t)nq * blockIdx.x / gridDim.x)), r1 = min(N, q_rows * (int)((int64_t)nq * (blockIdx.x + 1) / gridDim.x));
     const int steps = (r1 - r0 + GR - 1) / GR;
     const size_t stage_bytes = (size_t)GR * pitch;
     if (threadIdx.x == 0) {
@@ -122,15 +250,44 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
         if (lane == 0) {
             int s = 0;
             uint32_t phase = 1;
+            int early = 0;
+            if constexpr (PICK == SKN_PICK_COLS) {
+                // the first stages' own pieces depend on no kernel before this one
+                for (; early < stages && early < steps; ++early) {
+                    const int row = r0 + early * GR, n = min(GR, r1 - row);
+                    skn_mbar_expect_tx(&full_bar[early], (uint32_t)(n * pitch));
+                    for (int j = 0; j < n; ++j)
+                        skn_bulk_g2s(ring + early * stage_bytes + j * pitch, W + (int64_t)(row + j) * pk.pitch1, (uint32_t)pk.pitch1, &full_bar[early]);
+                }
+            }
+            if constexpr (PICK != SKN_PICK_NONE) skn_pdl_wait();
             for (int i = 0; i < steps; ++i) {
                 const int row = r0 + i * GR;
-                if (!skn_mbar_wait(&empty_bar[s], phase)) {
+                if (i >= early && !skn_mbar_wait(&empty_bar[s], phase)) {
                     atomicExch(status, SKN_ERR_TIMEOUT);
                     break;
                 }
-                const uint32_t bytes = (uint32_t)(min(GR, r1 - row) * pitch);
-                skn_mbar_expect_tx(&full_bar[s], bytes);
-                skn_bulk_g2s(ring + s * stage_bytes, W + (int64_t)row * pitch, bytes, &full_bar[s]);
+                const int n = min(GR, r1 - row);
+                const uint32_t bytes = (uint32_t)(n * pitch);
+                if (i >= early) skn_mbar_expect_tx(&full_bar[s], bytes);
+                uint8_t *dst = ring + s * stage_bytes;
+                if constexpr (PICK == SKN_PICK_NONE) {
+                    skn_bulk_g2s(dst, W + (int64_t)row * pitch, bytes, &full_bar[s]);
+                } else if constexpr (PICK == SKN_PICK_ROWS) {
+                    for (int j = 0; j < n; ++j) {
+                        const int r = row + j, x = r / pk.rows_per;
+                        skn_bulk_g2s(dst + j * pitch, W + ((int64_t)__ldcg(pk.expert + x) * pk.rows_per + r - x * pk.rows_per) * pitch, (uint32_t)pitch, &full_bar[s]);
+                    }
+                } else {
+                    for (int j = 0; j < n; ++j) {
+                        const int r = row + j;
+                        uint8_t *d = dst + j * pitch;
+                        if (i >= early) skn_bulk_g2s(d, W + (int64_t)r * pk.pitch1, (uint32_t)pk.pitch1, &full_bar[s]);
+                        d += pk.pitch1;
+                        for (int x = 0; x < pk.n; ++x, d += pk.pitch2)
+                            skn_bulk_g2s(d, pk.w2 + ((int64_t)__ldcg(pk.expert + x) * N + r) * pk.pitch2, (uint32_t)pk.pitch2, &full_bar[s]);
+                    }
+                }
                 if (++s == stages) {
                     s = 0;
                     phase ^= 1u;
@@ -155,10 +312,11 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
     if constexpr (UU > 0) {
         // rows that are whole aligned vectors (the usual case) are read 16 bytes at a time
         const bool vec = K % 8 == 0 && ka % 8 == 0 && ldx % 4 == 0 && ldxb % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xb)) & 15) == 0;
-        float q = 0.f;
+        float q = 0.f, vsq[UU];
 #pragma unroll
         for (int u = 0; u < UU; ++u) {
             const int i = v0 + u * 32 + lane;
+            vsq[u] = 0.f;
             float f[8];
             const int k = i * 8;
             if (vec && i < v1) {
@@ -170,8 +328,9 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
                 for (int j = 0; j < 8; ++j) f[j] = i < v1 ? fetch(0, k + j) : 0.f;
             }
 #pragma unroll
-            for (int j = 0; j < 8; ++j) q = fmaf(f[j], f[j], q);
-            if (gain && i < v1) {
+            for (int j = 0; j < 8; ++j) vsq[u] = fmaf(f[j], f[j], vsq[u]);
+            q += vsq[u];
+            if (gain && i < v1 && (!partial || k < nm.cols)) {
                 if (vec) {
                     const float4 g0 = __ldg(reinterpret_cast<const float4 *>(gain + k)), g1 = __ldg(reinterpret_cast<const float4 *>(gain + k + 4));
                     f[0] *= g0.x; f[1] *= g0.y; f[2] *= g0.z; f[3] *= g0.w;
@@ -186,6 +345,20 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
             xr[2 * u + 1] = make_float4(f[4], f[5], f[6], f[7]);
         }
         ss[0] = q;
+        if (partial) {
+            const int pv = nm.cols / nm.parts / 8;                     // vectors of a part
+            for (int p = 0; p < nm.parts; ++p) {
+                float t = 0.f;
+#pragma unroll
+                for (int u = 0; u < UU; ++u) {
+                    const int i = v0 + u * 32 + lane;
+                    if (i < v1 && i / pv == p) t += vsq[u];
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+                if (lane == 0) psum[0][warp][p] = t;
+            }
+        }
     } else {
 #pragma unroll
         for (int m = 0; m < MR; ++m) {
@@ -193,9 +366,25 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
             for (int k = threadIdx.x; k < K8; k += MVD_WARPS * 32) {
                 float v = fetch(m, k);
                 ss[m] = fmaf(v, v, ss[m]);
-                if (gain && k < K) v *= __ldg(gain + k);
+                if (gain && k < K && !partial) v *= __ldg(gain + k);
                 xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] = v;
             }
+        }
+        if (partial) {
+            const int pc = nm.cols / nm.parts;
+            mvd_barrier();
+#pragma unroll
+            for (int m = 0; m < MR; ++m)
+                for (int p = 0; p < nm.parts; ++p) {
+                    float t = 0.f;
+                    for (int k = p * pc + threadIdx.x; k < (p + 1) * pc; k += MVD_WARPS * 32) {
+                        const float v = xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)];
+                        t = fmaf(v, v, t);
+                    }
+#pragma unroll
+                    for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+                    if (lane == 0) psum[m][warp][p] = t;
+                }
         }
     }
 #pragma unroll
@@ -209,11 +398,40 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
 #pragma unroll
     for (int m = 0; m < MR; ++m) {
         rs[m] = 1.f;
-        if (gain) {
+        if (gain && !partial) {
             float t = 0.f;
 #pragma unroll
             for (int w = 0; w < MVD_WARPS; ++w) t += red[w][m];
-            rs[m] = 1.f / sqrtf(t / (float)K + eps);
+            rs[m] = 1.f / sqrtf(t / (float)K + nm.eps);
+        }
+    }
+    if (partial) {
+        const int pc = nm.cols / nm.parts;
+        auto scale = [&](int m, int p) {
+            float t = 0.f;
+#pragma unroll
+            for (int w = 0; w < MVD_WARPS; ++w) t += psum[m][w][p];
+            return 1.f / sqrtf(t / (float)pc + nm.eps);
+        };
+        if constexpr (UU > 0) {
+#pragma unroll
+            for (int u = 0; u < UU; ++u) {
+                const int k = (v0 + u * 32 + lane) * 8;
+                if (k < nm.cols) {
+                    const float f = scale(0, k / pc);
+                    xr[2 * u].x *= f; xr[2 * u].y *= f; xr[2 * u].z *= f; xr[2 * u].w *= f;
+                    xr[2 * u + 1].x *= f; xr[2 * u + 1].y *= f; xr[2 * u + 1].z *= f; xr[2 * u + 1].w *= f;
+                }
+            }
+        } else {
+#pragma unroll
+            for (int m = 0; m < MR; ++m)
+                for (int p = 0; p < nm.parts; ++p) {
+                    const float f = scale(m, p);
+                    for (int k = p * pc + threadIdx.x; k < (p + 1) * pc; k += MVD_WARPS * 32)
+                        xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] *= f * __ldg(gain + k);
+                }
+            mvd_barrier();
         }
     }
 
@@ -297,12 +515,24 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
         filled += rows;
         if (filled + 8 > MVD_ROWS || g0 + 8 >= r1 - r0) {
             mvd_barrier();
-            for (int j = threadIdx.x; j < filled * MR; j += MVD_WARPS * 32) {
-                const int m = j / filled, r = j % filled;
+            auto total = [&](int m, int r) {
                 float t = 0.f;
 #pragma unroll
                 for (int w8 = 0; w8 < MVD_WARPS; ++w8) t += part[buf][m][w8][r];
-                dense_store_any(e, m0 + m, base + r, t);
+                return t;
+            };
+            if (pairs) {
+                const int np = (filled + 1) / 2;
+                for (int j = threadIdx.x; j < np * MR; j += MVD_WARPS * 32) {
+                    const int m = j / np, r = j % np * 2;
+                    const bool both = r + 1 < filled;
+                    const float a = total(m, r), b = both ? total(m, r + 1) : 0.f;
+                    if (e.kind == SKN_EPI_ROTATE) dense_store_pair<SKN_EPI_ROTATE>(e, m0 + m, base + r, a, b, both);
+                    else dense_store_pair<SKN_EPI_SILU_TAIL>(e, m0 + m, base + r, a, b, both);
+                }
+            } else for (int j = threadIdx.x; j < filled * MR; j += MVD_WARPS * 32) {
+                const int m = j / filled, r = j % filled;
+                dense_store_any(e, m0 + m, base + r, total(m, r));
             }
             base += filled;
             filled = 0;
@@ -311,47 +541,69 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
     }
 }
 
-template <int MR, int UU>
+// bytes of the joint weight row
+static int64_t mvd_pitch(const skn_linear &l) { return l.pick.kind == SKN_PICK_COLS ? l.w->pitch + l.pick.n * l.pick.w2->pitch : l.w->pitch; }
+
+template <int MR, int UU, int PICK>
 static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int m0, cudaStream_t st) {
-    auto kern = skn_dense_matvec_kernel<MR, UU>;
+    auto kern = skn_dense_matvec_kernel<MR, UU, PICK>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, mvd_smem(MR));
         if (e != cudaSuccess) return e;
         attr_done[ctx->device & 63] = true;
     }
-    const int64_t pitch = l.w->pitch;
-    const int N = (int)l.w->n_rows, K = (int)l.w->n_cols, rows = mvd_stage_rows(MR, UU);
+    const int64_t pitch = mvd_pitch(l);
+    const int N = PICK == SKN_PICK_ROWS ? l.pick.n * l.pick.rows_per : (int)l.w->n_rows, K = (int)skn_linear_cols(l), rows = mvd_stage_rows(MR, UU);
     const size_t xbytes = UU > 0 ? 0 : (size_t)MR * pitch * 2;
     size_t room = mvd_smem(MR) - xbytes;
     if (room > (size_t)MVD_RING) room = MVD_RING;
     int stages = (int)(room / (rows * pitch));
     if (stages < 1) return cudaErrorNotSupported;
     if (stages > MVD_MAX_STAGES) stages = MVD_MAX_STAGES;
-    const int grid = N < ctx->sm_count ? N : ctx->sm_count;
+    const int units = skn_epi_pairs(l.epi.kind) ? (N + 1) / 2 : N;
+    const int grid = units < ctx->sm_count ? units : ctx->sm_count;
+    const mvd_norm nm = {l.gain, l.eps, l.gain ? l.norm_cols : 0, l.norm_parts > 0 ? l.norm_parts : 1};
+    const mvd_pick pk = {l.pick.expert, PICK == SKN_PICK_COLS ? (const uint8_t *)l.pick.w2->d_blocks : nullptr, l.w->pitch,
+                         PICK == SKN_PICK_COLS ? l.pick.w2->pitch : 0, l.pick.n, l.pick.rows_per};
     return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks, pitch,
-                          N, K, m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, l.gain, l.eps, stages, l.epi, ctx->d_status);
+                          N, K, m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, nm, pk, stages, l.epi, ctx->d_status);
+}
+
+template <int PICK>
+static cudaError_t launch_mvd_pick(skn_ctx *ctx, const skn_linear &l, int uu, cudaStream_t st) {
+    if (l.M != 1) return cudaErrorInvalidValue;
+    switch (uu) {
+    case 1: return launch_mvd<1, 1, PICK>(ctx, l, 0, st);
+    case 2: return launch_mvd<1, 2, PICK>(ctx, l, 0, st);
+    case 3: case 4: return launch_mvd<1, 4, PICK>(ctx, l, 0, st);
+    default: return launch_mvd<1, 0, PICK>(ctx, l, 0, st);
+    }
 }
 
 cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStream_t st) {
-    const int64_t pitch = l.w->pitch;
+    const int64_t pitch = mvd_pitch(l);
     if (pitch * 3 > mvd_smem(1)) return cudaErrorNotSupported;       // one stage and one activation row must fit
+    if (l.gain && l.norm_cols > 0 && !skn_norm_folds(l.norm_cols, l.norm_parts)) return cudaErrorInvalidValue;
     const int uu = (int)(((pitch / 16 + MVD_WARPS - 1) / MVD_WARPS + 31) / 32);
+    if (l.pick.kind == SKN_PICK_ROWS) return launch_mvd_pick<SKN_PICK_ROWS>(ctx, l, uu, st);
+    if (l.pick.kind == SKN_PICK_COLS) return launch_mvd_pick<SKN_PICK_COLS>(ctx, l, uu, st);
+    constexpr int P = SKN_PICK_NONE;
     for (int m0 = 0; m0 < l.M;) {
         const int left = l.M - m0;
         cudaError_t e;
         int mr = 1;
-        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0>(ctx, l, m0, st); }
-        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0>(ctx, l, m0, st); }
+        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0, P>(ctx, l, m0, st); }
+        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0, P>(ctx, l, m0, st); }
         else switch (uu) {
-            case 1: e = launch_mvd<1, 1>(ctx, l, m0, st); break;
-            case 2: e = launch_mvd<1, 2>(ctx, l, m0, st); break;
-            case 3: e = launch_mvd<1, 3>(ctx, l, m0, st); break;
-            case 4: e = launch_mvd<1, 4>(ctx, l, m0, st); break;
-            case 5: e = launch_mvd<1, 5>(ctx, l, m0, st); break;
-            case 6: e = launch_mvd<1, 6>(ctx, l, m0, st); break;
-            case 7: e = launch_mvd<1, 7>(ctx, l, m0, st); break;
-            default: e = launch_mvd<1, 0>(ctx, l, m0, st); break;
+            case 1: e = launch_mvd<1, 1, P>(ctx, l, m0, st); break;
+            case 2: e = launch_mvd<1, 2, P>(ctx, l, m0, st); break;
+            case 3: e = launch_mvd<1, 3, P>(ctx, l, m0, st); break;
+            case 4: e = launch_mvd<1, 4, P>(ctx, l, m0, st); break;
+            case 5: e = launch_mvd<1, 5, P>(ctx, l, m0, st); break;
+            case 6: e = launch_mvd<1, 6, P>(ctx, l, m0, st); break;
+            case 7: e = launch_mvd<1, 7, P>(ctx, l, m0, st); break;
+            default: e = launch_mvd<1, 0, P>(ctx, l, m0, st); break;
         }
         if (e != cudaSuccess) return e;
         m0 += mr;
@@ -363,15 +615,26 @@ cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStrea
 // 64 tokens x 64 weight rows per CTA, K in steps of 16; a thread owns 4 x 4 outputs
 constexpr int F32_BM = 64, F32_BN = 64, F32_BK = 16;
 
-template <int EPI>
+template <int EPI, bool GROUPS>
 __global__ void __launch_bounds__(256)
 skn_dense_f32_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int K, int M, const float *__restrict__ x, int64_t ldx,
-                     const float *__restrict__ xb, int64_t ldxb, int ka, skn_epi e) {
+                     const float *__restrict__ xb, int64_t ldxb, int ka, const int32_t *offset, int E, skn_epi e) {
     __shared__ float xt[F32_BK][F32_BM + 4], wt[F32_BK][F32_BN + 4];
-    const int m0 = blockIdx.y * F32_BM, n0 = blockIdx.x * F32_BN;
+    __shared__ int start[GROUPS ? SKN_MAX_EXPERTS + 1 : 1], off[GROUPS ? SKN_MAX_EXPERTS + 1 : 1];
+    const int n0 = blockIdx.x * F32_BN;
+    int m0 = blockIdx.y * F32_BM;
     const int tm = (threadIdx.x >> 4) * 4, tn = (threadIdx.x & 15) * 4;
     skn_pdl_launch_dependents();
     skn_pdl_wait();
+    if (GROUPS) {
+        if (threadIdx.x < 32) dense_group_tiles(offset, E, F32_BM, start, off);
+        __syncthreads();
+        if ((int)blockIdx.y >= start[E]) return;
+        const int g = dense_group_of(start, E, blockIdx.y);
+        m0 = off[g] + ((int)blockIdx.y - start[g]) * F32_BM;
+        M = off[g + 1];
+        W += (int64_t)g * N * pitch;
+    }
     float acc[4][4] = {};
     for (int k0 = 0; k0 < K; k0 += F32_BK) {
 #pragma unroll
@@ -400,25 +663,42 @@ skn_dense_f32_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int K,
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            if (m0 + tm + i < M && n0 + tn + j < N) dense_store<EPI>(e, m0 + tm + i, n0 + tn + j, acc[i][j]);
+        for (int j = 0; j < 4; j += skn_epi_pairs(EPI) ? 2 : 1) {
+            if (m0 + tm + i >= M || n0 + tn + j >= N) continue;
+            if constexpr (skn_epi_pairs(EPI)) dense_store_pair<EPI>(e, m0 + tm + i, n0 + tn + j, acc[i][j], acc[i][j + 1], n0 + tn + j + 1 < N);
+            else dense_store<EPI>(e, m0 + tm + i, n0 + tn + j, acc[i][j]);
+        }
+}
+
+// most tiles of T rows that M rows in E groups can need
+static int group_tiles_bound(int M, int E, int T) { return (M + T - 1) / T + (E < M ? E : M); }
+
+template <int EPI>
+static cudaError_t launch_f32(const skn_linear &l, cudaStream_t st) {
+    const bool groups = l.pick.kind == SKN_PICK_GROUPS;
+    const int N = groups ? l.pick.rows_per : (int)l.w->n_rows, K = (int)l.w->n_cols;
+    const dim3 grid((N + F32_BN - 1) / F32_BN, groups ? group_tiles_bound(l.M, l.pick.n, F32_BM) : (l.M + F32_BM - 1) / F32_BM);
+    const int ka = l.x32b ? (int)l.k_a : K;
+    if constexpr (EPI == SKN_EPI_STORE || EPI == SKN_EPI_SILU_TAIL)
+        if (groups)
+            return skn_launch_pdl(skn_dense_f32_kernel<EPI, true>, grid, dim3(256), 0, st, 1, (const uint8_t *)l.w->d_blocks, l.w->pitch, N, K, l.M,
+                                  l.x32, l.ld_x32, l.x32b, l.ld_x32b, ka, l.pick.offset, l.pick.n, l.epi);
+    if (groups) return cudaErrorInvalidValue;
+    return skn_launch_pdl(skn_dense_f32_kernel<EPI, false>, grid, dim3(256), 0, st, 1, (const uint8_t *)l.w->d_blocks, l.w->pitch, N, K, l.M,
+                          l.x32, l.ld_x32, l.x32b, l.ld_x32b, ka, (const int32_t *)nullptr, 0, l.epi);
 }
 
 cudaError_t skn_launch_dense_f32(skn_ctx *, const skn_linear &l, cudaStream_t st) {
-    const int N = (int)l.w->n_rows, K = (int)l.w->n_cols;
-    const dim3 grid((N + F32_BN - 1) / F32_BN, (l.M + F32_BM - 1) / F32_BM);
-    const int ka = l.x32b ? (int)l.k_a : K;
-#define F32_CASE(EPI) \
-    case EPI: \
-        return skn_launch_pdl(skn_dense_f32_kernel<EPI>, grid, dim3(256), 0, st, 1, (const uint8_t *)l.w->d_blocks, l.w->pitch, N, K, l.M, \
-                              l.x32, l.ld_x32, l.x32b, l.ld_x32b, ka, l.epi)
+    if (l.M == 0) return cudaSuccess;
     switch (l.epi.kind) {
-        F32_CASE(SKN_EPI_STORE);
-        F32_CASE(SKN_EPI_ADD);
-        F32_CASE(SKN_EPI_RELU2);
-        F32_CASE(SKN_EPI_GELU_TABLE);
+    case SKN_EPI_STORE: return launch_f32<SKN_EPI_STORE>(l, st);
+    case SKN_EPI_ADD: return launch_f32<SKN_EPI_ADD>(l, st);
+    case SKN_EPI_RELU2: return launch_f32<SKN_EPI_RELU2>(l, st);
+    case SKN_EPI_GELU_TABLE: return launch_f32<SKN_EPI_GELU_TABLE>(l, st);
+    case SKN_EPI_GELU_TAIL: return launch_f32<SKN_EPI_GELU_TAIL>(l, st);
+    case SKN_EPI_SILU_TAIL: return launch_f32<SKN_EPI_SILU_TAIL>(l, st);
+    case SKN_EPI_ROTATE: return launch_f32<SKN_EPI_ROTATE>(l, st);
     }
-#undef F32_CASE
     return cudaErrorInvalidValue;
 }
 
@@ -431,23 +711,43 @@ constexpr int DTC_MAX_STAGES = 8;
 
 __device__ __forceinline__ void dtc_barrier_epilogue() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-template <int EPI>
+struct dtc_tile {
+    int m0, cols, sp, n0, w0;           // first token and tokens of the tile, K split, first row of the output, and of the weight
+};
+
+template <int EPI, bool GROUPS>
 __global__ void __launch_bounds__(DTC_THREADS, 1)
 skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, int N, int K, int M, int NT,
-                    int stages, int splits, float *__restrict__ partial, unsigned *__restrict__ tickets, skn_epi e,
+                    int stages, int splits, float *__restrict__ partial, unsigned *__restrict__ tickets, const int32_t *offset, int E, skn_epi e,
                     int32_t *__restrict__ status) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ uint64_t full_bar[DTC_MAX_STAGES], empty_bar[DTC_MAX_STAGES], acc_full[2], acc_empty[2];
     __shared__ uint32_t tmem_slot, last_flag;
+    __shared__ int start[GROUPS ? SKN_MAX_EXPERTS + 1 : 1], off[GROUPS ? SKN_MAX_EXPERTS + 1 : 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int stage_bytes = DTC_A_BYTES + NT * DTC_BK * 2;
     const int acc_cols = NT < 32 ? 32 : NT;
     uint32_t tmem_cols = 32;
     while ((int)tmem_cols < 2 * acc_cols) tmem_cols *= 2;
     const int ksteps = (K + DTC_BK - 1) / DTC_BK;
-    const int mt = (M + NT - 1) / NT, nt = (N + DTC_BM - 1) / DTC_BM;
-    const int units = mt * nt * splits;          // token tiles fastest, then splits, then weight tiles
+    const int nt = (N + DTC_BM - 1) / DTC_BM;
+    int mt = (M + NT - 1) / NT, units = mt * nt * splits;      // token tiles fastest, then splits, then weight tiles
+    auto tile_of = [&](int u) {
+        dtc_tile t;
+        t.sp = GROUPS ? 0 : (u / mt) % splits;
+        t.n0 = (u / mt / splits) * DTC_BM;
+        t.w0 = t.n0;
+        t.m0 = (u % mt) * NT;
+        t.cols = min(NT, M - t.m0);
+        if (GROUPS) {
+            const int g = dense_group_of(start, E, u % mt);
+            t.m0 = off[g] + (u % mt - start[g]) * NT;
+            t.cols = min(NT, off[g + 1] - t.m0);
+            t.w0 += g * N;
+        }
+        return t;
+    };
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < stages; ++s) {
@@ -467,7 +767,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     const uint32_t tmem = tmem_slot;
     // the weights depend on no kernel before this one: the first unit's first stages are requested ahead of the wait
     int early = 0;
-    if (warp == 5 && lane == 0 && (int)blockIdx.x < units) {
+    if (!GROUPS && warp == 5 && lane == 0 && (int)blockIdx.x < units) {
         const int sp = (blockIdx.x / mt) % splits, n0 = (blockIdx.x / mt / splits) * DTC_BM;
         const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
         for (; early < stages && early < ke - kb; ++early) {
@@ -476,13 +776,20 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
         }
     }
     skn_pdl_wait();
+    if (GROUPS) {
+        if (warp == 0) dense_group_tiles(offset, E, NT, start, off);
+        __syncthreads();
+        mt = start[E];
+        units = mt * nt;
+    }
 
     if (warp == 5) {
         if (lane == 0) {
             bool ok = true;
             int it = 0;
             for (int u = blockIdx.x; u < units && ok; u += gridDim.x) {
-                const int m0 = (u % mt) * NT, sp = (u / mt) % splits, n0 = (u / mt / splits) * DTC_BM;
+                const dtc_tile tl = tile_of(u);
+                const int m0 = tl.m0, sp = tl.sp, n0 = tl.w0;
                 const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
                 for (int k = kb; k < ke; ++k, ++it) {
                     const int s = it % stages;
@@ -513,7 +820,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
             bool ok = true;
             int it = 0, tile = 0;
             for (int u = blockIdx.x; u < units && ok; u += gridDim.x, ++tile) {
-                const int sp = (u / mt) % splits;
+                const int sp = GROUPS ? 0 : (u / mt) % splits;
                 const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
                 const int b = tile & 1;
                 if (!skn_mbar_wait(&acc_empty[b], ((uint32_t)(tile >> 1) & 1u) ^ 1u)) {
@@ -544,7 +851,8 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
         bool ok = true;
         int tile = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, ++tile) {
-            const int m0 = (u % mt) * NT, sp = (u / mt) % splits, nti = u / mt / splits, n0 = nti * DTC_BM;
+            const dtc_tile tl = tile_of(u);
+            const int m0 = tl.m0, sp = tl.sp, nti = u / mt / splits, n0 = tl.n0;
             const int b = tile & 1;
             if (ok && !skn_mbar_wait(&acc_full[b], (uint32_t)(tile >> 1) & 1u)) {
                 if (lane == 0) atomicExch(status, SKN_ERR_TIMEOUT);
@@ -552,7 +860,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
             }
             tc_fence_after();
             const int n = n0 + warp * 32 + lane;
-            const int cols = min(NT, M - m0);
+            const int cols = tl.cols;
             const uint32_t src = tmem + (uint32_t)(b * acc_cols) + ((uint32_t)(warp * 32) << 16);
             const int tidx = nti * mt + u % mt;
             float *pbase = partial + ((size_t)tidx * splits) * NT * DTC_BM + warp * 32 + lane;
@@ -561,7 +869,12 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 uint32_t acc[32];
                 tc_ld32(src + c0, acc);
                 if (splits == 1) {
-                    if (n < N && ok) {
+                    if constexpr (skn_epi_pairs(EPI)) {
+                        float v[32];
+#pragma unroll
+                        for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
+                        dense_store_run_pairs<EPI, 32>(e, m0 + c0, n, v, cols - c0, n < N && ok);
+                    } else if (n < N && ok) {
                         float v[32];
 #pragma unroll
                         for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
@@ -592,7 +905,8 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                         for (int s = 0; s < splits; ++s)
 #pragma unroll
                             for (int c = 0; c < 16; ++c) v[c] += __ldcg(pbase + ((size_t)s * NT + c0 + c) * DTC_BM);
-                        if (n < N && ok) dense_store_run<EPI, 16>(e, m0 + c0, n, v, cols - c0);
+                        if constexpr (skn_epi_pairs(EPI)) dense_store_run_pairs<EPI, 16>(e, m0 + c0, n, v, cols - c0, n < N && ok);
+                        else if (n < N && ok) dense_store_run<EPI, 16>(e, m0 + c0, n, v, cols - c0);
                     }
                     if (threadIdx.x == 0) tickets[tidx] = 0;
                 }
@@ -609,22 +923,25 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     }
 }
 
-template <int EPI>
+template <int EPI, bool GROUPS>
 static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense_ws &ws, cudaStream_t st) {
-    auto kern = skn_dense_tc_kernel<EPI>;
+    auto kern = skn_dense_tc_kernel<EPI, GROUPS>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM + 1024);
         if (e != cudaSuccess) return e;
         attr_done[ctx->device & 63] = true;
     }
-    const int N = (int)l.w->n_rows, K = (int)l.w->n_cols, M = l.M, sms = ctx->sm_count;
+    const int N = GROUPS ? l.pick.rows_per : (int)l.w->n_rows, K = (int)l.w->n_cols, M = l.M, sms = ctx->sm_count;
     const int nt = (N + DTC_BM - 1) / DTC_BM;
     const int ksteps = (K + DTC_BK - 1) / DTC_BK;
     // token tile: the narrowest that covers M; beyond that, of the widths whose operands the shared memory feeds at full
     // rate, the one with the least time in waves (a wave of narrower tiles costs less, but loads more per product)
     int NT = 16;
-    if (M <= 128) {
+    if (GROUPS) {
+        // tiles that an expert's share of the rows fills about once
+        while (NT < 128 && NT * l.pick.n < M + M / 4) NT *= 2;
+    } else if (M <= 128) {
         while (NT < M) NT *= 2;
     } else {
         const int width[3] = {256, 192, 128};
@@ -639,11 +956,11 @@ static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense
             }
         }
     }
-    while (NT > 32 && nt * ((M + NT - 1) / NT) * 2 <= sms) NT = NT == 192 ? 128 : NT / 2;
-    const int mt = (M + NT - 1) / NT;
+    while (!GROUPS && NT > 32 && nt * ((M + NT - 1) / NT) * 2 <= sms) NT = NT == 192 ? 128 : NT / 2;
+    const int mt = GROUPS ? group_tiles_bound(M, l.pick.n, NT) : (M + NT - 1) / NT;
     // K splits that even out the load of the SMs (the tiles of a decode-size step are fewer than the SMs, or not many more)
     int splits = 1;
-    if (mt * nt < 2 * sms && mt * nt <= SKN_DENSE_MAX_TILES) {
+    if (!GROUPS && mt * nt < 2 * sms && mt * nt <= SKN_DENSE_MAX_TILES) {
         double best = 1e30;
         for (int s = 1; s <= 16 && (s == 1 || s <= ksteps / 4); ++s) {
             if (s > 1 && (size_t)mt * nt * s * NT * DTC_BM > SKN_DENSE_WS_FLOATS) break;
@@ -661,21 +978,30 @@ static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense
     int stages = (NT <= 64 ? DTC_SMEM / 2 : DTC_SMEM) / stage_bytes;
     if (stages > DTC_MAX_STAGES) stages = DTC_MAX_STAGES;
     CUtensorMap tw, tx;
-    cudaError_t e = skn_tmap_bf16(l.w->d_blocks, N, K, l.w->pitch, DTC_BM, &tw);
+    cudaError_t e = skn_tmap_bf16(l.w->d_blocks, l.w->n_rows, K, l.w->pitch, DTC_BM, &tw);
     if (e == cudaSuccess) e = skn_tmap_bf16(l.x16, M, K, l.ld_x16 * 2, NT, &tx);
     if (e != cudaSuccess) return e;
     const int units = mt * nt * splits;
     return skn_launch_pdl(kern, dim3(units < sms ? units : sms), dim3(DTC_THREADS), (size_t)stages * stage_bytes + 1024, st, 1, tw, tx, N, K, M, NT,
-                          stages, splits, ws.partial, ws.tickets, l.epi, ctx->d_status);
+                          stages, splits, ws.partial, ws.tickets, l.pick.offset, l.pick.n, l.epi, ctx->d_status);
 }
 
 cudaError_t skn_launch_dense_tc(skn_ctx *ctx, const skn_linear &l, const skn_dense_ws &ws, cudaStream_t st) {
     if (l.ld_x16 % 8) return cudaErrorInvalidValue;
+    if (l.M == 0) return cudaSuccess;
+    if (l.pick.kind == SKN_PICK_GROUPS) {
+        if (l.epi.kind == SKN_EPI_STORE) return launch_dtc<SKN_EPI_STORE, true>(ctx, l, ws, st);
+        if (l.epi.kind == SKN_EPI_SILU_TAIL) return launch_dtc<SKN_EPI_SILU_TAIL, true>(ctx, l, ws, st);
+        return cudaErrorInvalidValue;
+    }
     switch (l.epi.kind) {
-    case SKN_EPI_STORE: return launch_dtc<SKN_EPI_STORE>(ctx, l, ws, st);
-    case SKN_EPI_ADD: return launch_dtc<SKN_EPI_ADD>(ctx, l, ws, st);
-    case SKN_EPI_RELU2: return launch_dtc<SKN_EPI_RELU2>(ctx, l, ws, st);
-    case SKN_EPI_GELU_TABLE: return launch_dtc<SKN_EPI_GELU_TABLE>(ctx, l, ws, st);
+    case SKN_EPI_STORE: return launch_dtc<SKN_EPI_STORE, false>(ctx, l, ws, st);
+    case SKN_EPI_ADD: return launch_dtc<SKN_EPI_ADD, false>(ctx, l, ws, st);
+    case SKN_EPI_RELU2: return launch_dtc<SKN_EPI_RELU2, false>(ctx, l, ws, st);
+    case SKN_EPI_GELU_TABLE: return launch_dtc<SKN_EPI_GELU_TABLE, false>(ctx, l, ws, st);
+    case SKN_EPI_GELU_TAIL: return launch_dtc<SKN_EPI_GELU_TAIL, false>(ctx, l, ws, st);
+    case SKN_EPI_SILU_TAIL: return launch_dtc<SKN_EPI_SILU_TAIL, false>(ctx, l, ws, st);
+    case SKN_EPI_ROTATE: return launch_dtc<SKN_EPI_ROTATE, false>(ctx, l, ws, st);
     }
     return cudaErrorInvalidValue;
 }

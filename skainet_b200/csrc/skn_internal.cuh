@@ -136,6 +136,7 @@ struct skn_kvcache {
     // are k_pitch / v_pitch elements apart, and the owner keeps the lengths (d_len counts nothing)
     bool by_position;
     int32_t v_dim, k_pitch, v_pitch;
+    int32_t v_stride;            // elements between the rows of V (its pitch, or that of K where values are the start of a key row)
     void *d_k, *d_v;
     int32_t *d_len, *d_start;
     unsigned *d_tickets;         // [batch][n_kv_heads], zero between launches: split-attention merge tickets

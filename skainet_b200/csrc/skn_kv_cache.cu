@@ -30,7 +30,7 @@ int32_t skn_kv_create_typed(skn_ctx *ctx, int32_t batch, int32_t n_kv_heads, int
     kv->ctx = ctx;
     kv->batch = batch; kv->n_kv_heads = n_kv_heads; kv->head_dim = head_dim; kv->capacity = capacity;
     kv->dtype = kv_dtype;
-    kv->v_dim = kv->k_pitch = kv->v_pitch = head_dim;
+    kv->v_dim = kv->k_pitch = kv->v_pitch = kv->v_stride = head_dim;
     // Q8_0: an int8 plane, then the fp16 scales of its 32-dim blocks
     const size_t elems = (size_t)batch * n_kv_heads * capacity * head_dim;
     const size_t n = kv_dtype == SKN_KV_Q8_0 ? elems + elems / 32 * 2 : elems * (kv_dtype == SKN_KV_F16 ? 2 : sizeof(float));
@@ -88,10 +88,10 @@ int32_t skn_kv_create_by_position(skn_ctx *ctx, int32_t batch, int32_t n_kv_head
     *out = nullptr;
     if (kv_dtype != SKN_KV_F32 && kv_dtype != SKN_KV_BF16)
         return skn_fail(ctx, SKN_ERR_TYPE, "a position-addressed cache holds fp32 or bf16, not element type %d", kv_dtype);
-    if (batch < 1 || n_kv_heads < 1 || capacity < 1 || k_dim < 1 || v_dim < 1)
+    if (batch < 1 || n_kv_heads < 1 || capacity < 1 || k_dim < 1 || v_dim < 0)
         return skn_fail(ctx, SKN_ERR_ARG, "batch, heads, widths and capacity must be positive");
-    if (k_dim > SKN_ATTN_MAX_DIM || v_dim > SKN_ATTN_MAX_DIM)
-        return skn_fail(ctx, SKN_ERR_SHAPE, "head widths of %d and %d are above %d", k_dim, v_dim, SKN_ATTN_MAX_DIM);
+    if (k_dim > SKN_KV_MAX_DIM || v_dim > SKN_KV_MAX_DIM)
+        return skn_fail(ctx, SKN_ERR_SHAPE, "head widths of %d and %d are above %d", k_dim, v_dim, SKN_KV_MAX_DIM);
     skn_kvcache *kv = new (std::nothrow) skn_kvcache();
     if (!kv) return skn_fail(ctx, SKN_ERR_OOM, "host allocation failed");
     memset(kv, 0, sizeof(*kv));
@@ -101,18 +101,18 @@ int32_t skn_kv_create_by_position(skn_ctx *ctx, int32_t batch, int32_t n_kv_head
     kv->dtype = kv_dtype;
     kv->by_position = true;
     kv->k_pitch = (k_dim + 15) / 16 * 16;        // whole k-steps of the tensor-core kernel; the padding stays zero
-    kv->v_pitch = (v_dim + 15) / 16 * 16;
+    kv->v_pitch = kv->v_stride = (v_dim + 15) / 16 * 16;
     const size_t es = kv_dtype == SKN_KV_F32 ? 4 : 2, rows = (size_t)batch * n_kv_heads * capacity;
     cudaError_t e = cudaSetDevice(ctx->device);
     if (e == cudaSuccess) e = cudaMalloc(&kv->d_k, rows * kv->k_pitch * es);
-    if (e == cudaSuccess) e = cudaMalloc(&kv->d_v, rows * kv->v_pitch * es);
+    if (e == cudaSuccess && v_dim) e = cudaMalloc(&kv->d_v, rows * kv->v_pitch * es);
     if (e == cudaSuccess) e = cudaMalloc((void **)&kv->d_len, 2 * batch * sizeof(int32_t));
     if (e == cudaSuccess) {
         kv->d_start = kv->d_len + batch;
         e = cudaMemsetAsync(kv->d_len, 0, 2 * batch * sizeof(int32_t), ctx->stream);
     }
     if (e == cudaSuccess) e = cudaMemsetAsync(kv->d_k, 0, rows * kv->k_pitch * es, ctx->stream);
-    if (e == cudaSuccess) e = cudaMemsetAsync(kv->d_v, 0, rows * kv->v_pitch * es, ctx->stream);
+    if (e == cudaSuccess && v_dim) e = cudaMemsetAsync(kv->d_v, 0, rows * kv->v_pitch * es, ctx->stream);
     if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
     if (e != cudaSuccess) {
         skn_kv_destroy(kv);
@@ -151,8 +151,6 @@ int32_t skn_state_create(skn_ctx *ctx, int32_t slots, int32_t heads, int32_t k_d
     if (!out) return skn_fail(ctx, SKN_ERR_ARG, "out is NULL");
     *out = nullptr;
     if (slots < 1 || heads < 1 || k_dim < 1 || v_dim < 1) return skn_fail(ctx, SKN_ERR_ARG, "slots, heads and widths must be positive");
-    if (k_dim > SKN_ATTN_MAX_DIM || v_dim > SKN_ATTN_MAX_DIM)
-        return skn_fail(ctx, SKN_ERR_SHAPE, "head widths of %d and %d are above %d", k_dim, v_dim, SKN_ATTN_MAX_DIM);
     skn_state *s = new (std::nothrow) skn_state();
     if (!s) return skn_fail(ctx, SKN_ERR_OOM, "host allocation failed");
     s->magic = SKN_MAGIC_STATE;

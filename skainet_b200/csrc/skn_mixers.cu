@@ -11,7 +11,7 @@
 //  skn_ret_*_kernel        retention in chunks of 64 tokens: what each chunk adds to the state, the states at the chunk
 //                          starts, and the outputs; on the CUDA cores (fp32 decoder) or the tensor cores (two-term tf32)
 #include "skn_mixers.cuh"
-#include "skn_ptx.cuh"
+#include "skn_mma.cuh"
 
 #include <math.h>
 #include <stdlib.h>
@@ -83,6 +83,11 @@ __device__ __forceinline__ void prep_head(const float *src, int dim, int pad, co
     __syncwarp();
 }
 
+// first key that the query at position p sees
+__device__ __forceinline__ int first_visible(const skn_attn_args &a, int p) {
+    return a.chunk > 0 ? p / a.chunk * a.chunk : a.window > 0 ? max(0, p - a.window + 1) : 0;
+}
+
 __device__ __forceinline__ void put_out(const skn_rows_out &o, int64_t m, int64_t c, float v) {
     if (o.y32) o.y32[m * o.ld32 + c] = v;
     if (o.y16) o.y16[m * o.ld16 + c] = __float2bfloat16_rn(v);
@@ -98,7 +103,7 @@ static size_t attn_split_smem(int kp, int vp) {
 
 template <class CT, int RT, bool APPEND>
 __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT *__restrict__ kc_, const CT *__restrict__ vc_, int G, int cap, int dim,
-                           int vdim, int kp, int vp, int split, int max_splits, int hg, int m, float *sm) {
+                           int vdim, int kp, int vp, int vld, int split, int max_splits, int hg, int m, float *sm) {
     constexpr int VE = CacheVec<CT>::N;
     __shared__ float s_red[MIX_THREADS / 32][RT], s_max[RT], s_sum[RT];
     __shared__ bool s_last;
@@ -107,21 +112,22 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
     const int h0 = g * R + sub * RT, nh = min(RT, R - sub * RT);
     const int seq = m / st.T, slot = st.slot0 + seq;
     const int p = min(st.pos[slot] + m % st.T, st.max_pos - 1);
-    const int lo = a.chunk > 0 ? p / a.chunk * a.chunk : 0;
+    const int lo = first_visible(a, p);
     const int live = (p - lo) / KS + 1;
     if (split >= live) return;
     const int j0 = lo + split * KS, nk = min(KS, p + 1 - j0);
     const bool newest = APPEND && split == live - 1;       // this split ends with the step's own key
     float *qs = sm, *kn = qs + RT * kp, *vn = kn + kp, *ws = vn + vp, *red = ws + RT * KS;
     const size_t head_rows = ((size_t)slot * G + g) * cap;
-    CT *kc = const_cast<CT *>(kc_) + head_rows * kp, *vc = const_cast<CT *>(vc_) + head_rows * vp;
+    CT *kc = const_cast<CT *>(kc_) + head_rows * kp, *vc = const_cast<CT *>(vc_) + head_rows * vld;
     // keys and values on their way into L2 while the query is prepared: two threads per key
     const int key = tid >> 1, half = tid & 1;
     const int kslot = (j0 + key) % cap;
     if (key < nk) {
-        const char *kr = reinterpret_cast<const char *>(kc + (size_t)kslot * kp), *vr = reinterpret_cast<const char *>(vc + (size_t)kslot * vp);
+        const char *kr = reinterpret_cast<const char *>(kc + (size_t)kslot * kp), *vr = reinterpret_cast<const char *>(vc + (size_t)kslot * vld);
         for (int i = half * 128; i < (int)(kp * sizeof(CT)); i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(kr + i));
-        for (int i = half * 128; i < (int)(vp * sizeof(CT)); i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(vr + i));
+        if (vc != kc)
+            for (int i = half * 128; i < (int)(vp * sizeof(CT)); i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(vr + i));
     }
 
     for (int i = warp; i < RT + 2; i += MIX_THREADS / 32) {
@@ -137,7 +143,7 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
         } else if (newest) {
             for (int d = lane; d < vp; d += 32) {
                 const float v = d < vdim ? __ldcg(a.v + (int64_t)m * a.ld + (int64_t)g * vdim + d) : 0.f;
-                if (sub == 0 && d < vdim) CacheVec<CT>::store(vc + (size_t)(p % cap) * vp + d, v);
+                if (sub == 0 && d < vdim) CacheVec<CT>::store(vc + (size_t)(p % cap) * vld + d, v);
                 vn[d] = CacheVec<CT>::round(v);
             }
         }
@@ -215,7 +221,7 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
             if (newest && j == nk - 1) {
 #pragma unroll
                 for (int e = 0; e < VE; ++e) vv[e] = vn[cg_ * VE + e];
-            } else CacheVec<CT>::load(vc + (size_t)sl * vp + cg_ * VE, vv);
+            } else CacheVec<CT>::load(vc + (size_t)sl * vld + cg_ * VE, vv);
 #pragma unroll
             for (int r = 0; r < RT; ++r) {
                 const float w = ws[r * KS + j];
@@ -246,7 +252,7 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
         const int r = i / vdim, c = i % vdim;
         float o = 0.f;
         for (int k2 = 0; k2 < nk_l; ++k2) o += red[((size_t)k2 * RT + r) * vp + c];
-        if (live == 1) put_out(a.out, m, (int64_t)(h0 + r) * vdim + c, o / s_sum[r] * a.out_scale);
+        if (live == 1) put_out(a.out, m, (int64_t)(h0 + r) * vdim + c, o / (a.sink ? s_sum[r] + expf(a.sink[h0 + r] - s_max[r]) : s_sum[r]) * a.out_scale);
         else __stcg(a.scratch + (((size_t)m * a.heads + h0 + r) * max_splits + split) * (vdim + 2) + 2 + c, o);
     }
     if (live == 1) return;
@@ -268,9 +274,11 @@ __device__ void attn_split(const skn_attn_args &a, const skn_step &st, const CT 
         float top = -INFINITY;
         for (int x = lane; x < live; x += 32) top = fmaxf(top, __ldcg(rec + (size_t)x * (vdim + 2)));
         top = warp_max(top);
+        const float sink = a.sink ? a.sink[h0 + r] : -INFINITY;
+        top = fmaxf(top, sink);
         float den = 0.f;
         for (int x = lane; x < live; x += 32) den += expf(__ldcg(rec + (size_t)x * (vdim + 2)) - top) * __ldcg(rec + (size_t)x * (vdim + 2) + 1);
-        den = warp_sum(den);
+        den = warp_sum(den) + (a.sink ? expf(sink - top) : 0.f);
         for (int x = lane; x < live; x += 32)
             if (x < KS) ws[r * KS + x] = expf(__ldcg(rec + (size_t)x * (vdim + 2)) - top) / den;
         if (lane == 0) { s_max[r] = top; s_sum[r] = den; }
@@ -357,39 +365,41 @@ __device__ void ret_step(const skn_ret_args &r, const skn_step &st, float *__res
 template <class CT, int RT>
 __global__ void __launch_bounds__(MIX_THREADS, 4)
 skn_mix_decode_kernel(skn_attn_args a, skn_ret_args r, skn_step st, const CT *kc, const CT *vc, int G, int cap, int dim, int vdim, int kp,
-                      int vp, int max_splits, int n_attn, float *S, int RH, int rdk, int rdv, int rvp) {
+                      int vp, int vld, int max_splits, int n_attn, float *S, int RH, int rdk, int rdv, int rvp) {
     extern __shared__ __align__(16) float sm[];
     // the next launch starts only when this one's CTAs end (no early trigger): the weights it would stream meanwhile make
     // every step of this chain of dependent loads wait longer
     skn_pdl_wait();
     const int m = blockIdx.y, b = blockIdx.x;
-    if (b < n_attn) attn_split<CT, RT, true>(a, st, kc, vc, G, cap, dim, vdim, kp, vp, b % max_splits, max_splits, b / max_splits, m, sm);
+    if (b < n_attn) attn_split<CT, RT, true>(a, st, kc, vc, G, cap, dim, vdim, kp, vp, vld, b % max_splits, max_splits, b / max_splits, m, sm);
     else ret_step(r, st, S, RH, rdk, rdv, rvp, b - n_attn, m, sm);
 }
 
 template <class CT, int RT>
 __global__ void __launch_bounds__(MIX_THREADS)
-skn_attn_rows_kernel(skn_attn_args a, skn_step st, const CT *kc, const CT *vc, int G, int cap, int dim, int vdim, int kp, int vp, int max_splits) {
+skn_attn_rows_kernel(skn_attn_args a, skn_step st, const CT *kc, const CT *vc, int G, int cap, int dim, int vdim, int kp, int vp, int vld,
+                     int max_splits) {
     extern __shared__ __align__(16) float sm[];
     skn_pdl_launch_dependents();
     skn_pdl_wait();
-    attn_split<CT, RT, false>(a, st, kc, vc, G, cap, dim, vdim, kp, vp, blockIdx.x % max_splits, max_splits, blockIdx.x / max_splits, blockIdx.y, sm);
+    attn_split<CT, RT, false>(a, st, kc, vc, G, cap, dim, vdim, kp, vp, vld, blockIdx.x % max_splits, max_splits, blockIdx.x / max_splits, blockIdx.y, sm);
 }
 
 template <class CT, int RT>
 static cudaError_t launch_decode_t(const skn_step &s, const skn_attn_args *a, const skn_ret_args *r, bool rows_only, cudaStream_t st) {
     skn_attn_args aa = {};
     skn_ret_args rr = {};
-    int G = 1, cap = 1, dim = 1, vdim = 1, kp = 16, vp = 16, ms = 1, n_attn = 0, RH = 0, dk = 1, dv = 1, rvp = 4;
+    int G = 1, cap = 1, dim = 1, vdim = 1, kp = 16, vp = 16, vld = 16, ms = 1, n_attn = 0, RH = 0, dk = 1, dv = 1, rvp = 4;
     const CT *kc = nullptr, *vc = nullptr;
     float *S = nullptr;
     size_t smem = 0;
     if (a) {
         aa = *a;
         G = a->kv->n_kv_heads; cap = a->kv->capacity; dim = a->kv->head_dim; vdim = a->kv->v_dim; kp = a->kv->k_pitch; vp = a->kv->v_pitch;
+        vld = a->kv->v_stride;
         kc = (const CT *)a->kv->d_k;
         vc = (const CT *)a->kv->d_v;
-        ms = skn_chunk_attn_splits(a->chunk, s.max_pos);
+        ms = skn_attn_splits(a->chunk > 0 ? a->chunk : a->window, s.max_pos);
         n_attn = ms * G * ((a->heads / G + RT - 1) / RT);
         smem = attn_split_smem<CT, RT>(kp, vp);
     }
@@ -405,12 +415,12 @@ static cudaError_t launch_decode_t(const skn_step &s, const skn_attn_args *a, co
         auto kern = skn_attn_rows_kernel<CT, RT>;
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
         if (e != cudaSuccess) return e;
-        return skn_launch_pdl(kern, grid, dim3(MIX_THREADS), smem, st, 1, aa, s, kc, vc, G, cap, dim, vdim, kp, vp, ms);
+        return skn_launch_pdl(kern, grid, dim3(MIX_THREADS), smem, st, 1, aa, s, kc, vc, G, cap, dim, vdim, kp, vp, vld, ms);
     }
     auto kern = skn_mix_decode_kernel<CT, RT>;
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
     if (e != cudaSuccess) return e;
-    return skn_launch_pdl(kern, grid, dim3(MIX_THREADS), smem, st, 1, aa, rr, s, kc, vc, G, cap, dim, vdim, kp, vp, ms, n_attn, S, RH, dk, dv, rvp);
+    return skn_launch_pdl(kern, grid, dim3(MIX_THREADS), smem, st, 1, aa, rr, s, kc, vc, G, cap, dim, vdim, kp, vp, vld, ms, n_attn, S, RH, dk, dv, rvp);
 }
 
 static cudaError_t launch_split(const skn_step &s, const skn_attn_args *a, const skn_ret_args *r, bool rows_only, cudaStream_t st) {
@@ -421,6 +431,8 @@ static cudaError_t launch_split(const skn_step &s, const skn_attn_args *a, const
     return R > 2 ? launch_decode_t<float, 4>(s, a, r, rows_only, st) : R == 2 ? launch_decode_t<float, 2>(s, a, r, rows_only, st)
                                                                    : launch_decode_t<float, 1>(s, a, r, rows_only, st);
 }
+
+cudaError_t skn_launch_attn_rows(const skn_step &s, const skn_attn_args &a, cudaStream_t st) { return launch_split(s, &a, nullptr, true, st); }
 
 cudaError_t skn_launch_mix_decode(skn_ctx *, const skn_step &s, const skn_attn_args *a, const skn_ret_args *r, cudaStream_t st) {
     if (s.T != 1) return cudaErrorInvalidValue;
@@ -471,25 +483,6 @@ skn_head_prep_kernel(skn_attn_args a, skn_ret_args r, skn_step st, prep_args p, 
 constexpr int ATQ = 64, ATK = 32;      // queries and keys of a tile
 constexpr int AT_THREADS = ATQ * 2;    // a warp owns 16 queries
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool in) {
-    const int n = in ? 16 : 0;         // 0: the 16 bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t *>(&h);
-}
 // tanh through one exponential; absolute error a few 1e-7
 __device__ __forceinline__ float tanh_exp(float y) {
     const float t = __expf(2.f * fminf(fmaxf(y, -20.f), 20.f));
@@ -498,21 +491,21 @@ __device__ __forceinline__ float tanh_exp(float y) {
 
 template <int DV>
 __global__ void __launch_bounds__(AT_THREADS, DV <= 128 ? 3 : 1)
-skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict__ kc_, const __nv_bfloat16 *__restrict__ vc_, int G, int cap, int vdim,
-                   int kp, int vp) {
+skn_attn_tc_kernel(skn_attn_args a, skn_step st, skn_attn_keys src) {
     extern __shared__ __align__(16) uint8_t smb[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int kp = src.kp, vp = src.vp, cap = src.cap, vdim = src.vdim;
     const int ks = kp + 8, vs = DV + 8;                                  // row strides in elements
     __nv_bfloat16 *Q = reinterpret_cast<__nv_bfloat16 *>(smb), *K = Q + ATQ * ks, *V = K + 2 * ATK * ks;
     skn_pdl_launch_dependents();
     skn_pdl_wait();
-    const int t0 = (gridDim.x - 1 - blockIdx.x) * ATQ, h = blockIdx.y, seq = blockIdx.z, slot = st.slot0 + seq, g = h / (a.heads / G);
+    const int t0 = (gridDim.x - 1 - blockIdx.x) * ATQ, h = blockIdx.y, seq = blockIdx.z, slot = st.slot0 + seq, g = h / src.group;
     const int p0 = st.pos[slot], nq = min(ATQ, st.T - t0);
     const int pf = p0 + t0, pl = pf + nq - 1;                            // first and last query position
-    const int lo = a.chunk > 0 ? pf / a.chunk * a.chunk : 0;
+    const int lo = first_visible(a, pf);
     const int tiles = (pl - lo) / ATK + 1;
-    const size_t head_rows = ((size_t)slot * G + g) * cap;
-    const __nv_bfloat16 *kc = kc_ + head_rows * kp, *vc = vc_ + head_rows * vp;
+    const __nv_bfloat16 *kc = src.k + slot * src.k_slot + g * src.k_head, *vc = src.v + slot * src.v_slot + g * src.v_head;
+    const __nv_bfloat16 *kc2 = src.k2 ? src.k2 + slot * src.k2_slot : nullptr;
 
     const int slot0 = lo % cap;
     const bool idle = warp * 16 >= nq;                                   // none of this warp's queries exist
@@ -523,9 +516,9 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
         const bool in = j <= pl;
         int sl = slot0 + t * ATK + cr;
         if (sl >= cap) sl %= cap;
-        const __nv_bfloat16 *kr = kc + (size_t)sl * kp, *vr = vc + (size_t)sl * vp;
+        const __nv_bfloat16 *kr = kc + sl * src.k_row, *vr = vc + sl * src.v_row, *kr2 = kc2 + sl * src.k2_row - src.k1;
         const uint32_t kd = skn_smem_u32(K + ((size_t)buf * ATK + cr) * ks), vd = skn_smem_u32(V + ((size_t)buf * ATK + cr) * vs);
-        for (int c = cc * 8; c < kp; c += 32) cp_async16(kd + c * 2, kr + c, in);
+        for (int c = cc * 8; c < kp; c += 32) cp_async16(kd + c * 2, (c < src.k1 ? kr : kr2) + c, in);
 #pragma unroll
         for (int c = cc * 8; c < DV; c += 32) cp_async16(vd + c * 2, vr + (c < vp ? c : 0), in && c < vp);
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -540,14 +533,15 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
     float o[DV / 8][4];
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+    // a sink is one more key without a value: it opens the running maximum and, once per row, the sum
+    const float L2E = 1.4426950408889634f, sink = a.sink ? a.sink[h] * L2E : -INFINITY, l0 = a.sink && (lane & 3) == 0 ? 1.f : 0.f;
+    float mrow[2] = {sink, sink}, lrow[2] = {l0, l0};
     const int r0 = warp * 16 + (lane >> 2);
     const int qi[2] = {pf + r0, pf + r0 + 8};
     int qlo[2];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) qlo[i] = a.chunk > 0 ? qi[i] / a.chunk * a.chunk : 0;
-    const int w0 = pf + warp * 16, wlo = a.chunk > 0 ? w0 / a.chunk * a.chunk : 0, whi = a.chunk > 0 ? (w0 + 15) / a.chunk * a.chunk : 0;
-    const float L2E = 1.4426950408889634f;
+    for (int i = 0; i < 2; ++i) qlo[i] = first_visible(a, qi[i]);
+    const int w0 = pf + warp * 16, wlo = first_visible(a, w0), whi = first_visible(a, w0 + 15);
     const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
 
     for (int t = 0; t < tiles; ++t) {
@@ -648,23 +642,40 @@ skn_attn_tc_kernel(skn_attn_args a, skn_step st, const __nv_bfloat16 *__restrict
             const int c = n * 8 + (lane & 3) * 2;
 #pragma unroll
             for (int e = 0; e < 2; ++e)
-                if (c + e < vdim) put_out(a.out, m, (int64_t)h * vdim + c + e, o[n][i * 2 + e] * f);
+                if (c + e < vdim) {
+                    float v = o[n][i * 2 + e] * f;
+                    if (a.gate) v *= __fdividef(1.f, 1.f + __expf(fminf(-__ldcg(a.gate + m * a.ld_gate + (int64_t)h * vdim + c + e), 80.f)));
+                    put_out(a.out, m, (int64_t)h * vdim + c + e, v);
+                }
         }
     }
 }
 
 template <int DV>
-static cudaError_t launch_attn_tc(const skn_step &s, const skn_attn_args &a, cudaStream_t st) {
+static cudaError_t launch_attn_tc(const skn_step &s, const skn_attn_args &a, const skn_attn_keys &k, cudaStream_t st) {
     auto kern = skn_attn_tc_kernel<DV>;
-    const int kp = a.kv->k_pitch;
-    const size_t smem = ((size_t)(ATQ + 2 * ATK) * (kp + 8) + (size_t)2 * ATK * (DV + 8)) * 2;
+    const size_t smem = ((size_t)(ATQ + 2 * ATK) * (k.kp + 8) + (size_t)2 * ATK * (DV + 8)) * 2;
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return e;
-    return skn_launch_pdl(kern, dim3((s.T + ATQ - 1) / ATQ, a.heads, s.n_seqs), dim3(AT_THREADS), smem, st, 1, a, s, (const __nv_bfloat16 *)a.kv->d_k,
-                          (const __nv_bfloat16 *)a.kv->d_v, a.kv->n_kv_heads, a.kv->capacity, a.kv->v_dim, kp, a.kv->v_pitch);
+    return skn_launch_pdl(kern, dim3((s.T + ATQ - 1) / ATQ, a.heads, s.n_seqs), dim3(AT_THREADS), smem, st, 1, a, s, k);
 }
 
-bool skn_chunk_attn_tc(const skn_kvcache *kv) { return kv->dtype == SKN_KV_BF16 && kv->k_pitch <= 256 && kv->v_pitch <= 256; }
+cudaError_t skn_launch_attn_tiles(const skn_step &s, const skn_attn_args &a, const skn_attn_keys &k, cudaStream_t st) {
+    const int vp = k.vp;
+    return vp <= 32 ? launch_attn_tc<32>(s, a, k, st) : vp <= 64 ? launch_attn_tc<64>(s, a, k, st) : vp <= 96 ? launch_attn_tc<96>(s, a, k, st)
+           : vp <= 128 ? launch_attn_tc<128>(s, a, k, st) : vp <= 192 ? launch_attn_tc<192>(s, a, k, st) : launch_attn_tc<256>(s, a, k, st);
+}
+
+static skn_attn_keys cache_keys(const skn_kvcache *kv, int heads) {
+    skn_attn_keys k = {};
+    k.kp = k.k1 = kv->k_pitch; k.vp = kv->v_pitch; k.vdim = kv->v_dim; k.cap = kv->capacity; k.group = heads / kv->n_kv_heads;
+    k.k = (const __nv_bfloat16 *)kv->d_k; k.k_row = kv->k_pitch; k.k_head = (int64_t)kv->capacity * kv->k_pitch; k.k_slot = k.k_head * kv->n_kv_heads;
+    k.v = (const __nv_bfloat16 *)kv->d_v; k.v_row = kv->v_stride; k.v_head = (int64_t)kv->capacity * kv->v_stride; k.v_slot = k.v_head * kv->n_kv_heads;
+    return k;
+}
+
+bool skn_attn_tiles_fit(int kp, int vp) { return kp <= 256 && vp <= 256; }
+bool skn_chunk_attn_tc(const skn_kvcache *kv) { return kv->dtype == SKN_KV_BF16 && skn_attn_tiles_fit(kv->k_pitch, kv->v_pitch); }
 
 // ---- retention in chunks --------------------------------------------------------------------------------------------
 constexpr int RC = SKN_RET_CHUNK;
@@ -1034,9 +1045,7 @@ cudaError_t skn_launch_mix_prefill(skn_ctx *, const skn_step &s, const skn_attn_
     if (e != cudaSuccess) return e;
     if (a) {
         if (skn_chunk_attn_tc(a->kv)) {
-            const int vp = a->kv->v_pitch;
-            e = vp <= 32 ? launch_attn_tc<32>(s, *a, st) : vp <= 64 ? launch_attn_tc<64>(s, *a, st) : vp <= 96 ? launch_attn_tc<96>(s, *a, st)
-                : vp <= 128 ? launch_attn_tc<128>(s, *a, st) : vp <= 192 ? launch_attn_tc<192>(s, *a, st) : launch_attn_tc<256>(s, *a, st);
+            e = skn_launch_attn_tiles(s, *a, cache_keys(a->kv, a->heads), st);
         } else {
             e = launch_split(s, a, nullptr, true, st);
         }
@@ -1091,8 +1100,9 @@ cudaError_t skn_launch_rot_table(const skn_step &s, const double *freq, int half
     return skn_launch_pdl(skn_rot_table_kernel, dim3(s.n_seqs * s.T), dim3(128), 0, st, 1, s, freq, half, out, ld);
 }
 
+// Triggers no launch early: what follows it in the stream (the next step) starts when every launch before it is done, so a
+// step's kernels may read what earlier steps left (states, caches) ahead of their own dependency wait.
 __global__ void skn_advance_kernel(skn_step st, int32_t *pos, int32_t *status) {
-    skn_pdl_launch_dependents();
     skn_pdl_wait();
     for (int s = threadIdx.x; s < st.n_seqs; s += blockDim.x) {
         const int p = pos[st.slot0 + s] + st.T;
@@ -1141,7 +1151,7 @@ void skn_decay_powers(const double *decay, int heads, float *out) {
 }
 
 int32_t skn_check_attn_spec(skn_ctx *ctx, const skn_attn_spec *a) {
-    if (a->heads < 1 || a->kv_heads < 1 || a->dim < 1 || a->vdim < 1 || a->chunk < 0) return skn_fail(ctx, SKN_ERR_ARG, "invalid attention geometry");
+    if (a->heads < 1 || a->kv_heads < 1 || a->dim < 1 || a->vdim < 1 || a->chunk < 0 || a->window < 0 || (a->chunk && a->window)) return skn_fail(ctx, SKN_ERR_ARG, "invalid attention geometry");
     if (a->heads % a->kv_heads || a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > a->dim || a->dim > SKN_ATTN_MAX_DIM || a->vdim > SKN_ATTN_MAX_DIM)
         return skn_fail(ctx, SKN_ERR_SHAPE, "Shapes do not align.");
     return SKN_OK;
@@ -1158,7 +1168,7 @@ extern "C" {
 
 int32_t skn_chunk_attn(skn_kvcache *kv, const skn_attn_spec *spec, int32_t seq0, int32_t n_seqs, int32_t T, const int32_t *pos_host,
                        int32_t max_ctx, const float *q_gain_host, const float *k_gain_host, const float *q_host, const float *k_host,
-                       const float *v_host, float *out_host) {
+                       const float *v_host, const float *sink_host, float *out_host) {
     if (!skn_kv_ok(kv) || !kv->by_position) return skn_fail(nullptr, SKN_ERR_BAD_HANDLE, "not a position-addressed cache");
     skn_ctx *ctx = kv->ctx;
     SKN_ENTER(ctx);
@@ -1167,21 +1177,22 @@ int32_t skn_chunk_attn(skn_kvcache *kv, const skn_attn_spec *spec, int32_t seq0,
     if (rc) return rc;
     if (spec->kv_heads != kv->n_kv_heads || spec->dim != kv->head_dim || spec->vdim != kv->v_dim) return skn_fail(ctx, SKN_ERR_SHAPE, "Shapes do not align.");
     if ((rc = check_step(ctx, kv->batch, seq0, n_seqs, T, pos_host, max_ctx))) return rc;
-    const int need = spec->chunk > 0 && spec->chunk + T < max_ctx ? spec->chunk + T : max_ctx;
+    const int span = spec->chunk > 0 ? spec->chunk : spec->window;
+    const int need = span > 0 && span + T < max_ctx ? span + T : max_ctx;
     if (kv->capacity < need) return skn_fail(ctx, SKN_ERR_SHAPE, "this step needs a cache of %d tokens", need);
     SKN_CUDA(ctx, cudaSetDevice(ctx->device));
     const int H = spec->heads, G = spec->kv_heads, D = spec->dim, V = spec->vdim, M = n_seqs * T, half = spec->rot_dims / 2;
-    float *q, *out, *scratch, *qg, *kg;
+    float *q, *out, *scratch, *qg, *kg, *sink;
     int32_t *pos;
     unsigned *tickets;
     float2 *rot;
     double *freq;
     __nv_bfloat16 *q16;
-    const size_t nscr = skn_chunk_attn_scratch(M, H, V, spec->chunk, max_ctx);
+    const size_t nscr = skn_attn_scratch(M, H, V, span, max_ctx);
     Arena a = {nullptr, 0};
     for (int pass = 0; pass < 2; ++pass) {
         q = a.take<float>((size_t)M * ((size_t)H * D + (size_t)G * (D + V)));
-        out = a.take<float>((size_t)M * H * V); scratch = a.take<float>(nscr); qg = a.take<float>(D); kg = a.take<float>(D);
+        out = a.take<float>((size_t)M * H * V); scratch = a.take<float>(nscr); qg = a.take<float>(D); kg = a.take<float>(D); sink = a.take<float>(H);
         pos = a.take<int32_t>(kv->batch); tickets = a.take<unsigned>((size_t)M * H); rot = a.take<float2>((size_t)M * (half + 1));
         freq = a.take<double>(half + 1); q16 = a.take<__nv_bfloat16>((size_t)M * H * kv->k_pitch);
         if (pass == 0) {
@@ -1194,6 +1205,7 @@ int32_t skn_chunk_attn(skn_kvcache *kv, const skn_attn_spec *spec, int32_t seq0,
     skn_rot_freqs(spec->rot_base, spec->rot_dims, hf);
     if ((rc = upload(ctx, pos + seq0, pos_host, sizeof(int32_t) * n_seqs)) || (rc = upload(ctx, freq, hf, sizeof(double) * half))) return rc;
     if (q_gain_host && ((rc = upload(ctx, qg, q_gain_host, sizeof(float) * D)) || (rc = upload(ctx, kg, k_gain_host, sizeof(float) * D)))) return rc;
+    if (sink_host && (rc = upload(ctx, sink, sink_host, sizeof(float) * H))) return rc;
     SKN_CUDA(ctx, cudaMemsetAsync(tickets, 0, (size_t)M * H * sizeof(unsigned), ctx->stream));
     // joint rows [q | k | v], as the projection of a decoder leaves them
     const int64_t ld = (int64_t)H * D + (int64_t)G * (D + V);
@@ -1203,7 +1215,7 @@ int32_t skn_chunk_attn(skn_kvcache *kv, const skn_attn_spec *spec, int32_t seq0,
     const skn_step st = {seq0, n_seqs, T, pos, max_ctx};
     if (half) SKN_CUDA(ctx, skn_launch_rot_table(st, freq, half, rot, half, ctx->stream));
     skn_attn_args x = {};
-    x.kv = kv; x.heads = H; x.chunk = spec->chunk; x.scale = spec->scale; x.softcap = spec->softcap; x.eps = spec->eps;
+    x.kv = kv; x.heads = H; x.chunk = spec->chunk; x.window = spec->window; x.sink = sink_host ? sink : nullptr; x.scale = spec->scale; x.softcap = spec->softcap; x.eps = spec->eps;
     x.q_gain = q_gain_host ? qg : nullptr; x.k_gain = q_gain_host ? kg : nullptr;
     x.rot = skn_rot{rot, half, half};
     x.q = q; x.k = q + H * D; x.v = q + H * D + G * D; x.ld = ld;

@@ -8,11 +8,6 @@
 #pragma once
 #include "skn_dense.cuh"
 
-struct skn_rot {                    // angles of a step: row m, pair i at table[m * ld + i] = (cos, sin); half = 0: no rotation
-    const float2 *table;
-    int ld, half;
-};
-
 struct skn_step {
     int slot0, n_seqs, T;
     const int32_t *pos;             // device, per slot
@@ -21,7 +16,9 @@ struct skn_step {
 
 struct skn_attn_args {
     const skn_kvcache *kv;
-    int heads, chunk;               // chunk 0: every earlier key is visible
+    int heads;
+    int chunk, window;              // 0: every earlier key is visible; else the query's chunk, or the last `window` positions
+    const float *sink;              // [heads] scores that join the softmax denominator, NULL: none
     float scale, softcap;           // softcap 0: none
     float eps;
     const float *q_gain, *k_gain;   // [dim], NULL: no norm
@@ -30,9 +27,20 @@ struct skn_attn_args {
     int64_t ld;
     float out_scale;
     skn_rows_out out;               // pointers at the first column of this mixer's heads
-    float *scratch;                 // skn_chunk_attn_scratch() floats
+    const float *gate;              // raw gate rows [heads][vdim] whose sigmoid multiplies the heads (tile kernel only), NULL: none
+    int64_t ld_gate;
+    float *scratch;                 // skn_attn_scratch() floats
     unsigned *tickets;              // rows * heads, zero between launches
     __nv_bfloat16 *q16;             // [rows][heads][k_pitch] (tensor-core form)
+};
+
+// Where the tile kernel finds keys and values (bf16).  Slot s of the ring of sequence b, key head g: the first k1 elements of a key at
+// k + b k_slot + g k_head + s k_row, the rest (shared by the heads) at k2 + b k2_slot + s k2_row.  Every stride and width is a multiple of
+// 8 elements, kp of 16.
+struct skn_attn_keys {
+    const __nv_bfloat16 *k, *k2, *v;
+    int64_t k_row, k_head, k_slot, k2_row, k2_slot, v_row, v_head, v_slot;
+    int k1, kp, vp, vdim, cap, group;   // group: query heads per key head
 };
 
 struct skn_ret_args {
@@ -52,18 +60,24 @@ struct skn_ret_args {
 constexpr int SKN_RET_CHUNK = 64;
 constexpr int SKN_ATTN_SPLIT_KEYS = 128;
 
-// most key splits a query can need
-static inline int skn_chunk_attn_splits(int chunk, int max_pos) {
-    const int n = chunk > 0 && chunk < max_pos ? chunk : max_pos;
+// most key splits a query can need; span: chunk or window, 0 for none
+static inline int skn_attn_splits(int span, int max_pos) {
+    const int n = span > 0 && span < max_pos ? span : max_pos;
     return (n + SKN_ATTN_SPLIT_KEYS - 1) / SKN_ATTN_SPLIT_KEYS;
 }
 // floats of scratch for `rows` query rows on the split kernel
-static inline size_t skn_chunk_attn_scratch(int rows, int heads, int v_dim, int chunk, int max_pos) {
-    const int s = skn_chunk_attn_splits(chunk, max_pos);
+static inline size_t skn_attn_scratch(int rows, int heads, int v_dim, int span, int max_pos) {
+    const int s = skn_attn_splits(span, max_pos);
     return s > 1 ? (size_t)rows * heads * s * (v_dim + 2) : 1;
 }
 // whether many-token steps of this cache run on the tensor-core kernel (bf16 cache, head widths up to 256)
 bool skn_chunk_attn_tc(const skn_kvcache *kv);
+
+bool skn_attn_tiles_fit(int kp, int vp);
+// attention of prepared queries over the cache, whose newest keys are in place: any element type, any number of tokens
+cudaError_t skn_launch_attn_rows(const skn_step &s, const skn_attn_args &a, cudaStream_t st);
+// the same on the tensor-core tile kernel, queries in a.q16
+cudaError_t skn_launch_attn_tiles(const skn_step &s, const skn_attn_args &a, const skn_attn_keys &k, cudaStream_t st);
 
 // (cos, sin) of pos * freq[i] for every row of the step; angles in double
 cudaError_t skn_launch_rot_table(const skn_step &s, const double *freq, int half, float2 *out, int ld, cudaStream_t st);

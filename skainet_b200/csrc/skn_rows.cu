@@ -253,3 +253,80 @@ cudaError_t skn_launch_token_side(const skn_tensor *wg, const skn_tensor *wp, co
                           wg->pitch, (const uint8_t *)wp->d_blocks, wp->pitch, (const uint8_t *)table->d_blocks, table->pitch, table->n_rows, col, ids, x,
                           ldx, D, S, gain, eps);
 }
+
+// ---- norms of parts of a row, vectors added to rows ----------------------------------------------------------------
+// A row holds heads of `pitch` columns, the first `head` of each valid; the valid columns, heads in a row, fall into equal parts.
+__global__ void __launch_bounds__(256)
+skn_part_norm_kernel(const float *x, int64_t ldx, int heads, int head, int pitch, int parts, float eps, const float *__restrict__ gain, skn_rows_out out) {
+    __shared__ float red[8];
+    skn_pdl_launch_dependents();
+    skn_pdl_wait();
+    const int64_t m = blockIdx.x;
+    const float *xr = x + m * ldx;
+    const int len = heads * head / parts, p = blockIdx.y;
+    if (head == pitch && len % 4 == 0 && len <= 8192 && ldx % 4 == 0) {
+        // the part stays in registers
+        float4 v[8];
+        float ss = 0.f;
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int i = (u * 256 + threadIdx.x) * 4;
+            v[u] = i < len ? *reinterpret_cast<const float4 *>(xr + p * len + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+        }
+        const float r = 1.f / sqrtf(row_block_sum(ss, red) / (float)len + eps);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int i = (u * 256 + threadIdx.x) * 4, c = p * len + i;
+            if (i >= len) continue;
+            const float4 g = __ldg(reinterpret_cast<const float4 *>(gain + c));
+            const float4 f = make_float4(v[u].x * r * g.x, v[u].y * r * g.y, v[u].z * r * g.z, v[u].w * r * g.w);
+            if (out.y32) {
+                float *y = out.y32 + m * out.ld32 + c;
+                y[0] = f.x; y[1] = f.y; y[2] = f.z; y[3] = f.w;
+            }
+            if (out.y16) {
+                __nv_bfloat16 *y = out.y16 + m * out.ld16 + c;
+                *reinterpret_cast<__nv_bfloat162 *>(y) = __floats2bfloat162_rn(f.x, f.y);
+                *reinterpret_cast<__nv_bfloat162 *>(y + 2) = __floats2bfloat162_rn(f.z, f.w);
+            }
+        }
+        return;
+    }
+    auto column = [&](int i) { return (p * len + i) / head * pitch + (p * len + i) % head; };
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < len; i += 256) {
+        const float v = xr[column(i)];
+        ss = fmaf(v, v, ss);
+    }
+    const float r = 1.f / sqrtf(row_block_sum(ss, red) / (float)len + eps);
+    for (int i = threadIdx.x; i < len; i += 256) {
+        const int c = column(i);
+        const float v = xr[c] * r * gain[c];
+        if (out.y32) out.y32[m * out.ld32 + c] = v;
+        if (out.y16) out.y16[m * out.ld16 + c] = __float2bfloat16_rn(v);
+    }
+}
+
+cudaError_t skn_launch_part_norm_rows(const float *x, int64_t ldx, int M, int heads, int head, int pitch, int parts, float eps, const float *gain,
+                                      const skn_rows_out &out, cudaStream_t st) {
+    if (M == 0) return cudaSuccess;
+    return skn_launch_pdl(skn_part_norm_kernel, dim3(M, parts), dim3(256), 0, st, 1, x, ldx, heads, head, pitch, parts, eps, gain, out);
+}
+
+__global__ void __launch_bounds__(256)
+skn_add_vec_rows_kernel(float *x, int64_t ldx, int D, const float *__restrict__ vec, const float *add, int64_t ld_add) {
+    skn_pdl_launch_dependents();
+    skn_pdl_wait();
+    const int64_t m = blockIdx.x;
+    for (int i = threadIdx.x; i < D; i += 256) {
+        float v = x[m * ldx + i];
+        if (add) v += add[m * ld_add + i];
+        x[m * ldx + i] = v + vec[i];
+    }
+}
+
+cudaError_t skn_launch_add_vec_rows(float *x, int64_t ldx, int M, int D, const float *vec, const float *add, int64_t ld_add, cudaStream_t st) {
+    if (M == 0) return cudaSuccess;
+    return skn_launch_pdl(skn_add_vec_rows_kernel, dim3(M), dim3(256), 0, st, 1, x, ldx, D, vec, add, ld_add);
+}

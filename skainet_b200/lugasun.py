@@ -2,19 +2,19 @@
 
 A layer runs chunked softmax attention and retention side by side on one normalised input (`parallel` mixer), then an
 optional squared-relu feed-forward, then a token side input; a range of layers may be looped with a cache and a state
-per pass.  The decoder keeps `max_seqs` sequences of any lengths in slots; forward() advances one slot, or a range of
-them by the same number of tokens."""
+per pass."""
 from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import List, Optional, Sequence
+from typing import List, Optional
 
 import numpy as np
 
 from . import _ffi
+from .decoder import DenseDecoder, loop_runs
 from .registry import register
-from .tensor import Context, DenseTensor, SKN_OK, _check, _raise, from_bf16_bits
+from .tensor import Context, _check, from_bf16_bits
 
 
 @dataclass
@@ -102,12 +102,7 @@ class LugasunConfig:
 
     @property
     def runs(self) -> List[int]:
-        """Layer index of every layer run, the loop unrolled."""
-        n = len(self.layers)
-        if not self.loop:
-            return list(range(n))
-        a, b, times = self.loop
-        return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
+        return loop_runs(len(self.layers), self.loop)
 
     def tensor_shapes(self) -> dict:
         """name -> shape of every tensor of a checkpoint."""
@@ -131,20 +126,9 @@ class LugasunConfig:
         return out
 
 
-class LugasunDecoder:
-    """Owns the dense weights and the native decoder.  dtype "bfloat16" serves with bf16 operands and fp32 accumulation,
-    "float32" computes everything in fp32."""
-
-    DTYPES = {"float32": 0, "bfloat16": 1}
-
-    def __init__(self, ctx: Context, cfg: LugasunConfig, max_seqs: int = 1, max_tokens: int = 512, max_ctx: int = 4096,
-                 dtype: str = "bfloat16"):
-        if dtype not in self.DTYPES:
-            raise ValueError(f"dtype must be one of {sorted(self.DTYPES)}")
-        self.ctx, self.cfg, self.dtype = ctx, cfg, dtype
-        self.max_seqs, self.max_tokens, self.max_ctx = max_seqs, max(max_tokens, max_seqs), max_ctx
-        self._tensors: List[DenseTensor] = []
-        self._h = ctypes.c_void_p()
+class LugasunDecoder(DenseDecoder):
+    def _native_spec(self):
+        cfg = self.cfg
         decays = [(ctypes.c_double * len(l.right.decay))(*l.right.decay) for l in cfg.layers]
         layers = (_ffi.LugasunLayer * len(cfg.layers))()
         for l, c, d in zip(layers, cfg.layers, decays):
@@ -154,24 +138,7 @@ class LugasunDecoder:
             l.left_scale, l.right_scale, l.ff = c.left_scale, c.right_scale, c.ff
         start, stop, times = cfg.loop or (0, 0, 0)
         spec = _ffi.LugasunSpec(len(cfg.layers), cfg.width, cfg.vocab, cfg.side_dim, start, stop, times, cfg.eps, layers)
-        rc = _ffi.lib().skn_lugasun_create(ctx.handle, ctypes.byref(spec), max_seqs, self.max_tokens, max_ctx, self.DTYPES[dtype],
-                                           ctypes.byref(self._h))
-        if rc != SKN_OK:
-            self._h = ctypes.c_void_p()
-            _raise(ctx.handle, rc)
-
-    @property
-    def handle(self):
-        return self._h
-
-    @property
-    def vocab(self) -> int:
-        return self.cfg.vocab
-
-    def _up(self, bits: np.ndarray) -> DenseTensor:
-        t = DenseTensor(self.ctx, bits)
-        self._tensors.append(t)
-        return t
+        return _ffi.lib().skn_lugasun_create, spec, (layers, decays)
 
     def load(self, get) -> "LugasunDecoder":
         """get(name, shape) -> bf16 bit patterns (uint16) of a checkpoint tensor (SafetensorsFile.bf16_bits).  The
@@ -204,74 +171,6 @@ class LugasunDecoder:
         _check(self.ctx.handle, _ffi.lib().skn_lugasun_set_head(self._h, embed.handle, norm.ctypes.data, loop_in and loop_in.handle,
                                                                side and side.handle))
         return self
-
-    def reset(self, seq: int = -1):
-        """Forget the tokens of one sequence (-1: of all); its slot can be used again at once."""
-        _check(self.ctx.handle, _ffi.lib().skn_lugasun_reset(self._h, seq))
-
-    def position(self, seq: int = 0) -> int:
-        return int(_ffi.lib().skn_lugasun_position(self._h, seq))
-
-    def forward(self, tokens, seq: int = 0, want: Sequence[int] = (), want_next: bool = True):
-        """tokens [T] (one sequence) or [n, T] (the slots seq .. seq + n - 1); None with want_next: feed back the last
-        greedy id of slot `seq`.  Longer prompts than a step holds are run in portions.  Returns (next ids [n] or None,
-        logits [len(want), vocab] or None); want counts the rows of [n, T] flattened."""
-        if tokens is None:
-            return self._step(None, seq, 1, 1, list(want), want_next)
-        t = np.ascontiguousarray(tokens, dtype=np.int32)
-        t = t.reshape(1, -1) if t.ndim == 1 else t
-        n, T = t.shape
-        want = [int(x) for x in want]
-        if n < 1 or T < 1 or any(x < 0 or x >= n * T for x in want):
-            raise ValueError("Shapes do not align.")
-        per = self.max_tokens // n
-        logits = np.empty((len(want), self.vocab), dtype=np.float32) if want else None
-        nxt = None
-        for a in range(0, T, per):
-            b = min(T, a + per)
-            here = [(k, (x // T) * (b - a) + x % T - a) for k, x in enumerate(want) if a <= x % T < b]
-            nxt, lg = self._step(np.ascontiguousarray(t[:, a:b]), seq, n, b - a, [r for _, r in here], want_next and b == T)
-            if here:
-                logits[[k for k, _ in here]] = lg
-        return nxt, logits
-
-    def _step(self, t, seq, n, T, rows, want_next):
-        nxt = np.empty(n, dtype=np.int32) if want_next else None
-        want = np.asarray(rows, dtype=np.int32)
-        logits = np.empty((len(rows), self.vocab), dtype=np.float32) if len(rows) else None
-        _check(self.ctx.handle, _ffi.lib().skn_lugasun_forward(
-            self._h, seq, n, None if t is None else t.ctypes.data, T, len(rows), want.ctypes.data if len(rows) else None,
-            None if logits is None else logits.ctypes.data, None if nxt is None else nxt.ctypes.data))
-        return nxt, logits
-
-    def forward_dev(self, tokens_dev=None, T: int = 1, seq: int = 0, n: int = 1, head: bool = True):
-        """Enqueue one step: tokens_dev is a device address or tensor of [n, T] int32, None feeds back the greedy ids."""
-        ptr = None if tokens_dev is None else (tokens_dev.data_ptr() if hasattr(tokens_dev, "data_ptr") else tokens_dev)
-        _check(self.ctx.handle, _ffi.lib().skn_lugasun_forward_dev(self._h, seq, n, ptr, T, 1 if head else 0))
-
-    def trace_layers(self, on: bool):
-        """Record the residual stream after every layer run of the steps that follow (layer_outputs)."""
-        _check(self.ctx.handle, _ffi.lib().skn_lugasun_trace(self._h, 1 if on else 0, 0, None))
-
-    def layer_outputs(self, rows: int) -> np.ndarray:
-        """[layer runs, rows, width] of the last step."""
-        out = np.empty((len(self.cfg.runs), rows, self.cfg.width), dtype=np.float32)
-        _check(self.ctx.handle, _ffi.lib().skn_lugasun_trace(self._h, 1, rows, out.ctypes.data))
-        return out
-
-    def close(self):
-        if self._h:
-            _ffi.lib().skn_lugasun_destroy(self._h)
-            self._h = ctypes.c_void_p()
-        for t in self._tensors:
-            t.close()
-        self._tensors = []
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
 
 
 @register("Lugasun", family="lugasun")

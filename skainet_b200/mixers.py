@@ -1,4 +1,4 @@
-"""Token mixers on their own: a position-addressed KV cache with chunked softmax attention, and recurrent states with
+"""Token mixers on their own: a position-addressed KV cache with chunked or windowed softmax attention, and recurrent states with
 retention (skn_chunk_attn, skn_retention).  The decoders over dense weights run the same kernels inside their steps."""
 from __future__ import annotations
 
@@ -36,19 +36,22 @@ class PositionCache:
     def handle(self):
         return self._h
 
-    def attend(self, q, k, v, pos, scale: float, *, seq: int = 0, chunk: int = 0, softcap: float = 0.0, rot_dims: int = 0,
-               rot_base: float = 10000.0, q_gain=None, k_gain=None, eps: float = 1e-5, max_ctx: int = 1 << 20) -> np.ndarray:
+    def attend(self, q, k, v, pos, scale: float, *, seq: int = 0, chunk: int = 0, window: int = 0, softcap: float = 0.0,
+               rot_dims: int = 0, rot_base: float = 10000.0, q_gain=None, k_gain=None, sink=None, eps: float = 1e-5,
+               max_ctx: int = 1 << 20) -> np.ndarray:
         """q [n, T, heads, dim], k [n, T, kv_heads, dim], v [n, T, kv_heads, vdim] (raw heads) of the sequences seq ..,
-        pos[n] tokens having come before; returns [n, T, heads, vdim]."""
+        pos[n] tokens having come before; returns [n, T, heads, vdim].  A query sees the earlier keys of its own chunk, or the
+        last `window` ones, or all; sink [heads] joins the softmax denominators."""
         n, T, H, D = np.shape(q)
         q, k, v = _rows(q, n, T, H, D), _rows(k, n, T, self.kv_heads, D), _rows(v, n, T, self.kv_heads, self.vdim)
         pos = np.ascontiguousarray(pos, dtype=np.int32).reshape(n)
         gains = [None if g is None else _rows(g, D) for g in (q_gain, k_gain)]
-        spec = _ffi.AttnSpec(H, self.kv_heads, D, self.vdim, rot_dims, chunk, rot_base, scale, softcap, eps, 0)
+        spec = _ffi.AttnSpec(H, self.kv_heads, D, self.vdim, rot_dims, chunk, rot_base, scale, softcap, eps, window)
+        sinks = None if sink is None else _rows(sink, H)
         out = np.empty((n, T, H, self.vdim), dtype=np.float32)
         _check(self.ctx.handle, _ffi.lib().skn_chunk_attn(
             self._h, ctypes.byref(spec), seq, n, T, pos.ctypes.data, max_ctx, *[None if g is None else g.ctypes.data for g in gains],
-            q.ctypes.data, k.ctypes.data, v.ctypes.data, out.ctypes.data))
+            q.ctypes.data, k.ctypes.data, v.ctypes.data, None if sinks is None else sinks.ctypes.data, out.ctypes.data))
         return out
 
     def close(self):
