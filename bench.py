@@ -870,7 +870,7 @@ def run_decode(args):
 
 
 # --------------------------------------------------------------------------------------------
-# --workload lugasun: the Lugasun decoder beside the Llama-style decoder of the same width and size
+# --workload lugasun / tutezen: a decoder over dense weights beside the closest other one of the same width and size
 # --------------------------------------------------------------------------------------------
 LUGASUN_SIZES = {
     # width: heads, kv heads, head width, retention heads, their q/k and value widths, feed-forward, side width, layers
@@ -899,20 +899,20 @@ def lugasun_bench_configs(width: int):
     return cfg, LlamaConfig(n_layers=n, d_model=width, n_heads=H, n_kv_heads=G, head_dim=D, ffn_dim=ffn, vocab=LUGASUN_VOCAB)
 
 
-def _random_lugasun(ctx, cfg, **kw):
-    """Random weights; the layers share one set of values in buffers of their own."""
-    from skainet_b200.lugasun import LugasunDecoder
+def _random_dense(ctx, cls, cfg, **kw):
+    """A decoder over dense weights with random values; layers and experts share one set of values in buffers of their own."""
+    import re
     from skainet_b200.tensor import to_bf16_bits
     g, cache = np.random.default_rng(7), {}
 
     def get(name, shape):
-        key = name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name
+        key = re.sub(r"\.e\d+\.", ".e.", re.sub(r"^l\d+\.", "", name)), shape
         if key not in cache:
             a = np.ones(shape, np.float32) if len(shape) == 1 else \
-                g.standard_normal(size=shape, dtype=np.float32) * np.float32((1.0 if "embed" in key else shape[1] ** -0.5))
+                g.standard_normal(size=shape, dtype=np.float32) * np.float32((1.0 if "embed" in name else shape[1] ** -0.5))
             cache[key] = to_bf16_bits(a)
         return cache[key]
-    return LugasunDecoder(ctx, cfg, **kw).load(get)
+    return cls(ctx, cfg, **kw).load(get)
 
 
 def _random_llama(ctx, cfg, batch, T, max_ctx):
@@ -932,9 +932,65 @@ def _random_llama(ctx, cfg, batch, T, max_ctx):
     return dec
 
 
+TUTEZEN_SIZES = {
+    # width: state-space heads (of 64), attention heads, query and key latents, feed-forward, expert and shared widths, layers
+    1024: (32, 8, 512, 256, 4096, 512, 1024, 8),
+    2048: (64, 16, 1024, 512, 8192, 1024, 2048, 8),
+    4096: (128, 32, 1536, 512, 14336, 1536, 4096, 8),
+}
+TUTEZEN_WINDOW, TUTEZEN_EXPERTS, TUTEZEN_TOP = 1024, 32, 4
+
+
+def tutezen_bench_configs(width: int):
+    """(Tutezen configuration, its parameters in the layers, those that a token uses, Lugasun configuration with as many per layer as a
+    token of the first uses)."""
+    from skainet_b200.lugasun import LugasunConfig
+    from skainet_b200.tutezen import TutezenConfig
+    SH, H, QR, KR, F, EF, SF, n = TUTEZEN_SIZES[width]
+    dense = {"kind": "dense", "ff": F}
+    moe = {"kind": "moe", "router": {"experts": TUTEZEN_EXPERTS, "top": TUTEZEN_TOP}, "expert": {"ff": EF}, "shared": {"ff": SF}}
+    ssm = {"type": "mamba2", "mixer": {"heads": SH, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}}
+    att = {"type": "latent_attention", "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": QR, "kv_rank": KR, "scale": 192 ** -0.5,
+                                                 "mask": {"size": TUTEZEN_WINDOW}, "rot": {"base": 10000.0, "dims": 64}}}
+    pattern = [(ssm, dense), (ssm, moe), (ssm, moe), (att, dense), (ssm, dense), (ssm, moe), (ssm, dense), (att, moe)]
+    cfg = TutezenConfig.from_dict({"vocab": LUGASUN_VOCAB, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+                                   "layers": [dict(m, mlp=f) for m, f in pattern[:n]], "loop": {"start": 1, "stop": n - 1, "times": 1}})
+    sizes = {k: int(np.prod(v)) for k, v in cfg.tensor_shapes().items() if k[0] == "l" and k[1].isdigit()}
+    experts = sum(v for k, v in sizes.items() if ".mlp.e" in k)
+    used = sum(sizes.values()) - experts + experts * TUTEZEN_TOP // TUTEZEN_EXPERTS
+    lug, _ = lugasun_bench_configs(width)
+    base = sum(int(np.prod(v)) for k, v in lug.tensor_shapes().items() if k.startswith("l0.")) - 2 * width * lug.layers[0].ff
+    for l in lug.layers:
+        l.ff = max(256, round((used / n - base) / (2 * width) / 64) * 64)
+    return cfg, sum(sizes.values()), used, lug
+
+
 def run_lugasun(args):
-    """Prefill of a LUGASUN_PROMPT-token prompt (batch 1) and greedy decode (batch 1 and 16, one CUDA graph replay per
-    step, after the prompt) of both decoders, random weights.  Weights exceed L2 from width 2048 on."""
+    """Lugasun beside the Llama-style decoder (see run_decoders)."""
+    def arms(width):
+        lcfg, mcfg = lugasun_bench_configs(width)
+        n = sum(int(np.prod(v)) for k, v in lcfg.tensor_shapes().items() if "embed" not in k)
+        return [("lugasun", lcfg, n, n), ("llama", mcfg, n, n)]
+    run_decoders(args, "lugasun", arms, LUGASUN_SIZES,
+                 f"Lugasun (bf16) beside a Llama-style decoder (Q4_K, fp16 cache) of the same width, layers and parameters per layer; "
+                 f"{args.prompt}-token prompt, chunks of {LUGASUN_CHUNK}, vocabulary {LUGASUN_VOCAB}")
+
+
+def run_tutezen(args):
+    """Tutezen beside Lugasun, both over dense bf16 weights (see run_decoders)."""
+    def arms(width):
+        cfg, n, used, lcfg = tutezen_bench_configs(width)
+        m = sum(int(np.prod(v)) for k, v in lcfg.tensor_shapes().items() if k[0] == "l" and k[1].isdigit())
+        return [("tutezen", cfg, n, used), ("lugasun", lcfg, m, m)]
+    run_decoders(args, "tutezen", arms, TUTEZEN_SIZES,
+                 f"Tutezen beside Lugasun (both bf16) of the same width and layers, as many parameters per layer as a token of the first uses "
+                 f"({TUTEZEN_TOP} of {TUTEZEN_EXPERTS} experts); {args.prompt}-token prompt, window and chunks of {TUTEZEN_WINDOW}, vocabulary {LUGASUN_VOCAB}")
+
+
+def run_decoders(args, first, arms, sizes, workload):
+    """Prefill of a prompt (batch 1) and greedy decode (batch 1 and 16, one CUDA graph replay per step, after the prompt) of the decoders
+    in arms(width) = [(model, configuration, parameters in the layers, those that a token uses)], random weights.  Weights exceed L2
+    from width 2048 on."""
     import torch
     import skainet_b200 as skn
     torch.cuda.set_device(0)
@@ -944,21 +1000,23 @@ def run_lugasun(args):
     ctx.set_stream(stream.cuda_stream)
     T, steps = args.prompt, max(1, min(args.steps, 128))
     max_ctx = T + 4 * steps + 160
+    classes = {"lugasun": skn.LugasunDecoder, "tutezen": skn.TutezenDecoder}
     rows = []
     sampler = ClockSampler(0)
     sampler.start()
-    for width in ([args.width] if args.width else sorted(LUGASUN_SIZES)):
-        lcfg, mcfg = lugasun_bench_configs(width)
-        dense = sum(int(np.prod(v)) for k, v in lcfg.tensor_shapes().items() if "embed" not in k)
-        for name in ([args.only] if args.only else ["lugasun", "llama"]):
-            row = {"model": name, "width": width, "layers": len(lcfg.layers), "parameters_in_layers": dense}
+    for width in ([args.width] if args.width else sorted(sizes)):
+        for name, cfg, params, used in arms(width):
+            if args.only and name != args.only:
+                continue
+            n_layers = len(cfg.layers) if name in classes else cfg.n_layers
+            row = {"model": name, "width": width, "layers": n_layers, "parameters_in_layers": params, "parameters_per_token": used}
             for B in ([args.batch] if args.only else [1, 16]):
                 # decode at batch B; the prompt is timed at batch 1
                 prompt_len = T if B == 1 else 512
                 g = np.random.default_rng(3)
                 toks = torch.from_numpy(g.integers(0, LUGASUN_VOCAB, size=(B, prompt_len)).astype(np.int32)).cuda()
-                if name == "lugasun":
-                    dec = _random_lugasun(ctx, lcfg, max_seqs=B, max_tokens=max(prompt_len, B), max_ctx=max_ctx)
+                if name in classes:
+                    dec = _random_dense(ctx, classes[name], cfg, max_seqs=B, max_tokens=max(prompt_len, B), max_ctx=max_ctx)
 
                     def prefill():
                         dec.reset()
@@ -970,7 +1028,7 @@ def run_lugasun(args):
                 else:
                     # the Llama-style decoder advances all its sequences together: its prompt tokens go in portions
                     per = prompt_len if B == 1 else 64
-                    dec = _random_llama(ctx, mcfg, B, per, max_ctx)
+                    dec = _random_llama(ctx, cfg, B, per, max_ctx)
                     parts = [toks[:, i:i + per].contiguous() for i in range(0, prompt_len, per)]
 
                     def prefill():
@@ -1001,20 +1059,18 @@ def run_lugasun(args):
                 ms = _events_ms(torch, stream, graph.replay if graph else decode, steps, 3)
                 ctx.sync()
                 row[f"decode_b{B}_ms"], row[f"decode_b{B}_tok_s"] = ms, B * 1e3 / ms
-                if name == "lugasun" and B == 1:
-                    row["decode_weight_gbs"] = 2 * (dense + LUGASUN_VOCAB * width) / (ms * 1e-3) / 1e9
+                if name in classes and B == 1:
+                    row["decode_weight_gbs"] = 2 * (used + LUGASUN_VOCAB * width) / (ms * 1e-3) / 1e9
                 del graph
                 dec.close()
             rows.append(row)
     clocks = sampler.stop()
     peak, kind = measured_peak()
-    big = [r for r in rows if r["model"] == "lugasun"] or rows
+    big = [r for r in rows if r["model"] == first] or rows
     print(json.dumps({
-        "metric": "lugasun_decode_tok_s", "value": big[-1].get("decode_b1_tok_s", big[-1].get(f"decode_b{args.batch}_tok_s")), "unit": "tok/s",
+        "metric": f"{first}_decode_tok_s", "value": big[-1].get("decode_b1_tok_s", big[-1].get(f"decode_b{args.batch}_tok_s")), "unit": "tok/s",
         "n_gpus": 1, "steps": steps, "warmup": 3, "ms_per_step": None, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
-        "dtype": "bf16", "data": "synthetic",
-        "config": {"workload": f"Lugasun (bf16) beside a Llama-style decoder (Q4_K, fp16 cache) of the same width, layers and parameters "
-                               f"per layer; {T}-token prompt, chunks of {LUGASUN_CHUNK}, vocabulary {LUGASUN_VOCAB}"},
+        "dtype": "bf16", "data": "synthetic", "config": {"workload": workload},
         "hbm_peak_gbs": peak, "peak_kind": kind, "rows": rows, "clocks": clocks}), flush=True)
     ctx.close()
 
@@ -1045,15 +1101,17 @@ def main():
     ap.add_argument("--fused-exchange", default="auto", choices=["auto", "on", "off"],
                     help="tensor-parallel decode: push partial sums from the matvec epilogue (SKN_OPT_FUSED_EXCHANGE); "
                          "auto = the library's choice (off)")
-    ap.add_argument("--workload", default="matvec", choices=["matvec", "ffn", "attn", "sweep", "decode", "lugasun"],
+    ap.add_argument("--workload", default="matvec", choices=["matvec", "ffn", "attn", "sweep", "decode", "lugasun", "tutezen"],
                     help="matvec is the headline line; the others print one secondary JSON line (1 GPU)")
-    ap.add_argument("--width", type=int, default=0, choices=[0, *LUGASUN_SIZES], help="lugasun workload: this width only")
-    ap.add_argument("--only", default="", choices=["", "lugasun", "llama"], help="lugasun workload: this decoder only, at --batch")
-    ap.add_argument("--prompt", type=int, default=LUGASUN_PROMPT, help="lugasun workload: prompt tokens")
-    ap.add_argument("--no-prefill", action="store_true", help="lugasun workload: decode only")
+    ap.add_argument("--width", type=int, default=0, choices=[0, *LUGASUN_SIZES], help="lugasun / tutezen workloads: this width only")
+    ap.add_argument("--only", default="", choices=["", "lugasun", "llama", "tutezen"],
+                    help="lugasun / tutezen workloads: this decoder only, at --batch")
+    ap.add_argument("--prompt", type=int, default=LUGASUN_PROMPT, help="lugasun / tutezen workloads: prompt tokens")
+    ap.add_argument("--no-prefill", action="store_true", help="lugasun / tutezen workloads: decode only")
     args = ap.parse_args()
     if args.impl == "ours" and args.workload != "matvec":
-        return {"ffn": run_ffn, "attn": run_attn, "sweep": run_sweep, "decode": run_decode, "lugasun": run_lugasun}[args.workload](args)
+        return {"ffn": run_ffn, "attn": run_attn, "sweep": run_sweep, "decode": run_decode, "lugasun": run_lugasun,
+                "tutezen": run_tutezen}[args.workload](args)
     if args.impl == "reference":
         run_reference(args)
     else:

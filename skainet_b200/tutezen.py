@@ -204,7 +204,10 @@ class TutezenDecoder(DenseDecoder):
         S = self.cfg.tensor_shapes()
 
         def w(name):
-            return np.ascontiguousarray(get(name, S[name]))
+            a = np.ascontiguousarray(get(name, S[name]))
+            if a.shape != S[name]:               # (padding would hide it from the native check)
+                raise ValueError(f"{name} is {list(a.shape)}, expected {list(S[name])}")
+            return a
 
         def vec(name):
             return from_bf16_bits(w(name))
