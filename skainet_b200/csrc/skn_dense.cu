@@ -125,18 +125,30 @@ __device__ __forceinline__ void dense_store_run(const skn_epi &e, int64_t m, int
 template <int EPI, int NC>
 __device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count, bool in) {
     const bool odd = n & 1;
-    const bool act = EPI == SKN_EPI_SILU_TAIL && n >= e.n_act;
+    if (EPI == SKN_EPI_ROTATE) {
+        // the angles of the run are loaded before its first store
+        const int i = ((int)(n % e.rot_head) - e.rot_lo) >> 1;
+        const bool turn = in && i >= 0 && i < e.rot.half;
+        float2 cs[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) cs[c] = turn && c < count ? __ldcg(e.rot.table + (m + c) * e.rot.ld + i) : make_float2(1.f, 0.f);
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            const float other = __shfl_xor_sync(0xffffffffu, v[c], 1);
+            v[c] = odd ? v[c] * cs[c].x + other * cs[c].y : v[c] * cs[c].x - other * cs[c].y;
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+            if (c < count && in) dense_put(e, m + c, n, v[c]);
+        return;
+    }
+    const bool act = n >= e.n_act;
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
         const float other = __shfl_xor_sync(0xffffffffu, v[c], 1);
         if (c >= count || !in) continue;
-        if (act) {
-            if (!odd) dense_put_silu(e, m + c, n, v[c], other);
-            continue;
-        }
-        float2 cs;
-        if (EPI == SKN_EPI_ROTATE && dense_angle(e, m + c, n, cs)) v[c] = odd ? v[c] * cs.x + other * cs.y : v[c] * cs.x - other * cs.y;
-        dense_put(e, m + c, n, v[c]);
+        if (!act) dense_put(e, m + c, n, v[c]);
+        else if (!odd) dense_put_silu(e, m + c, n, v[c], other);
     }
 }
 
@@ -212,10 +224,11 @@ __device__ __forceinline__ int mvd_row(int lane) { return ((lane >> 4) & 1) * 4 
 struct mvd_pick {
     const int32_t *expert;
     const uint8_t *w2;                  // SKN_PICK_COLS
-    int64_t pitch1;                     // bytes of a row of w / of w2 (the joint row has `pitch` bytes)
+    int64_t pitch1;                     // SKN_PICK_COLS: bytes that w (0: none of it) and each expert have in a joint row of `pitch` bytes
     int64_t pitch2;
     int n, rows_per;
 };
+constexpr int MVD_PICKS = 64;           // experts whose numbers are kept in shared memory
 struct mvd_norm {
     const float *gain;
     float eps;
@@ -224,11 +237,12 @@ struct mvd_norm {
 
 template <int MR, int UU, int PICK>
 __global__ void __launch_bounds__(MVD_THREADS, 2)
-skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int K, int m0, const float *x, int64_t ldx, const float *xb,
+skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitch, int N, int K, int m0, const float *x, int64_t ldx, const float *xb,
                         int64_t ldxb, int ka, mvd_norm nm, mvd_pick pk, int stages, skn_epi e, int32_t *status) {
     extern __shared__ __align__(128) uint8_t ring[];
     constexpr int GR = mvd_stage_rows(MR, UU);
     __shared__ uint64_t full_bar[MVD_MAX_STAGES], empty_bar[MVD_MAX_STAGES];
+    __shared__ int picks[PICK != SKN_PICK_NONE ? MVD_PICKS : 1];
     __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS], psum[MR][MVD_WARPS][SKN_NORM_PARTS];
     const float *__restrict__ gain = nm.gain;
     const bool pairs = skn_epi_pairs(e.kind), partial = gain && nm.cols > 0;
@@ -253,14 +267,18 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
             int early = 0;
             if constexpr (PICK == SKN_PICK_COLS) {
                 // the first stages' own pieces depend on no kernel before this one
-                for (; early < stages && early < steps; ++early) {
+                for (; pk.pitch1 && early < stages && early < steps; ++early) {
                     const int row = r0 + early * GR, n = min(GR, r1 - row);
                     skn_mbar_expect_tx(&full_bar[early], (uint32_t)(n * pitch));
                     for (int j = 0; j < n; ++j)
-                        skn_bulk_g2s(ring + early * stage_bytes + j * pitch, W + (int64_t)(row + j) * pk.pitch1, (uint32_t)pk.pitch1, &full_bar[early]);
+                        skn_bulk_g2s(ring + early * stage_bytes + j * pitch, W + (row + j) * wld, (uint32_t)pk.pitch1, &full_bar[early]);
                 }
             }
-            if constexpr (PICK != SKN_PICK_NONE) skn_pdl_wait();
+            if constexpr (PICK != SKN_PICK_NONE) {
+                skn_pdl_wait();
+                for (int x = 0; x < min(pk.n, MVD_PICKS); ++x) picks[x] = __ldcg(pk.expert + x);
+            }
+            auto picked = [&](int x) { return (int64_t)(x < MVD_PICKS ? picks[x] : __ldcg(pk.expert + x)); };
             for (int i = 0; i < steps; ++i) {
                 const int row = r0 + i * GR;
                 if (i >= early && !skn_mbar_wait(&empty_bar[s], phase)) {
@@ -272,20 +290,22 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
                 if (i >= early) skn_mbar_expect_tx(&full_bar[s], bytes);
                 uint8_t *dst = ring + s * stage_bytes;
                 if constexpr (PICK == SKN_PICK_NONE) {
-                    skn_bulk_g2s(dst, W + (int64_t)row * pitch, bytes, &full_bar[s]);
+                    if (wld == pitch) skn_bulk_g2s(dst, W + row * wld, bytes, &full_bar[s]);
+                    else
+                        for (int j = 0; j < n; ++j) skn_bulk_g2s(dst + j * pitch, W + (row + j) * wld, (uint32_t)pitch, &full_bar[s]);
                 } else if constexpr (PICK == SKN_PICK_ROWS) {
                     for (int j = 0; j < n; ++j) {
                         const int r = row + j, x = r / pk.rows_per;
-                        skn_bulk_g2s(dst + j * pitch, W + ((int64_t)__ldcg(pk.expert + x) * pk.rows_per + r - x * pk.rows_per) * pitch, (uint32_t)pitch, &full_bar[s]);
+                        skn_bulk_g2s(dst + j * pitch, W + (picked(x) * pk.rows_per + r - x * pk.rows_per) * wld, (uint32_t)pitch, &full_bar[s]);
                     }
                 } else {
                     for (int j = 0; j < n; ++j) {
                         const int r = row + j;
                         uint8_t *d = dst + j * pitch;
-                        if (i >= early) skn_bulk_g2s(d, W + (int64_t)r * pk.pitch1, (uint32_t)pk.pitch1, &full_bar[s]);
+                        if (i >= early && pk.pitch1) skn_bulk_g2s(d, W + r * wld, (uint32_t)pk.pitch1, &full_bar[s]);
                         d += pk.pitch1;
                         for (int x = 0; x < pk.n; ++x, d += pk.pitch2)
-                            skn_bulk_g2s(d, pk.w2 + ((int64_t)__ldcg(pk.expert + x) * N + r) * pk.pitch2, (uint32_t)pk.pitch2, &full_bar[s]);
+                            skn_bulk_g2s(d, pk.w2 + (picked(x) * N + r) * pk.pitch2, (uint32_t)pk.pitch2, &full_bar[s]);
                     }
                 }
                 if (++s == stages) {
@@ -541,11 +561,14 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t pitch, int N, int
     }
 }
 
-// bytes of the joint weight row
-static int64_t mvd_pitch(const skn_linear &l) { return l.pick.kind == SKN_PICK_COLS ? l.w->pitch + l.pick.n * l.pick.w2->pitch : l.w->pitch; }
+// columns [col0, col0 + cols) of w (whole vectors of 8), then the picked experts' rows
+struct mvd_piece {
+    int64_t col0, cols;
+    bool experts;
+};
 
 template <int MR, int UU, int PICK>
-static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int m0, cudaStream_t st) {
+static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, const mvd_piece &pc, int m0, cudaStream_t st) {
     auto kern = skn_dense_matvec_kernel<MR, UU, PICK>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
@@ -553,8 +576,10 @@ static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int m0, cudaStr
         if (e != cudaSuccess) return e;
         attr_done[ctx->device & 63] = true;
     }
-    const int64_t pitch = mvd_pitch(l);
-    const int N = PICK == SKN_PICK_ROWS ? l.pick.n * l.pick.rows_per : (int)l.w->n_rows, K = (int)skn_linear_cols(l), rows = mvd_stage_rows(MR, UU);
+    const int64_t own = pc.cols * 2, pitch = own + (pc.experts ? l.pick.n * l.pick.w2->pitch : 0), all = l.w->pitch / 2;
+    const bool whole = pc.col0 == 0 && (pc.experts || pc.cols == all);
+    const int N = PICK == SKN_PICK_ROWS ? l.pick.n * l.pick.rows_per : (int)l.w->n_rows, rows = mvd_stage_rows(MR, UU);
+    const int K = (int)(whole ? skn_linear_cols(l) : pc.experts ? pitch / 2 : pc.col0 + pc.cols < l.w->n_cols ? pc.cols : l.w->n_cols - pc.col0);
     const size_t xbytes = UU > 0 ? 0 : (size_t)MR * pitch * 2;
     size_t room = mvd_smem(MR) - xbytes;
     if (room > (size_t)MVD_RING) room = MVD_RING;
@@ -563,48 +588,90 @@ static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int m0, cudaStr
     if (stages > MVD_MAX_STAGES) stages = MVD_MAX_STAGES;
     const int units = skn_epi_pairs(l.epi.kind) ? (N + 1) / 2 : N;
     const int grid = units < ctx->sm_count ? units : ctx->sm_count;
-    const mvd_norm nm = {l.gain, l.eps, l.gain ? l.norm_cols : 0, l.norm_parts > 0 ? l.norm_parts : 1};
-    const mvd_pick pk = {l.pick.expert, PICK == SKN_PICK_COLS ? (const uint8_t *)l.pick.w2->d_blocks : nullptr, l.w->pitch,
+    // the piece of x, and the norm if it lies in it
+    const float *x = l.x32 + pc.col0;
+    int64_t ldx = l.ld_x32, ka = l.x32b ? l.k_a - pc.col0 : K;
+    if (ka <= 0) {
+        x = l.x32b - ka;
+        ldx = l.ld_x32b;
+        ka = K;
+    } else if (ka > K) {
+        ka = K;
+    }
+    const bool norm = l.gain && pc.col0 == 0;
+    const mvd_norm nm = {norm ? l.gain : nullptr, l.eps, norm ? l.norm_cols : 0, l.norm_parts > 0 ? l.norm_parts : 1};
+    const mvd_pick pk = {l.pick.expert, PICK == SKN_PICK_COLS ? (const uint8_t *)l.pick.w2->d_blocks : nullptr, own,
                          PICK == SKN_PICK_COLS ? l.pick.w2->pitch : 0, l.pick.n, l.pick.rows_per};
-    return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks, pitch,
-                          N, K, m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, nm, pk, stages, l.epi, ctx->d_status);
+    return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks + pc.col0 * 2,
+                          l.w->pitch, pitch, N, K, m0, x, ldx, l.x32b, l.ld_x32b, (int)ka, nm, pk, stages, l.epi, ctx->d_status);
 }
 
+// vectors per lane of a row of `cols` columns
+static int mvd_uu(int64_t cols) { return (int)(((cols / 8 + MVD_WARPS - 1) / MVD_WARPS + 31) / 32); }
+constexpr int MVD_MAX_UU = 7;
+constexpr int64_t MVD_PIECE = (int64_t)MVD_MAX_UU * 32 * MVD_WARPS * 8;      // columns of x that the registers hold
+
 template <int PICK>
-static cudaError_t launch_mvd_pick(skn_ctx *ctx, const skn_linear &l, int uu, cudaStream_t st) {
-    if (l.M != 1) return cudaErrorInvalidValue;
-    switch (uu) {
-    case 1: return launch_mvd<1, 1, PICK>(ctx, l, 0, st);
-    case 2: return launch_mvd<1, 2, PICK>(ctx, l, 0, st);
-    case 3: case 4: return launch_mvd<1, 4, PICK>(ctx, l, 0, st);
-    default: return launch_mvd<1, 0, PICK>(ctx, l, 0, st);
+static cudaError_t launch_mvd_pick(skn_ctx *ctx, const skn_linear &l, const mvd_piece &pc, int64_t cols, cudaStream_t st) {
+    switch (mvd_uu(cols)) {
+    case 1: return launch_mvd<1, 1, PICK>(ctx, l, pc, 0, st);
+    case 2: return launch_mvd<1, 2, PICK>(ctx, l, pc, 0, st);
+    case 3: case 4: return launch_mvd<1, 4, PICK>(ctx, l, pc, 0, st);
+    case 5: case 6: case 7: return launch_mvd<1, 7, PICK>(ctx, l, pc, 0, st);
+    default: return launch_mvd<1, 0, PICK>(ctx, l, pc, 0, st);
     }
 }
 
-cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStream_t st) {
-    const int64_t pitch = mvd_pitch(l);
-    if (pitch * 3 > mvd_smem(1)) return cudaErrorNotSupported;       // one stage and one activation row must fit
-    if (l.gain && l.norm_cols > 0 && !skn_norm_folds(l.norm_cols, l.norm_parts)) return cudaErrorInvalidValue;
-    const int uu = (int)(((pitch / 16 + MVD_WARPS - 1) / MVD_WARPS + 31) / 32);
-    if (l.pick.kind == SKN_PICK_ROWS) return launch_mvd_pick<SKN_PICK_ROWS>(ctx, l, uu, st);
-    if (l.pick.kind == SKN_PICK_COLS) return launch_mvd_pick<SKN_PICK_COLS>(ctx, l, uu, st);
+static cudaError_t launch_mvd_row(skn_ctx *ctx, const skn_linear &l, const mvd_piece &pc, int m0, cudaStream_t st) {
     constexpr int P = SKN_PICK_NONE;
+    switch (mvd_uu(pc.cols)) {
+    case 1: return launch_mvd<1, 1, P>(ctx, l, pc, m0, st);
+    case 2: return launch_mvd<1, 2, P>(ctx, l, pc, m0, st);
+    case 3: return launch_mvd<1, 3, P>(ctx, l, pc, m0, st);
+    case 4: return launch_mvd<1, 4, P>(ctx, l, pc, m0, st);
+    case 5: return launch_mvd<1, 5, P>(ctx, l, pc, m0, st);
+    case 6: return launch_mvd<1, 6, P>(ctx, l, pc, m0, st);
+    case 7: return launch_mvd<1, 7, P>(ctx, l, pc, m0, st);
+    default: return launch_mvd<1, 0, P>(ctx, l, pc, m0, st);
+    }
+}
+
+// One activation row whose columns exceed the registers: sums that add to the residual stream may be formed piece by piece, each piece
+// at the rate of a short row (x in registers, many stages in the ring).
+static cudaError_t launch_mvd_pieces(skn_ctx *ctx, const skn_linear &l, int m0, cudaStream_t st) {
+    const int64_t all = l.w->pitch / 2, least = l.gain ? l.norm_cols : 0;
+    const int64_t n = (all + MVD_PIECE - 1) / MVD_PIECE;
+    int64_t size = ((all + n - 1) / n + 7) / 8 * 8;
+    if (size < least) size = least;
+    for (int64_t c = 0; c < all; c += size) {
+        const cudaError_t e = launch_mvd_row(ctx, l, mvd_piece{c, all - c < size ? all - c : size, false}, m0, st);
+        if (e != cudaSuccess) return e;
+    }
+    return cudaSuccess;
+}
+
+cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStream_t st) {
+    const int64_t all = l.w->pitch / 2, cols = l.pick.kind == SKN_PICK_COLS ? skn_linear_cols(l) : all, pitch = cols * 2;
+    if (l.gain && l.norm_cols > 0 && !skn_norm_folds(l.norm_cols, l.norm_parts)) return cudaErrorInvalidValue;
+    if (l.pick.kind && l.M != 1) return cudaErrorInvalidValue;
+    // (a whole-row norm needs the whole row at once)
+    const bool pieces = l.epi.kind == SKN_EPI_ADD && (!l.gain || (l.norm_cols > 0 && l.norm_cols <= MVD_PIECE));
+    if (l.pick.kind == SKN_PICK_ROWS) return launch_mvd_pick<SKN_PICK_ROWS>(ctx, l, mvd_piece{0, all, false}, all, st);
+    if (l.pick.kind == SKN_PICK_COLS) {
+        if (!pieces || mvd_uu(cols) <= 4) return launch_mvd_pick<SKN_PICK_COLS>(ctx, l, mvd_piece{0, all, true}, cols, st);
+        const cudaError_t e = launch_mvd_pieces(ctx, l, 0, st);
+        return e != cudaSuccess ? e : launch_mvd_pick<SKN_PICK_COLS>(ctx, l, mvd_piece{all, 0, true}, cols - all, st);
+    }
+    if (pitch * 3 > mvd_smem(1)) return cudaErrorNotSupported;       // one stage and one activation row must fit
+    const mvd_piece whole = {0, all, false};
     for (int m0 = 0; m0 < l.M;) {
         const int left = l.M - m0;
         cudaError_t e;
         int mr = 1;
-        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0, P>(ctx, l, m0, st); }
-        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0, P>(ctx, l, m0, st); }
-        else switch (uu) {
-            case 1: e = launch_mvd<1, 1, P>(ctx, l, m0, st); break;
-            case 2: e = launch_mvd<1, 2, P>(ctx, l, m0, st); break;
-            case 3: e = launch_mvd<1, 3, P>(ctx, l, m0, st); break;
-            case 4: e = launch_mvd<1, 4, P>(ctx, l, m0, st); break;
-            case 5: e = launch_mvd<1, 5, P>(ctx, l, m0, st); break;
-            case 6: e = launch_mvd<1, 6, P>(ctx, l, m0, st); break;
-            case 7: e = launch_mvd<1, 7, P>(ctx, l, m0, st); break;
-            default: e = launch_mvd<1, 0, P>(ctx, l, m0, st); break;
-        }
+        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0, SKN_PICK_NONE>(ctx, l, whole, m0, st); }
+        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0, SKN_PICK_NONE>(ctx, l, whole, m0, st); }
+        else if (pieces && mvd_uu(all) > MVD_MAX_UU) e = launch_mvd_pieces(ctx, l, m0, st);
+        else e = launch_mvd_row(ctx, l, whole, m0, st);
         if (e != cudaSuccess) return e;
         m0 += mr;
     }
@@ -705,11 +772,13 @@ cudaError_t skn_launch_dense_f32(skn_ctx *, const skn_linear &l, cudaStream_t st
 // ---- tensor cores ------------------------------------------------------------------------------------------------
 constexpr int DTC_BM = 128, DTC_BK = 64;
 constexpr int DTC_A_BYTES = DTC_BM * DTC_BK * 2;
-constexpr int DTC_THREADS = 6 * 32;              // four epilogue warps, one MMA warp, one TMA warp
+constexpr int DTC_EPI = 8, DTC_MMA = DTC_EPI, DTC_TMA = DTC_EPI + 1;   // eight epilogue warps (two per quarter of TMEM's lanes), MMA, TMA
+constexpr int DTC_THREADS = (DTC_EPI + 2) * 32;
+constexpr int DTC_GROUP_BOX = 64;                // tokens of one TMA box of a grouped tile
 constexpr int DTC_SMEM = 208 * 1024;
 constexpr int DTC_MAX_STAGES = 8;
 
-__device__ __forceinline__ void dtc_barrier_epilogue() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void dtc_barrier_epilogue() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 struct dtc_tile {
     int m0, cols, sp, n0, w0;           // first token and tokens of the tile, K split, first row of the output, and of the weight
@@ -741,9 +810,10 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
         t.m0 = (u % mt) * NT;
         t.cols = min(NT, M - t.m0);
         if (GROUPS) {
-            const int g = dense_group_of(start, E, u % mt);
-            t.m0 = off[g] + (u % mt - start[g]) * NT;
-            t.cols = min(NT, off[g + 1] - t.m0);
+            // a group's tiles are of one size
+            const int g = dense_group_of(start, E, u % mt), n = start[g + 1] - start[g], size = ((off[g + 1] - off[g] + n - 1) / n + 15) / 16 * 16;
+            t.m0 = off[g] + (u % mt - start[g]) * size;
+            t.cols = min(size, off[g + 1] - t.m0);
             t.w0 += g * N;
         }
         return t;
@@ -756,18 +826,18 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
         }
         for (int b = 0; b < 2; ++b) {
             skn_mbar_init(&acc_full[b], 1);
-            skn_mbar_init(&acc_empty[b], 4);
+            skn_mbar_init(&acc_empty[b], DTC_EPI);
         }
         skn_fence_mbar_init();
     }
-    if (warp == 4) tc_alloc(&tmem_slot, tmem_cols);
+    if (warp == DTC_MMA) tc_alloc(&tmem_slot, tmem_cols);
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = tmem_slot;
     // the weights depend on no kernel before this one: the first unit's first stages are requested ahead of the wait
     int early = 0;
-    if (!GROUPS && warp == 5 && lane == 0 && (int)blockIdx.x < units) {
+    if (!GROUPS && warp == DTC_TMA && lane == 0 && (int)blockIdx.x < units) {
         const int sp = (blockIdx.x / mt) % splits, n0 = (blockIdx.x / mt / splits) * DTC_BM;
         const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
         for (; early < stages && early < ke - kb; ++early) {
@@ -783,7 +853,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
         units = mt * nt;
     }
 
-    if (warp == 5) {
+    if (warp == DTC_TMA) {
         if (lane == 0) {
             bool ok = true;
             int it = 0;
@@ -800,10 +870,13 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                             ok = false;
                             break;
                         }
-                        skn_mbar_expect_tx(&full_bar[s], (uint32_t)stage_bytes);
+                        const int boxes = (tl.cols + DTC_GROUP_BOX - 1) / DTC_GROUP_BOX, box = min(NT, DTC_GROUP_BOX);
+                        skn_mbar_expect_tx(&full_bar[s], (uint32_t)(GROUPS ? DTC_A_BYTES + boxes * box * DTC_BK * 2 : stage_bytes));
                         tc_tma_load_2d(a, &tmap_w, k * DTC_BK, n0, &full_bar[s]);
+                        if (GROUPS)
+                            for (int x = 0; x < boxes; ++x) tc_tma_load_2d(a + DTC_A_BYTES + x * box * DTC_BK * 2, &tmap_x, k * DTC_BK, m0 + x * box, &full_bar[s]);
                     }
-                    tc_tma_load_2d(a + DTC_A_BYTES, &tmap_x, k * DTC_BK, m0, &full_bar[s]);
+                    if (!GROUPS) tc_tma_load_2d(a + DTC_A_BYTES, &tmap_x, k * DTC_BK, m0, &full_bar[s]);
                 }
             }
             skn_pdl_launch_dependents();           // every load of this CTA is on its way: the next launch may come in
@@ -814,15 +887,16 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                     ok = false;
                 }
         }
-    } else if (warp == 4) {
+    } else if (warp == DTC_MMA) {
         if (lane == 0) {
-            const uint32_t idesc = tc_idesc(DTC_BM, NT);
+            uint32_t idesc = tc_idesc(DTC_BM, NT);
             bool ok = true;
             int it = 0, tile = 0;
             for (int u = blockIdx.x; u < units && ok; u += gridDim.x, ++tile) {
                 const int sp = GROUPS ? 0 : (u / mt) % splits;
                 const int kb = (int)((int64_t)ksteps * sp / splits), ke = (int)((int64_t)ksteps * (sp + 1) / splits);
                 const int b = tile & 1;
+                if (GROUPS) idesc = tc_idesc(DTC_BM, max(16, (tile_of(u).cols + 15) / 16 * 16));
                 if (!skn_mbar_wait(&acc_empty[b], ((uint32_t)(tile >> 1) & 1u) ^ 1u)) {
                     atomicExch(status, SKN_ERR_TIMEOUT);
                     break;
@@ -859,13 +933,14 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 ok = false;
             }
             tc_fence_after();
-            const int n = n0 + warp * 32 + lane;
+            const int quarter = warp & 3, second = warp >> 2;       // the two warps of a quarter take turns by 32 tokens
+            const int n = n0 + quarter * 32 + lane;
             const int cols = tl.cols;
-            const uint32_t src = tmem + (uint32_t)(b * acc_cols) + ((uint32_t)(warp * 32) << 16);
+            const uint32_t src = tmem + (uint32_t)(b * acc_cols) + ((uint32_t)(quarter * 32) << 16);
             const int tidx = nti * mt + u % mt;
-            float *pbase = partial + ((size_t)tidx * splits) * NT * DTC_BM + warp * 32 + lane;
+            float *pbase = partial + ((size_t)tidx * splits) * NT * DTC_BM + quarter * 32 + lane;
 #pragma unroll 1
-            for (int c0 = 0; c0 < cols; c0 += 32) {
+            for (int c0 = second * 32; c0 < cols; c0 += 64) {
                 uint32_t acc[32];
                 tc_ld32(src + c0, acc);
                 if (splits == 1) {
@@ -897,7 +972,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 dtc_barrier_epilogue();
                 if (last_flag) {
                     __threadfence();
-                    for (int c0 = 0; c0 < cols; c0 += 16) {
+                    for (int c0 = second * 16; c0 < cols; c0 += 32) {
                         float v[16];
 #pragma unroll
                         for (int c = 0; c < 16; ++c) v[c] = 0.f;
@@ -916,7 +991,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     }
     tc_fence_before();
     __syncthreads();
-    if (warp == 4) {
+    if (warp == DTC_MMA) {
         __syncwarp();
         tc_fence_after();
         tc_dealloc(tmem, tmem_cols);
@@ -940,7 +1015,7 @@ static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense
     int NT = 16;
     if (GROUPS) {
         // tiles that an expert's share of the rows fills about once
-        while (NT < 128 && NT * l.pick.n < M + M / 4) NT *= 2;
+        while (NT < 256 && NT * l.pick.n < M + M / 4) NT *= 2;
     } else if (M <= 128) {
         while (NT < M) NT *= 2;
     } else {
@@ -979,7 +1054,7 @@ static cudaError_t launch_dtc(skn_ctx *ctx, const skn_linear &l, const skn_dense
     if (stages > DTC_MAX_STAGES) stages = DTC_MAX_STAGES;
     CUtensorMap tw, tx;
     cudaError_t e = skn_tmap_bf16(l.w->d_blocks, l.w->n_rows, K, l.w->pitch, DTC_BM, &tw);
-    if (e == cudaSuccess) e = skn_tmap_bf16(l.x16, M, K, l.ld_x16 * 2, NT, &tx);
+    if (e == cudaSuccess) e = skn_tmap_bf16(l.x16, M, K, l.ld_x16 * 2, GROUPS && NT > DTC_GROUP_BOX ? DTC_GROUP_BOX : NT, &tx);
     if (e != cudaSuccess) return e;
     const int units = mt * nt * splits;
     return skn_launch_pdl(kern, dim3(units < sms ? units : sms), dim3(DTC_THREADS), (size_t)stages * stage_bytes + 1024, st, 1, tw, tx, N, K, M, NT,

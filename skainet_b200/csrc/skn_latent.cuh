@@ -23,7 +23,7 @@ struct skn_latent_args {
     skn_route_args route;           // rides along in the absorbed form's first launch
     float *q;                       // [rows][heads][dim + rp], before rotation
     float *ql, *ol;                 // absorbed: [rows][heads][kvp + rp], [rows][heads][kvp]
-    float *scratch;                 // skn_attn_scratch() floats
+    float *scratch;                 // skn_latent_scratch() floats
     unsigned *tickets;
     float *cq32;                    // normalised query latents, [rows][q_rank rounded up to 8]
     __nv_bfloat16 *cq16;
@@ -31,6 +31,8 @@ struct skn_latent_args {
     __nv_bfloat16 *kvx;             // expanded: [ring slots][heads * (dim + vdim)]
 };
 
+// floats of scratch for the absorbed form of up to `rows` rows
+size_t skn_latent_scratch(const skn_latent_args &a, int rows, int max_pos);
 bool skn_latent_expand_fits(const skn_latent_args &a);
 // The newest latents and rotated keys into the cache, and the normalised query latents to cq (either form, where given)
 cudaError_t skn_launch_latent_rows(const skn_step &s, const skn_latent_args &a, const skn_rows_out &cq, cudaStream_t st);

@@ -22,6 +22,7 @@ skn_group_pairs_kernel(const int32_t *expert, int pairs, int experts, int32_t *o
     skn_pdl_wait();
     const int e = blockIdx.x, tid = threadIdx.x, per = (pairs + 255) / 256, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
     int lo = 0, eq = 0;
+#pragma unroll 8
     for (int i = i0; i < i1; ++i) {
         const int v = __ldcg(expert + i);
         lo += v < e;
@@ -58,6 +59,7 @@ skn_group_pairs_kernel(const int32_t *expert, int pairs, int experts, int32_t *o
     }
     __syncthreads();
     int at = base_s + own[tid];
+#pragma unroll 8
     for (int i = i0; i < i1; ++i)
         if (__ldcg(expert + i) == e) place[i] = at++;
 }

@@ -7,8 +7,8 @@
 //  skn_ssm_scan_kernel    states at the chunk starts and after the step; files the convolution's last inputs
 //  skn_ssm_out_kernel     y_i = sum_{j <= i} exp(cum_i - cum_j) dt_j (C_i . B_j) x_j + exp(cum_i) S^T C_i + D x_i, times silu(z)
 //
-// In the chunk kernels x, B and C are bf16 and enter the tensor cores exactly; decays, weights and states are fp32 and enter as three
-// bf16 terms each (24 bits), summed in fp32.
+// In the chunk kernels x, B and C are bf16 and enter the tensor cores exactly, sums are fp32.  What is added to the state enters as three bf16
+// terms (24 bits); in the outputs, which only read the state, weights and states enter as two (16 bits), as softmax weights do.
 #include "skn_ssm.cuh"
 #include "skn_mma.cuh"
 
@@ -222,21 +222,21 @@ skn_ssm_conv_kernel(skn_ssm_args a, skn_step st, const float *ring_, int ring_pi
         return v;
     };
     if constexpr (TAPS > 0) {
-        float4 w[TAPS], u[TAPS];
+        // every input of the run is loaded before the first output is stored
+        float4 w[TAPS], u[CV_TOKENS + TAPS - 1];
 #pragma unroll
         for (int k = 0; k < TAPS; ++k) w[k] = __ldg(reinterpret_cast<const float4 *>(a.conv + (int64_t)k * channels + c));
 #pragma unroll
-        for (int k = 0; k < TAPS - 1; ++k) u[k + 1] = load(t0 - (TAPS - 1) + k);
+        for (int i = 0; i < CV_TOKENS + TAPS - 1; ++i) {
+            const int t = t0 - (TAPS - 1) + i;
+            u[i] = t < t1 ? load(t) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
 #pragma unroll
         for (int i = 0; i < CV_TOKENS; ++i) {
-            if (t0 + i >= t1) break;
-#pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k) u[k] = u[k + 1];
-            u[TAPS - 1] = load(t0 + i);
             float4 v = b;
 #pragma unroll
-            for (int k = 0; k < TAPS; ++k) v = fma4(w[k], u[k], v);
-            put(t0 + i, v);
+            for (int k = 0; k < TAPS; ++k) v = fma4(w[k], u[i + k], v);
+            if (t0 + i < t1) put(t0 + i, v);
         }
     } else {
         for (int t = t0; t < t1; ++t) {
@@ -257,13 +257,14 @@ __device__ __forceinline__ void ssm_load_rows(__nv_bfloat16 *dst, int stride, co
     }
 }
 
-// three bf16 terms of (a, b), packed
-__device__ __forceinline__ void three_terms(float a, float b, uint32_t (&o)[3]) {
-    o[0] = pack_bf16(a, b);
-    less_bf16(a, b, o[0]);
-    o[1] = pack_bf16(a, b);
-    less_bf16(a, b, o[1]);
-    o[2] = pack_bf16(a, b);
+// the first N bf16 terms of (a, b), packed
+template <int N>
+__device__ __forceinline__ void bf16_terms(float a, float b, uint32_t (&o)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        o[i] = pack_bf16(a, b);
+        if (i + 1 < N) less_bf16(a, b, o[i]);
+    }
 }
 
 __host__ __device__ constexpr int up16(int n) { return (n + 15) / 16 * 16; }
@@ -288,21 +289,34 @@ skn_ssm_chunk_kernel(skn_ssm_args a, int T, int nchunks, int per) {
     const __nv_bfloat16 *rows = a.xbc + row0 * channels;
     ssm_load_rows(B, bs, rows + inner + g * a.np, channels, L, a.np, np16);
     asm volatile("cp.async.commit_group;" ::: "memory");
+    // a head's x: PX pieces of 8 elements per thread, fetched while the head before is multiplied
+    constexpr int PX = SC * (DV / 8) / 128;
+    uint4 pre[PX];
+    auto fetch = [&](int h) {
+#pragma unroll
+        for (int i = 0; i < PX; ++i) {
+            const int at = tid + i * 128, t = at / (DV / 8), v = at % (DV / 8) * 8;
+            pre[i] = t < L && v < a.vp ? __ldcg(reinterpret_cast<const uint4 *>(rows + (int64_t)t * channels + h * a.vp + v)) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    };
+    fetch(h0);
     for (int h = h0; h < h0 + per; ++h) {
         if (tid < SC) wj[tid] = tid < L ? __expf(a.cum[(row0 + L - 1) * a.heads + h] - a.cum[(row0 + tid) * a.heads + h]) * a.dt[(row0 + tid) * a.heads + h] : 0.f;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        for (int i = tid; i < SC * (DV / 2); i += 128) {
-            const int t = i / (DV / 2), v = i % (DV / 2) * 2;
-            uint32_t o[3] = {0u, 0u, 0u};
-            if (t < L && v < a.vp) {
-                const uint32_t w = *reinterpret_cast<const uint32_t *>(rows + (int64_t)t * channels + h * a.vp + v);
-                three_terms(__uint_as_float(w << 16) * wj[t], __uint_as_float(w & 0xFFFF0000u) * wj[t], o);
-            }
 #pragma unroll
-            for (int x = 0; x < 3; ++x) *reinterpret_cast<uint32_t *>(X + ((size_t)x * SC + t) * xs + v) = o[x];
+        for (int i = 0; i < PX; ++i) {
+            const int at = tid + i * 128, t = at / (DV / 8), v = at % (DV / 8) * 8;
+            const uint32_t in[4] = {pre[i].x, pre[i].y, pre[i].z, pre[i].w};
+            const float w = wj[t];
+            uint32_t o[4][3];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) bf16_terms<3>(__uint_as_float(in[e] << 16) * w, __uint_as_float(in[e] & 0xFFFF0000u) * w, o[e]);
+#pragma unroll
+            for (int x = 0; x < 3; ++x) *reinterpret_cast<uint4 *>(X + ((size_t)x * SC + t) * xs + v) = make_uint4(o[0][x], o[1][x], o[2][x], o[3][x]);
         }
         __syncthreads();
+        if (h + 1 < h0 + per) fetch(h + 1);
         float *out = a.chunks + ((((int64_t)seq * nchunks + c) * a.heads + h) * a.np) * a.vp;
         for (int mt = warp; mt < np16 / 16; mt += 4) {
             float acc[DV / 8][4];
@@ -337,7 +351,7 @@ skn_ssm_chunk_kernel(skn_ssm_args a, int T, int nchunks, int per) {
     }
 }
 
-// chunk sums -> states at the chunk starts (in place), and the state after the step; CTAs from `blocks` on file the convolution's inputs
+// chunk sums -> states at the chunk starts (two bf16 terms), and the state after the step; CTAs from `blocks` on file the convolution's inputs
 __global__ void __launch_bounds__(128)
 skn_ssm_scan_kernel(skn_ssm_args a, skn_step st, float *S_, float *ring, int ring_pitch, int nchunks, int blocks) {
     skn_pdl_launch_dependents();
@@ -350,7 +364,9 @@ skn_ssm_scan_kernel(skn_ssm_args a, skn_step st, float *S_, float *ring, int rin
     const int64_t head = (int64_t)a.np * (a.vp / 4), per = a.heads * head, i = (int64_t)blockIdx.x * 128 + threadIdx.x;
     if (i >= per) return;
     const int h = (int)(i / head);
-    float4 *p = reinterpret_cast<float4 *>(a.chunks) + (int64_t)seq * nchunks * per + i;
+    const float4 *p = reinterpret_cast<const float4 *>(a.chunks) + (int64_t)seq * nchunks * per + i;
+    // term planes [np][vp] of a head behind one another
+    uint2 *start = reinterpret_cast<uint2 *>(a.starts) + ((int64_t)seq * nchunks * a.heads + h) * 2 * head + i % head;
     float4 *sp = reinterpret_cast<float4 *>(S_) + (int64_t)slot * per + i;
     float4 s = st.pos[slot] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
     const float *cum = a.cum + (int64_t)seq * T * a.heads + h;
@@ -366,7 +382,12 @@ skn_ssm_scan_kernel(skn_ssm_args a, skn_step st, float *S_, float *ring, int rin
 #pragma unroll
         for (int u = 0; u < 8; ++u)
             if (c0 + u < nchunks) {
-                __stcg(p + (int64_t)(c0 + u) * per, s);
+                uint32_t lo[2], hi[2];
+                bf16_terms<2>(s.x, s.y, lo);
+                bf16_terms<2>(s.z, s.w, hi);
+                uint2 *q = start + (int64_t)(c0 + u) * per * 2;
+                __stcg(q, make_uint2(lo[0], hi[0]));
+                __stcg(q + head, make_uint2(lo[1], hi[1]));
                 const float f = __expf(d[u]);
                 s = make_float4(fmaf(f, s.x, v[u].x), fmaf(f, s.y, v[u].y), fmaf(f, s.z, v[u].z), fmaf(f, s.w, v[u].w));
             }
@@ -374,8 +395,11 @@ skn_ssm_scan_kernel(skn_ssm_args a, skn_step st, float *S_, float *ring, int rin
     *sp = s;
 }
 
-// smem (bf16): B, C [SC][np16 + 8] | x [SC][DV + 8] | state, three terms [3][np16][DV + 8]
-static size_t ssm_out_smem(int np, int DV) { return ((size_t)2 * SC * (up16(np) + 8) + (size_t)SC * (DV + 8) + (size_t)3 * up16(np) * (DV + 8)) * 2; }
+// smem (bf16): C [SC][np16 + 8] | x [SC][DV + 8] | state, two terms [2][np16][DV + 8], before them B [SC][np16 + 8] in the same place
+static size_t ssm_out_smem(int np, int DV) {
+    const size_t state = (size_t)2 * up16(np) * (DV + 8), b = (size_t)SC * (up16(np) + 8);
+    return ((size_t)SC * (up16(np) + 8) + (size_t)SC * (DV + 8) + (state > b ? state : b)) * 2;
+}
 
 template <int DV>
 __global__ void __launch_bounds__(128)
@@ -385,7 +409,7 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
     skn_pdl_launch_dependents();
     skn_pdl_wait();
     const int np16 = up16(a.np), bs = np16 + 8, xs = DV + 8;
-    __nv_bfloat16 *B = reinterpret_cast<__nv_bfloat16 *>(smb), *C = B + SC * bs, *X = C + SC * bs, *St = X + SC * xs;
+    __nv_bfloat16 *C = reinterpret_cast<__nv_bfloat16 *>(smb), *X = C + SC * bs, *St = X + SC * xs, *B = St;
     const int c = blockIdx.x, h0 = blockIdx.y * per, seq = blockIdx.z, t0 = c * SC, L = min(SC, T - t0);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int channels = skn_ssm_channels(a.heads, a.vp, a.groups, a.np), inner = a.heads * a.vp, g = h0 / (a.heads / a.groups);
@@ -422,17 +446,13 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
             cum_s[tid] = a.cum[at];
             dt_s[tid] = tid < L ? a.dt[at] : 0.f;
         }
-        const float *S = a.chunks + ((((int64_t)seq * nchunks + c) * a.heads + h) * a.np) * a.vp;
-#pragma unroll 4
-        for (int i = tid; i < np16 * (DV / 4); i += 128) {
-            const int n = i / (DV / 4), v = i % (DV / 4) * 4;
-            const float4 f = n < a.np && v < a.vp ? __ldcg(reinterpret_cast<const float4 *>(S + (int64_t)n * a.vp + v)) : make_float4(0.f, 0.f, 0.f, 0.f);
-            uint32_t lo[3], hi[3];
-            three_terms(f.x, f.y, lo);
-            three_terms(f.z, f.w, hi);
-#pragma unroll
-            for (int x = 0; x < 3; ++x) *reinterpret_cast<uint2 *>(St + ((size_t)x * np16 + n) * xs + v) = make_uint2(lo[x], hi[x]);
+        const __nv_bfloat16 *S = a.starts + (((int64_t)seq * nchunks + c) * a.heads + h) * 2 * a.np * a.vp;
+        for (int i = tid; i < 2 * np16 * (DV / 8); i += 128) {
+            const int x = i / (np16 * (DV / 8)), n = i / (DV / 8) % np16, v = i % (DV / 8) * 8;
+            const bool in = n < a.np && v < a.vp;
+            cp_async16(skn_smem_u32(St + ((size_t)x * np16 + n) * xs + v), in ? S + ((int64_t)x * a.np + n) * a.vp + v : S, in);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         float o[DV / 8][4];
@@ -442,7 +462,7 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
             uint32_t af[4];
             ldsm4(af, skn_smem_u32(C + (size_t)(m0 + (lane & 15)) * bs + kk + (lane >> 4) * 8));
 #pragma unroll
-            for (int x = 2; x >= 0; --x)
+            for (int x = 1; x >= 0; --x)
 #pragma unroll
                 for (int n = 0; n < DV / 16; ++n) {
                     uint32_t bf[4];
@@ -460,23 +480,23 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
 #pragma unroll
         for (int kk = 0; kk < SC / 16; ++kk) {
             if (kk > warp) continue;
-            uint32_t pf[3][4];
+            uint32_t pf[2][4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int nt = 2 * kk + (x >> 1), r = x & 1, i = m0 + gr + r * 8, j = nt * 8 + gc;
                 const float p0 = j <= i ? s[nt][r * 2] * __expf(ci[r] - cum_s[j]) * dt_s[j] : 0.f;
                 const float p1 = j + 1 <= i ? s[nt][r * 2 + 1] * __expf(ci[r] - cum_s[j + 1]) * dt_s[j + 1] : 0.f;
-                uint32_t t3[3];
-                three_terms(p0, p1, t3);
-#pragma unroll
-                for (int y = 0; y < 3; ++y) pf[y][x] = t3[y];
+                uint32_t t2[2];
+                bf16_terms<2>(p0, p1, t2);
+                pf[0][x] = t2[0];
+                pf[1][x] = t2[1];
             }
 #pragma unroll
             for (int n = 0; n < DV / 16; ++n) {
                 uint32_t bf[4];
                 ldsm4t(bf, skn_smem_u32(X + (size_t)(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * xs + n * 16 + (lane >> 4) * 8));
 #pragma unroll
-                for (int y = 2; y >= 0; --y) {
+                for (int y = 1; y >= 0; --y) {
                     mma_bf16(o[2 * n], pf[y], bf[0], bf[1]);
                     mma_bf16(o[2 * n + 1], pf[y], bf[2], bf[3]);
                 }

@@ -24,7 +24,8 @@ struct skn_ssm_args {
     // many-token form
     __nv_bfloat16 *xbc;                 // [rows][channels]
     float *dt, *cum;                    // [rows][heads]: step sizes, and the log decays summed from the chunk's start
-    float *chunks;                      // [seqs][chunks][heads][np][vp]
+    float *chunks;                      // what each chunk adds to the state: [seqs][chunks][heads][np][vp]
+    __nv_bfloat16 *starts;              // the states at the chunk starts: [seqs][chunks][heads][2 terms][np][vp]
 };
 __host__ __device__ static inline int skn_ssm_channels(int heads, int vp, int groups, int np) { return heads * vp + 2 * groups * np; }
 

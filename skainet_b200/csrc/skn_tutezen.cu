@@ -45,6 +45,7 @@ struct Tutezen : skn_decoder {
     // state space
     __nv_bfloat16 *xbc;
     float *dt, *cum, *chunks;
+    __nv_bfloat16 *starts;
     // latent attention
     int64_t ldc;
     float *q, *ql, *ol, *scratch, *cq32;
@@ -135,13 +136,13 @@ static cudaError_t allocate(Tutezen *m) {
             const skn_kvcache *kv = m->caches[m->cache_of[i]];
             grow(C, (int64_t)l.qr);
             skn_latent_args la = {};
-            la.kv = kv; la.dim = l.dim; la.rp = l.rp; la.vdim = l.vp;
+            la.kv = kv; la.heads = a.heads; la.dim = l.dim; la.rp = l.rp; la.vdim = l.vp; la.kvp = l.kvp; la.window = a.window;
             const bool expand = skn_latent_expand_fits(la);
             const size_t rows = expand ? short_rows : R;             // rows that meet the absorbed form
             grow(q, rows * a.heads * (l.dim + l.rp));
             grow(ql, rows * a.heads * (l.kvp + l.rp));
             grow(ol, rows * a.heads * l.kvp);
-            grow(scratch, skn_attn_scratch((int)rows, a.heads, l.kvp, a.window, m->max_ctx));
+            grow(scratch, skn_latent_scratch(la, (int)rows, m->max_ctx));
             grow(tick, rows * a.heads);
             if (expand) {
                 grow(q16, R * a.heads * (l.dim + l.rp));
@@ -160,7 +161,7 @@ static cudaError_t allocate(Tutezen *m) {
 #define TUT_TAKE(p, n) if (e == cudaSuccess) e = m->take(&m->p, n)
     TUT_TAKE(x, R * m->ldw); TUT_TAKE(x0, m->passes > 1 ? R * m->ldw : 0); TUT_TAKE(step, (size_t)m->passes * m->width);
     TUT_TAKE(proj, R * P); TUT_TAKE(mix32, r32 * X); TUT_TAKE(mix16, r16 * X); TUT_TAKE(y, R * Y);
-    TUT_TAKE(xbc, xbc); TUT_TAKE(dt, heads); TUT_TAKE(cum, heads); TUT_TAKE(chunks, chunks);
+    TUT_TAKE(xbc, xbc); TUT_TAKE(dt, heads); TUT_TAKE(cum, heads); TUT_TAKE(chunks, chunks); TUT_TAKE(starts, 2 * chunks);
     TUT_TAKE(q, q); TUT_TAKE(ql, ql); TUT_TAKE(ol, ol); TUT_TAKE(scratch, scratch); TUT_TAKE(tickets, tick);
     TUT_TAKE(cq32, C ? r32 * C : 0); TUT_TAKE(cq16, C ? r16 * C : 0); TUT_TAKE(q16, q16); TUT_TAKE(kvx, kvx);
     TUT_TAKE(expert, pairs); TUT_TAKE(weight, pairs); TUT_TAKE(place, pairs); TUT_TAKE(offset, experts ? experts + 1 : 0);
@@ -192,7 +193,7 @@ int32_t Tutezen::ssm_mixer(const Layer &l, const skn_step &st, int run, bool few
     a.heads = s.heads; a.vp = l.vp; a.np = l.np; a.groups = s.groups; a.taps = s.taps;
     a.conv = l.conv; a.conv_b = l.conv_b; a.dt_bias = l.dt_bias; a.a = l.a; a.d = l.d;
     a.proj = proj; a.ld = ldp;
-    a.xbc = xbc; a.dt = dt; a.cum = cum; a.chunks = chunks;
+    a.xbc = xbc; a.dt = dt; a.cum = cum; a.chunks = chunks; a.starts = starts;
     if (few_rows) {
         a.y = mix32; a.ld_y = ldm;
         a.route = route;
