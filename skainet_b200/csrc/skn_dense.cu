@@ -193,7 +193,8 @@ __device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 
 // CTA b owns the weight rows [b N / grid, (b + 1) N / grid): a producer warp streams them, a few rows per bulk copy, through
 // a ring of shared-memory stages and starts before the kernel waits for its predecessor; eight warps each take an eighth of
 // the columns of every row.  Their partial sums meet in shared memory, 128 rows at a time.  One activation row lives in
-// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).  PICK: the weight rows, or pieces of
+// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).  Rows longer than the registers hold are taken in
+// column pieces, one after the other for all rows of the CTA (at most MVD_ROWS then), the partial sums waiting in shared memory.  PICK: the weight rows, or pieces of
 // them, belong to experts that a kernel before chose, so the stream of those starts after the dependency wait.
 constexpr int MVD_WARPS = 8, MVD_THREADS = (MVD_WARPS + 1) * 32, MVD_ROWS = 128;
 constexpr int MVD_RING = 96 * 1024, MVD_MAX_STAGES = 24;
@@ -228,7 +229,6 @@ struct mvd_pick {
     int64_t pitch2;
     int n, rows_per;
 };
-constexpr int MVD_PICKS = 64;           // experts whose numbers are kept in shared memory
 struct mvd_norm {
     const float *gain;
     float eps;
@@ -237,17 +237,16 @@ struct mvd_norm {
 
 template <int MR, int UU, int PICK>
 __global__ void __launch_bounds__(MVD_THREADS, 2)
-skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitch, int N, int K, int m0, const float *x, int64_t ldx, const float *xb,
-                        int64_t ldxb, int ka, mvd_norm nm, mvd_pick pk, int stages, skn_epi e, int32_t *status) {
+skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_bytes, int pieces, int64_t pitch, int N, int K, int m0, const float *x,
+                        int64_t ldx, const float *xb, int64_t ldxb, int ka, mvd_norm nm, mvd_pick pk, int stages, skn_epi e, int32_t *status) {
     extern __shared__ __align__(128) uint8_t ring[];
     constexpr int GR = mvd_stage_rows(MR, UU);
     __shared__ uint64_t full_bar[MVD_MAX_STAGES], empty_bar[MVD_MAX_STAGES];
-    __shared__ int picks[PICK != SKN_PICK_NONE ? MVD_PICKS : 1];
     __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS], psum[MR][MVD_WARPS][SKN_NORM_PARTS];
     const float *__restrict__ gain = nm.gain;
     const bool pairs = skn_epi_pairs(e.kind), partial = gain && nm.cols > 0;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2, per = (nv + MVD_WARPS - 1) / MVD_WARPS;
+    const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2;           // vectors of a piece (of the row, when there is one)
     const int q_rows = pairs ? 2 : 1, nq = (N + q_rows - 1) / q_rows;     // pairs of rows stay together
     const int r0 = min(N, q_rows * (int)((int64_t)nq * blockIdx.x / gridDim.x)), r1 = min(N, q_rows * (int)((int64_t)nq * (blockIdx.x + 1) / gridDim.x));
     const int steps = (r1 - r0 + GR - 1) / GR;
@@ -261,51 +260,55 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
     }
     __syncthreads();
     if (warp == MVD_WARPS) {
-        if (lane == 0) {
-            int s = 0;
-            uint32_t phase = 1;
-            int early = 0;
-            if constexpr (PICK == SKN_PICK_COLS) {
-                // the first stages' own pieces depend on no kernel before this one
-                for (; pk.pitch1 && early < stages && early < steps; ++early) {
-                    const int row = r0 + early * GR, n = min(GR, r1 - row);
-                    skn_mbar_expect_tx(&full_bar[early], (uint32_t)(n * pitch));
-                    for (int j = 0; j < n; ++j)
-                        skn_bulk_g2s(ring + early * stage_bytes + j * pitch, W + (row + j) * wld, (uint32_t)pk.pitch1, &full_bar[early]);
+        // lane 0 keeps the ring; the copies of a stage are issued by as many lanes as there are pieces of rows in it
+        int s = 0, early = 0;
+        uint32_t phase = 1;
+        const int64_t own = PICK == SKN_PICK_COLS ? pk.pitch1 : row_bytes;
+        if constexpr (PICK == SKN_PICK_COLS) {
+            // w's part of the first stages depends on no kernel before this one
+            const int64_t first = min(pitch, row_bytes), n_own = min(first, own);
+            for (; early < stages && early < steps; ++early) {
+                const int row = r0 + early * GR, n = min(GR, r1 - row);
+                if (lane == 0) skn_mbar_expect_tx(&full_bar[early], (uint32_t)(n * first));
+                __syncwarp();
+                if (lane < n) skn_bulk_g2s(ring + early * stage_bytes + lane * pitch, W + (row + lane) * wld, (uint32_t)n_own, &full_bar[early]);
+            }
+        }
+        if constexpr (PICK != SKN_PICK_NONE) skn_pdl_wait();
+        for (int i = 0, pc = 0; pc < pieces; ++pc) {
+            const int64_t lo = pc * pitch, hi = min(row_bytes, lo + pitch);
+            for (int g = 0; g < steps; ++g, ++i) {
+                const int row = r0 + g * GR, n = min(GR, r1 - row);
+                int good = 1;
+                if (lane == 0 && i >= early) {
+                    good = skn_mbar_wait(&empty_bar[s], phase);
+                    if (good) skn_mbar_expect_tx(&full_bar[s], (uint32_t)(n * (hi - lo)));
+                    else atomicExch(status, SKN_ERR_TIMEOUT);
                 }
-            }
-            if constexpr (PICK != SKN_PICK_NONE) {
-                skn_pdl_wait();
-                for (int x = 0; x < min(pk.n, MVD_PICKS); ++x) picks[x] = __ldcg(pk.expert + x);
-            }
-            auto picked = [&](int x) { return (int64_t)(x < MVD_PICKS ? picks[x] : __ldcg(pk.expert + x)); };
-            for (int i = 0; i < steps; ++i) {
-                const int row = r0 + i * GR;
-                if (i >= early && !skn_mbar_wait(&empty_bar[s], phase)) {
-                    atomicExch(status, SKN_ERR_TIMEOUT);
+                if (!__shfl_sync(0xffffffffu, good, 0)) {
+                    pc = pieces;
                     break;
                 }
-                const int n = min(GR, r1 - row);
-                const uint32_t bytes = (uint32_t)(n * pitch);
-                if (i >= early) skn_mbar_expect_tx(&full_bar[s], bytes);
                 uint8_t *dst = ring + s * stage_bytes;
                 if constexpr (PICK == SKN_PICK_NONE) {
-                    if (wld == pitch) skn_bulk_g2s(dst, W + row * wld, bytes, &full_bar[s]);
-                    else
-                        for (int j = 0; j < n; ++j) skn_bulk_g2s(dst + j * pitch, W + (row + j) * wld, (uint32_t)pitch, &full_bar[s]);
+                    if (wld == hi - lo) {
+                        if (lane == 0) skn_bulk_g2s(dst, W + row * wld, (uint32_t)(n * wld), &full_bar[s]);
+                    } else if (lane < n) {
+                        skn_bulk_g2s(dst + lane * pitch, W + (row + lane) * wld + lo, (uint32_t)(hi - lo), &full_bar[s]);
+                    }
                 } else if constexpr (PICK == SKN_PICK_ROWS) {
-                    for (int j = 0; j < n; ++j) {
-                        const int r = row + j, x = r / pk.rows_per;
-                        skn_bulk_g2s(dst + j * pitch, W + (picked(x) * pk.rows_per + r - x * pk.rows_per) * wld, (uint32_t)pitch, &full_bar[s]);
+                    if (lane < n) {
+                        const int r = row + lane, x = r / pk.rows_per;
+                        skn_bulk_g2s(dst + lane * pitch, W + ((int64_t)__ldcg(pk.expert + x) * pk.rows_per + r - x * pk.rows_per) * wld, (uint32_t)pitch, &full_bar[s]);
                     }
                 } else {
-                    for (int j = 0; j < n; ++j) {
-                        const int r = row + j;
-                        uint8_t *d = dst + j * pitch;
-                        if (i >= early && pk.pitch1) skn_bulk_g2s(d, W + r * wld, (uint32_t)pk.pitch1, &full_bar[s]);
-                        d += pk.pitch1;
-                        for (int x = 0; x < pk.n; ++x, d += pk.pitch2)
-                            skn_bulk_g2s(d, pk.w2 + (picked(x) * N + r) * pk.pitch2, (uint32_t)pk.pitch2, &full_bar[s]);
+                    // segment 0 of a joint row is w's, segment x + 1 belongs to the picked expert x
+                    for (int u = lane; u < n * (pk.n + 1); u += 32) {
+                        const int jr = u / (pk.n + 1), x = u % (pk.n + 1) - 1;
+                        const int64_t s0 = x < 0 ? 0 : own + x * pk.pitch2, s1 = x < 0 ? own : s0 + pk.pitch2, a = max(lo, s0), b = min(hi, s1);
+                        if (a >= b || (x < 0 && i < early)) continue;
+                        const uint8_t *src = x < 0 ? W + (row + jr) * wld : pk.w2 + ((int64_t)__ldcg(pk.expert + x) * N + row + jr) * pk.pitch2;
+                        skn_bulk_g2s(dst + jr * pitch + (a - lo), src + (a - s0), (uint32_t)(b - a), &full_bar[s]);
                     }
                 }
                 if (++s == stages) {
@@ -319,8 +322,14 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
     }
     skn_pdl_wait();
 
-    // this warp's columns: vectors v0 + lane + 32 u below v1
-    const int v0 = warp * per, v1 = min(nv, v0 + per);
+    bool ok = true;
+    int buf = 0, filled = 0, base = r0;            // rows base .. base + filled - 1 have partial sums in part[buf]
+    int s = 0;
+    uint32_t phase = 0;
+    const uint4 *w = reinterpret_cast<const uint4 *>(ring);
+    for (int pc = 0; pc < pieces; ++pc) {
+    // this warp's columns: vectors v0 + lane + 32 u below v1 of the piece, which starts at vector vb of the row
+    const int vb = pc * nv, nvp = min(nv, (int)(row_bytes >> 4) - vb), per = (nvp + MVD_WARPS - 1) / MVD_WARPS, v0 = warp * per, v1 = min(nvp, v0 + per);
     float4 xr[UU > 0 ? 2 * UU : 1];
     float *xs = reinterpret_cast<float *>(ring + stages * stage_bytes);     // UU = 0: [MR][2 planes][K8 / 2]: quads 0 and 1 of every eight columns
     float ss[MR];
@@ -338,7 +347,7 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             const int i = v0 + u * 32 + lane;
             vsq[u] = 0.f;
             float f[8];
-            const int k = i * 8;
+            const int k = (vb + i) * 8;
             if (vec && i < v1) {
                 const float *p = k < ka ? x + (int64_t)m0 * ldx + k : xb + (int64_t)m0 * ldxb + k - ka;
                 *reinterpret_cast<float4 *>(f) = __ldcg(reinterpret_cast<const float4 *>(p));
@@ -365,7 +374,7 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             xr[2 * u + 1] = make_float4(f[4], f[5], f[6], f[7]);
         }
         ss[0] = q;
-        if (partial) {
+        if (partial && pc == 0) {
             const int pv = nm.cols / nm.parts / 8;                     // vectors of a part
             for (int p = 0; p < nm.parts; ++p) {
                 float t = 0.f;
@@ -391,13 +400,13 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             }
         }
         if (partial) {
-            const int pc = nm.cols / nm.parts;
+            const int part_cols = nm.cols / nm.parts;
             mvd_barrier();
 #pragma unroll
             for (int m = 0; m < MR; ++m)
                 for (int p = 0; p < nm.parts; ++p) {
                     float t = 0.f;
-                    for (int k = p * pc + threadIdx.x; k < (p + 1) * pc; k += MVD_WARPS * 32) {
+                    for (int k = p * part_cols + threadIdx.x; k < (p + 1) * part_cols; k += MVD_WARPS * 32) {
                         const float v = xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)];
                         t = fmaf(v, v, t);
                     }
@@ -425,20 +434,20 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             rs[m] = 1.f / sqrtf(t / (float)K + nm.eps);
         }
     }
-    if (partial) {
-        const int pc = nm.cols / nm.parts;
+    if (partial && pc == 0) {                       // (the parts lie in the first piece)
+        const int part_cols = nm.cols / nm.parts;
         auto scale = [&](int m, int p) {
             float t = 0.f;
 #pragma unroll
             for (int w = 0; w < MVD_WARPS; ++w) t += psum[m][w][p];
-            return 1.f / sqrtf(t / (float)pc + nm.eps);
+            return 1.f / sqrtf(t / (float)part_cols + nm.eps);
         };
         if constexpr (UU > 0) {
 #pragma unroll
             for (int u = 0; u < UU; ++u) {
                 const int k = (v0 + u * 32 + lane) * 8;
                 if (k < nm.cols) {
-                    const float f = scale(0, k / pc);
+                    const float f = scale(0, k / part_cols);
                     xr[2 * u].x *= f; xr[2 * u].y *= f; xr[2 * u].z *= f; xr[2 * u].w *= f;
                     xr[2 * u + 1].x *= f; xr[2 * u + 1].y *= f; xr[2 * u + 1].z *= f; xr[2 * u + 1].w *= f;
                 }
@@ -448,7 +457,7 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             for (int m = 0; m < MR; ++m)
                 for (int p = 0; p < nm.parts; ++p) {
                     const float f = scale(m, p);
-                    for (int k = p * pc + threadIdx.x; k < (p + 1) * pc; k += MVD_WARPS * 32)
+                    for (int k = p * part_cols + threadIdx.x; k < (p + 1) * part_cols; k += MVD_WARPS * 32)
                         xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] *= f * __ldg(gain + k);
                 }
             mvd_barrier();
@@ -456,11 +465,8 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
     }
 
     // eight rows at a time: their sums are reduced across the warp together (9 shuffles for 8 rows)
-    bool ok = true;
-    int buf = 0, filled = 0, base = r0;            // rows base .. base + filled - 1 have partial sums in part[buf]
-    int s = 0;
-    uint32_t phase = 0;
-    const uint4 *w = reinterpret_cast<const uint4 *>(ring);
+    const bool last = pc + 1 == pieces;
+    filled = 0;
     for (int g0 = 0; g0 < r1 - r0; g0 += 8) {
         float acc[MR][8];
 #pragma unroll
@@ -469,7 +475,7 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             for (int j = 0; j < 8; ++j) acc[m][j] = 0.f;
         const int rows = min(8, r1 - r0 - g0);
         // the next launch comes in under the last rows: earlier, its own stream of weights delays this one's
-        if (g0 + 16 >= r1 - r0 && g0 + 8 < r1 - r0) skn_pdl_launch_dependents();
+        if (last && g0 + 16 >= r1 - r0 && g0 + 8 < r1 - r0) skn_pdl_launch_dependents();
 #pragma unroll
         for (int j0 = 0; j0 < 8; j0 += GR) {
             if (j0 < rows) {
@@ -530,10 +536,13 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             float t = acc[m][0];
             t += __shfl_xor_sync(0xffffffffu, t, 2);
             t += __shfl_xor_sync(0xffffffffu, t, 1);
-            if ((lane & 3) == 0) part[buf][m][warp][filled + mvd_row(lane)] = t * rs[m];
+            if ((lane & 3) == 0) {
+                float *p = &part[buf][m][warp][filled + mvd_row(lane)];
+                *p = pc > 0 ? *p + t : t * rs[m];
+            }
         }
         filled += rows;
-        if (filled + 8 > MVD_ROWS || g0 + 8 >= r1 - r0) {
+        if (last && (filled + 8 > MVD_ROWS || g0 + 8 >= r1 - r0)) {
             mvd_barrier();
             auto total = [&](int m, int r) {
                 float t = 0.f;
@@ -559,16 +568,17 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t pitc
             buf ^= 1;                              // the other half is free: every warp has passed the barrier of its readers
         }
     }
+    if (!last) mvd_barrier();                      // (the sums of squares are written again)
+    }
 }
 
-// columns [col0, col0 + cols) of w (whole vectors of 8), then the picked experts' rows
-struct mvd_piece {
-    int64_t col0, cols;
-    bool experts;
-};
+// vectors per lane of a row of `cols` columns
+static int mvd_uu(int64_t cols) { return (int)(((cols / 8 + MVD_WARPS - 1) / MVD_WARPS + 31) / 32); }
+constexpr int MVD_MAX_UU = 7;
+constexpr int64_t MVD_PIECE = (int64_t)MVD_MAX_UU * 32 * MVD_WARPS * 8;      // columns of x that the registers hold
 
 template <int MR, int UU, int PICK>
-static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, const mvd_piece &pc, int m0, cudaStream_t st) {
+static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int pieces, int64_t pitch, int m0, cudaStream_t st) {
     auto kern = skn_dense_matvec_kernel<MR, UU, PICK>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
@@ -576,10 +586,8 @@ static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, const mvd_piece
         if (e != cudaSuccess) return e;
         attr_done[ctx->device & 63] = true;
     }
-    const int64_t own = pc.cols * 2, pitch = own + (pc.experts ? l.pick.n * l.pick.w2->pitch : 0), all = l.w->pitch / 2;
-    const bool whole = pc.col0 == 0 && (pc.experts || pc.cols == all);
-    const int N = PICK == SKN_PICK_ROWS ? l.pick.n * l.pick.rows_per : (int)l.w->n_rows, rows = mvd_stage_rows(MR, UU);
-    const int K = (int)(whole ? skn_linear_cols(l) : pc.experts ? pitch / 2 : pc.col0 + pc.cols < l.w->n_cols ? pc.cols : l.w->n_cols - pc.col0);
+    const int N = PICK == SKN_PICK_ROWS ? l.pick.n * l.pick.rows_per : (int)l.w->n_rows, K = (int)skn_linear_cols(l), rows = mvd_stage_rows(MR, UU);
+    const int64_t row_bytes = PICK == SKN_PICK_COLS ? K * (int64_t)2 : l.w->pitch;
     const size_t xbytes = UU > 0 ? 0 : (size_t)MR * pitch * 2;
     size_t room = mvd_smem(MR) - xbytes;
     if (room > (size_t)MVD_RING) room = MVD_RING;
@@ -588,90 +596,51 @@ static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, const mvd_piece
     if (stages > MVD_MAX_STAGES) stages = MVD_MAX_STAGES;
     const int units = skn_epi_pairs(l.epi.kind) ? (N + 1) / 2 : N;
     const int grid = units < ctx->sm_count ? units : ctx->sm_count;
-    // the piece of x, and the norm if it lies in it
-    const float *x = l.x32 + pc.col0;
-    int64_t ldx = l.ld_x32, ka = l.x32b ? l.k_a - pc.col0 : K;
-    if (ka <= 0) {
-        x = l.x32b - ka;
-        ldx = l.ld_x32b;
-        ka = K;
-    } else if (ka > K) {
-        ka = K;
-    }
-    const bool norm = l.gain && pc.col0 == 0;
-    const mvd_norm nm = {norm ? l.gain : nullptr, l.eps, norm ? l.norm_cols : 0, l.norm_parts > 0 ? l.norm_parts : 1};
-    const mvd_pick pk = {l.pick.expert, PICK == SKN_PICK_COLS ? (const uint8_t *)l.pick.w2->d_blocks : nullptr, own,
+    const mvd_norm nm = {l.gain, l.eps, l.gain ? l.norm_cols : 0, l.norm_parts > 0 ? l.norm_parts : 1};
+    const mvd_pick pk = {l.pick.expert, PICK == SKN_PICK_COLS ? (const uint8_t *)l.pick.w2->d_blocks : nullptr, l.w->pitch,
                          PICK == SKN_PICK_COLS ? l.pick.w2->pitch : 0, l.pick.n, l.pick.rows_per};
-    return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks + pc.col0 * 2,
-                          l.w->pitch, pitch, N, K, m0, x, ldx, l.x32b, l.ld_x32b, (int)ka, nm, pk, stages, l.epi, ctx->d_status);
+    return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks, l.w->pitch,
+                          row_bytes, pieces, pitch, N, K, m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, nm, pk, stages, l.epi, ctx->d_status);
 }
 
-// vectors per lane of a row of `cols` columns
-static int mvd_uu(int64_t cols) { return (int)(((cols / 8 + MVD_WARPS - 1) / MVD_WARPS + 31) / 32); }
-constexpr int MVD_MAX_UU = 7;
-constexpr int64_t MVD_PIECE = (int64_t)MVD_MAX_UU * 32 * MVD_WARPS * 8;      // columns of x that the registers hold
-
+// one activation row; more columns than the registers hold go in pieces where the kernel can (the norm within the first one, few rows per CTA)
 template <int PICK>
-static cudaError_t launch_mvd_pick(skn_ctx *ctx, const skn_linear &l, const mvd_piece &pc, int64_t cols, cudaStream_t st) {
-    switch (mvd_uu(cols)) {
-    case 1: return launch_mvd<1, 1, PICK>(ctx, l, pc, 0, st);
-    case 2: return launch_mvd<1, 2, PICK>(ctx, l, pc, 0, st);
-    case 3: case 4: return launch_mvd<1, 4, PICK>(ctx, l, pc, 0, st);
-    case 5: case 6: case 7: return launch_mvd<1, 7, PICK>(ctx, l, pc, 0, st);
-    default: return launch_mvd<1, 0, PICK>(ctx, l, pc, 0, st);
+static cudaError_t launch_mvd_row(skn_ctx *ctx, const skn_linear &l, int64_t cols, int m0, cudaStream_t st) {
+    int pieces = 1;
+    int64_t size = cols;
+    if (cols > MVD_PIECE && PICK != SKN_PICK_ROWS && !skn_epi_pairs(l.epi.kind) && (!l.gain || (l.norm_cols > 0 && l.norm_cols <= MVD_PIECE)) &&
+        (l.w->n_rows + ctx->sm_count - 1) / ctx->sm_count <= MVD_ROWS - 8) {
+        pieces = (int)((cols + MVD_PIECE - 1) / MVD_PIECE);
+        size = ((cols + pieces - 1) / pieces + 7) / 8 * 8;
+        if (l.gain && size < l.norm_cols) size = l.norm_cols;
+        pieces = (int)((cols + size - 1) / size);
     }
-}
-
-static cudaError_t launch_mvd_row(skn_ctx *ctx, const skn_linear &l, const mvd_piece &pc, int m0, cudaStream_t st) {
-    constexpr int P = SKN_PICK_NONE;
-    switch (mvd_uu(pc.cols)) {
-    case 1: return launch_mvd<1, 1, P>(ctx, l, pc, m0, st);
-    case 2: return launch_mvd<1, 2, P>(ctx, l, pc, m0, st);
-    case 3: return launch_mvd<1, 3, P>(ctx, l, pc, m0, st);
-    case 4: return launch_mvd<1, 4, P>(ctx, l, pc, m0, st);
-    case 5: return launch_mvd<1, 5, P>(ctx, l, pc, m0, st);
-    case 6: return launch_mvd<1, 6, P>(ctx, l, pc, m0, st);
-    case 7: return launch_mvd<1, 7, P>(ctx, l, pc, m0, st);
-    default: return launch_mvd<1, 0, P>(ctx, l, pc, m0, st);
+    switch (mvd_uu(size)) {
+    case 1: return launch_mvd<1, 1, PICK>(ctx, l, pieces, size * 2, m0, st);
+    case 2: return launch_mvd<1, 2, PICK>(ctx, l, pieces, size * 2, m0, st);
+    case 3: return launch_mvd<1, 3, PICK>(ctx, l, pieces, size * 2, m0, st);
+    case 4: return launch_mvd<1, 4, PICK>(ctx, l, pieces, size * 2, m0, st);
+    case 5: return launch_mvd<1, 5, PICK>(ctx, l, pieces, size * 2, m0, st);
+    case 6: return launch_mvd<1, 6, PICK>(ctx, l, pieces, size * 2, m0, st);
+    case 7: return launch_mvd<1, 7, PICK>(ctx, l, pieces, size * 2, m0, st);
+    default: return launch_mvd<1, 0, PICK>(ctx, l, 1, cols * 2, m0, st);
     }
-}
-
-// One activation row whose columns exceed the registers: sums that add to the residual stream may be formed piece by piece, each piece
-// at the rate of a short row (x in registers, many stages in the ring).
-static cudaError_t launch_mvd_pieces(skn_ctx *ctx, const skn_linear &l, int m0, cudaStream_t st) {
-    const int64_t all = l.w->pitch / 2, least = l.gain ? l.norm_cols : 0;
-    const int64_t n = (all + MVD_PIECE - 1) / MVD_PIECE;
-    int64_t size = ((all + n - 1) / n + 7) / 8 * 8;
-    if (size < least) size = least;
-    for (int64_t c = 0; c < all; c += size) {
-        const cudaError_t e = launch_mvd_row(ctx, l, mvd_piece{c, all - c < size ? all - c : size, false}, m0, st);
-        if (e != cudaSuccess) return e;
-    }
-    return cudaSuccess;
 }
 
 cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStream_t st) {
-    const int64_t all = l.w->pitch / 2, cols = l.pick.kind == SKN_PICK_COLS ? skn_linear_cols(l) : all, pitch = cols * 2;
+    const int64_t cols = l.pick.kind == SKN_PICK_COLS ? skn_linear_cols(l) : l.w->pitch / 2, pitch = cols * 2;
     if (l.gain && l.norm_cols > 0 && !skn_norm_folds(l.norm_cols, l.norm_parts)) return cudaErrorInvalidValue;
     if (l.pick.kind && l.M != 1) return cudaErrorInvalidValue;
-    // (a whole-row norm needs the whole row at once)
-    const bool pieces = l.epi.kind == SKN_EPI_ADD && (!l.gain || (l.norm_cols > 0 && l.norm_cols <= MVD_PIECE));
-    if (l.pick.kind == SKN_PICK_ROWS) return launch_mvd_pick<SKN_PICK_ROWS>(ctx, l, mvd_piece{0, all, false}, all, st);
-    if (l.pick.kind == SKN_PICK_COLS) {
-        if (!pieces || mvd_uu(cols) <= 4) return launch_mvd_pick<SKN_PICK_COLS>(ctx, l, mvd_piece{0, all, true}, cols, st);
-        const cudaError_t e = launch_mvd_pieces(ctx, l, 0, st);
-        return e != cudaSuccess ? e : launch_mvd_pick<SKN_PICK_COLS>(ctx, l, mvd_piece{all, 0, true}, cols - all, st);
-    }
+    if (l.pick.kind == SKN_PICK_ROWS) return launch_mvd_row<SKN_PICK_ROWS>(ctx, l, cols, 0, st);
+    if (l.pick.kind == SKN_PICK_COLS) return launch_mvd_row<SKN_PICK_COLS>(ctx, l, cols, 0, st);
     if (pitch * 3 > mvd_smem(1)) return cudaErrorNotSupported;       // one stage and one activation row must fit
-    const mvd_piece whole = {0, all, false};
     for (int m0 = 0; m0 < l.M;) {
         const int left = l.M - m0;
         cudaError_t e;
         int mr = 1;
-        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0, SKN_PICK_NONE>(ctx, l, whole, m0, st); }
-        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0, SKN_PICK_NONE>(ctx, l, whole, m0, st); }
-        else if (pieces && mvd_uu(all) > MVD_MAX_UU) e = launch_mvd_pieces(ctx, l, m0, st);
-        else e = launch_mvd_row(ctx, l, whole, m0, st);
+        if (left >= 4 && pitch * 10 <= mvd_smem(4)) { mr = 4; e = launch_mvd<4, 0, SKN_PICK_NONE>(ctx, l, 1, pitch, m0, st); }
+        else if (left >= 2 && pitch * 6 <= mvd_smem(2)) { mr = 2; e = launch_mvd<2, 0, SKN_PICK_NONE>(ctx, l, 1, pitch, m0, st); }
+        else e = launch_mvd_row<SKN_PICK_NONE>(ctx, l, cols, m0, st);
         if (e != cudaSuccess) return e;
         m0 += mr;
     }

@@ -309,7 +309,8 @@ skn_latent_attn_kernel(skn_latent_args a, skn_step st, const __nv_bfloat16 *__re
 }
 
 // out[m][h][v] = sigmoid(gate) * (W_uv row (h, v) . ol[m][h]).  CTA: OL_ROWS rows of one head, RB tokens.  splits > 0: the latents of
-// the heads are put together here from the attention's splits, else they are in a.ol.  smem (floats): ol [RB][kvp]
+// the heads are put together here from the attention's splits, else they are in a.ol.  smem (floats): ol [RB][kvp], as often
+// as parts of the splits are summed apart
 template <int RB>
 __global__ void __launch_bounds__(LT)
 skn_latent_out_kernel(skn_latent_args a, skn_step st, const uint8_t *__restrict__ ukv, int64_t wpitch, int row_tiles, int M, int per, int splits,
@@ -340,19 +341,29 @@ skn_latent_out_kernel(skn_latent_args a, skn_step st, const uint8_t *__restrict_
             if (lane == 0) s_live[warp] = live;
         }
         __syncthreads();
-        for (int i = tid * 4; i < RB * a.kvp; i += LT * 4) {
-            const int r = i / a.kvp, k = i % a.kvp;
+        // a vector of columns by one thread, or its splits by several
+        const int vecs = RB * a.kvp / 4, parts = max(1, LT / vecs);
+        for (int u = tid; u < vecs * parts; u += LT) {
+            const int part = u / vecs, i = (u % vecs) * 4, r = i / a.kvp, k = i % a.kvp;
             float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
             if (m0 + r < M) {
                 const float *src = sums + (((int64_t)(m0 + r) * a.heads + h) * splits) * a.kvp + k;
 #pragma unroll 8
-                for (int x = 0; x < s_live[r]; ++x) {
+                for (int x = part; x < s_live[r]; x += parts) {
                     const float4 v = __ldcg(reinterpret_cast<const float4 *>(src + (int64_t)x * a.kvp));
                     const float f = share[r][x];
                     t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
                 }
             }
-            *reinterpret_cast<float4 *>(sm + i) = t;
+            *reinterpret_cast<float4 *>(sm + part * RB * a.kvp + i) = t;
+        }
+        if (parts > 1) {
+            __syncthreads();
+            for (int i = tid; i < RB * a.kvp; i += LT) {
+                float t = sm[i];
+                for (int x = 1; x < parts; ++x) t += sm[x * RB * a.kvp + i];
+                sm[i] = t;
+            }
         }
     } else {
         for (int i = tid; i < RB * a.kvp; i += LT) {
@@ -463,9 +474,10 @@ cudaError_t skn_launch_latent_absorbed(const skn_step &s, const skn_latent_args 
     }
     if (e != cudaSuccess) return e;
     const int RB = M == 1 ? 1 : 4;
+    const size_t osm = std::max((size_t)RB * a.kvp, (size_t)LT * 4) * sizeof(float);
     const dim3 grid(a.heads * row_tiles, (M + RB - 1) / RB);
-    if (M == 1) return skn_launch_pdl(skn_latent_out_kernel<1>, grid, dim3(LT), (size_t)a.kvp * 4, st, 1, a, s, w, a.ukv->pitch, row_tiles, M, per, splits, (const float2 *)stats, (const float *)sums);
-    return skn_launch_pdl(skn_latent_out_kernel<4>, grid, dim3(LT), (size_t)4 * a.kvp * 4, st, 1, a, s, w, a.ukv->pitch, row_tiles, M, per, splits, (const float2 *)stats, (const float *)sums);
+    if (M == 1) return skn_launch_pdl(skn_latent_out_kernel<1>, grid, dim3(LT), osm, st, 1, a, s, w, a.ukv->pitch, row_tiles, M, per, splits, (const float2 *)stats, (const float *)sums);
+    return skn_launch_pdl(skn_latent_out_kernel<4>, grid, dim3(LT), osm, st, 1, a, s, w, a.ukv->pitch, row_tiles, M, per, splits, (const float2 *)stats, (const float *)sums);
 }
 
 // ---- expanded form ----------------------------------------------------------------------------------------------------

@@ -18,6 +18,8 @@ constexpr int SC = SKN_SSM_CHUNK;
 constexpr int STEP_THREADS = 256, STEP_COLS = 64;
 
 __device__ __forceinline__ float ssm_silu(float v) { return v / (1.f + expf(-v)); }
+// relative error a few 1e-7: where the result is rounded to bf16 or many are formed
+__device__ __forceinline__ float ssm_silu_fast(float v) { return __fdividef(v, 1.f + __expf(fminf(-v, 80.f))); }
 __device__ __forceinline__ float ssm_softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 
 // convolution and silu of channel c at token t of a sequence whose rows start at `rows` and that had p0 tokens before
@@ -213,8 +215,8 @@ skn_ssm_conv_kernel(skn_ssm_args a, skn_step st, const float *ring_, int ring_pi
     __nv_bfloat16 *out = a.xbc + (int64_t)seq * st.T * channels + c;
     auto put = [&](int t, float4 v) {
         uint2 w;
-        w.x = pack_bf16(ssm_silu(v.x), ssm_silu(v.y));
-        w.y = pack_bf16(ssm_silu(v.z), ssm_silu(v.w));
+        w.x = pack_bf16(ssm_silu_fast(v.x), ssm_silu_fast(v.y));
+        w.y = pack_bf16(ssm_silu_fast(v.z), ssm_silu_fast(v.w));
         *reinterpret_cast<uint2 *>(out + (int64_t)t * channels) = w;
     };
     auto fma4 = [](const float4 &w, const float4 &u, float4 v) {
@@ -453,6 +455,16 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
             cp_async16(skn_smem_u32(St + ((size_t)x * np16 + n) * xs + v), in ? S + ((int64_t)x * a.np + n) * a.vp + v : S, in);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
+        // on their way into L2: this head's gate rows, the next one's state and x
+        for (int i = tid; i < L * ((a.vp + 31) / 32); i += 128) {
+            const int t = i % L, c = i / L * 32;
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(a.proj + (row0 + t) * a.ld + h * a.vp + c));
+        }
+        if (h + 1 < h0 + per) {
+            const __nv_bfloat16 *next = S + (int64_t)2 * a.np * a.vp;
+            for (int i = tid * 64; i < 2 * a.np * a.vp; i += 128 * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(next + i));
+            if (tid < L) asm volatile("prefetch.global.L2 [%0];" ::"l"(rows + (int64_t)tid * channels + (h + 1) * a.vp));
+        }
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         float o[DV / 8][4];
@@ -510,15 +522,17 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
             const int64_t m = row0 + i;
             const float *zr = a.proj + m * a.ld + h * a.vp;
             float *yr = a.y + m * a.ld_y + h * a.vp;
+            float2 z[DV / 8];                       // loaded before the first store
+#pragma unroll
+            for (int n = 0; n < DV / 8; ++n) z[n] = n * 8 + gc < a.vp ? __ldcg(reinterpret_cast<const float2 *>(zr + n * 8 + gc)) : make_float2(0.f, 0.f);
 #pragma unroll
             for (int n = 0; n < DV / 8; ++n) {
                 const int v = n * 8 + gc;
                 if (v >= a.vp) continue;
                 const uint32_t xw = *reinterpret_cast<const uint32_t *>(X + i * xs + v);
-                const float2 z = __ldcg(reinterpret_cast<const float2 *>(zr + v));
                 float2 y;
-                y.x = fmaf(dv, __uint_as_float(xw << 16), o[n][r * 2]) * __fdividef(z.x, 1.f + __expf(fminf(-z.x, 80.f)));
-                y.y = fmaf(dv, __uint_as_float(xw & 0xFFFF0000u), o[n][r * 2 + 1]) * __fdividef(z.y, 1.f + __expf(fminf(-z.y, 80.f)));
+                y.x = fmaf(dv, __uint_as_float(xw << 16), o[n][r * 2]) * ssm_silu_fast(z[n].x);
+                y.y = fmaf(dv, __uint_as_float(xw & 0xFFFF0000u), o[n][r * 2 + 1]) * ssm_silu_fast(z[n].y);
                 *reinterpret_cast<float2 *>(yr + v) = y;
             }
         }
@@ -541,7 +555,7 @@ static cudaError_t launch_chunks(const skn_step &s, const skn_ssm_args &a, cudaS
     const int group = a.heads / a.groups;
     int per = 1;
     for (int p = 2; p <= 8; p *= 2)
-        if (group % p == 0 && (int64_t)nchunks * s.n_seqs * (a.heads / p) >= 512) per = p;
+        if (group % p == 0 && (int64_t)nchunks * s.n_seqs * (a.heads / p) >= 1024) per = p;
     const dim3 grid(nchunks, a.heads / per, s.n_seqs);
     if ((e = cudaFuncSetAttribute(skn_ssm_chunk_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)) != cudaSuccess) return e;
     if ((e = skn_launch_pdl(skn_ssm_chunk_kernel<DV>, grid, dim3(128), ssm_chunk_smem(a.np, DV), st, 1, a, s.T, nchunks, per)) != cudaSuccess) return e;
