@@ -185,20 +185,32 @@ skn_ssm_conv_kernel(skn_ssm_args a, skn_step st, const float *ring_, int ring_pi
     const int channels = skn_ssm_channels(a.heads, a.vp, a.groups, a.np);
     const float *row0 = a.proj + (int64_t)seq * st.T * a.ld;
     if ((int)blockIdx.x >= tiles) {
-        // cum restarts with every chunk; the chunk's rows of this block's tokens are walked by one thread per head
-        const int t0 = blockIdx.y * CV_TOKENS;
+        // one chunk, 32 heads: a warp takes a quarter of the tokens, a lane one head
+        const int t0 = blockIdx.y * CV_TOKENS, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
         if (t0 % SC) return;
-        const int h = ((int)blockIdx.x - tiles) * 128 + threadIdx.x;
-        if (h >= a.heads) return;
-        const float av = a.a[h], bias = a.dt_bias[h];
+        __shared__ float quarter[4][32];
+        const int h = ((int)blockIdx.x - tiles) * 32 + lane, first = t0 + warp * (SC / 4);
+        const bool in = h < a.heads;
+        const float av = in ? a.a[h] : 0.f, bias = in ? a.dt_bias[h] : 0.f;
+        float dt[SC / 4], sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < SC / 4; ++i) dt[i] = in && first + i < st.T ? __ldcg(row0 + (int64_t)(first + i) * a.ld + inner + channels + h) : 0.f;
+#pragma unroll
+        for (int i = 0; i < SC / 4; ++i) {
+            dt[i] = ssm_softplus(dt[i] + bias);
+            sum += dt[i];
+        }
+        quarter[warp][lane] = sum;
+        __syncthreads();
         float cum = 0.f;
-#pragma unroll 8
-        for (int t = t0; t < min(st.T, t0 + SC); ++t) {
-            const float dt = ssm_softplus(__ldcg(row0 + (int64_t)t * a.ld + inner + channels + h) + bias);
-            cum = fmaf(av, dt, cum);
-            const int64_t at = ((int64_t)seq * st.T + t) * a.heads + h;
-            a.dt[at] = dt;
-            a.cum[at] = cum;
+        for (int w = 0; w < warp; ++w) cum += quarter[w][lane];
+#pragma unroll
+        for (int i = 0; i < SC / 4; ++i) {
+            cum += dt[i];
+            if (!in || first + i >= st.T) continue;
+            const int64_t at = ((int64_t)seq * st.T + first + i) * a.heads + h;
+            a.dt[at] = dt[i];
+            a.cum[at] = av * cum;
         }
         return;
     }
@@ -249,13 +261,23 @@ skn_ssm_conv_kernel(skn_ssm_args a, skn_step st, const float *ring_, int ring_pi
     }
 }
 
-// rows of a chunk in shared memory: `cols` valid columns (a multiple of 8) of src, zero beyond, row stride `stride`
+// rows of a chunk in shared memory: `cols` valid columns (a multiple of 8) of src, zero beyond, row stride `stride`.  A warp takes a row.
 __device__ __forceinline__ void ssm_load_rows(__nv_bfloat16 *dst, int stride, const __nv_bfloat16 *src, int64_t ld, int L, int cols, int wide) {
-    const int pieces = wide / 8;
-    for (int i = threadIdx.x; i < SC * pieces; i += blockDim.x) {
-        const int t = i / pieces, c = i % pieces * 8;
-        const bool in = t < L && c < cols;
-        cp_async16(skn_smem_u32(dst + t * stride + c), in ? src + t * ld + c : src, in);
+    const int lane = threadIdx.x & 31;
+    for (int t = threadIdx.x >> 5; t < SC; t += 4)
+        for (int c = lane * 8; c < wide; c += 256) {
+            const bool in = t < L && c < cols;
+            cp_async16(skn_smem_u32(dst + t * stride + c), in ? src + t * ld + c : src, in);
+        }
+}
+// the same for rows of DV columns, DV / 8 threads to a row: row n at src + n * ld for n < valid
+template <int DV>
+__device__ __forceinline__ void ssm_load_tile(__nv_bfloat16 *dst, const __nv_bfloat16 *src, int64_t ld, int rows, int valid, int cols) {
+    constexpr int TPR = DV / 8;
+    const int c = threadIdx.x % TPR * 8;
+    for (int n = threadIdx.x / TPR; n < rows; n += 128 / TPR) {
+        const bool in = n < valid && c < cols;
+        cp_async16(skn_smem_u32(dst + n * (DV + 8) + c), in ? src + n * ld + c : src, in);
     }
 }
 
@@ -441,7 +463,7 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
     }
     for (int h = h0; h < h0 + per; ++h) {
         __syncthreads();                            // the head before is done with x, the state and the decays
-        ssm_load_rows(X, xs, rows + h * a.vp, channels, L, a.vp, DV);
+        ssm_load_tile<DV>(X, rows + h * a.vp, channels, SC, L, a.vp);
         asm volatile("cp.async.commit_group;" ::: "memory");
         if (tid < SC) {
             const int64_t at = (row0 + min(tid, L - 1)) * a.heads + h;
@@ -449,17 +471,12 @@ skn_ssm_out_kernel(skn_ssm_args a, int T, int nchunks, int per) {
             dt_s[tid] = tid < L ? a.dt[at] : 0.f;
         }
         const __nv_bfloat16 *S = a.starts + (((int64_t)seq * nchunks + c) * a.heads + h) * 2 * a.np * a.vp;
-        for (int i = tid; i < 2 * np16 * (DV / 8); i += 128) {
-            const int x = i / (np16 * (DV / 8)), n = i / (DV / 8) % np16, v = i % (DV / 8) * 8;
-            const bool in = n < a.np && v < a.vp;
-            cp_async16(skn_smem_u32(St + ((size_t)x * np16 + n) * xs + v), in ? S + ((int64_t)x * a.np + n) * a.vp + v : S, in);
-        }
+#pragma unroll
+        for (int x = 0; x < 2; ++x) ssm_load_tile<DV>(St + (size_t)x * np16 * xs, S + (int64_t)x * a.np * a.vp, a.vp, np16, a.np, a.vp);
         asm volatile("cp.async.commit_group;" ::: "memory");
         // on their way into L2: this head's gate rows, the next one's state and x
-        for (int i = tid; i < L * ((a.vp + 31) / 32); i += 128) {
-            const int t = i % L, c = i / L * 32;
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(a.proj + (row0 + t) * a.ld + h * a.vp + c));
-        }
+        for (int c = 0; c < a.vp; c += 32)
+            if (tid < L) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.proj + (row0 + tid) * a.ld + h * a.vp + c));
         if (h + 1 < h0 + per) {
             const __nv_bfloat16 *next = S + (int64_t)2 * a.np * a.vp;
             for (int i = tid * 64; i < 2 * a.np * a.vp; i += 128 * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(next + i));
@@ -544,7 +561,7 @@ bool skn_ssm_chunks_fit(int vp, int np) { return vp <= 128 && np <= 256 && ssm_o
 template <int DV>
 static cudaError_t launch_chunks(const skn_step &s, const skn_ssm_args &a, cudaStream_t st) {
     const int nchunks = (s.T + SC - 1) / SC, channels = skn_ssm_channels(a.heads, a.vp, a.groups, a.np);
-    const int ctiles = (channels / 4 + 127) / 128, htiles = (a.heads + 127) / 128;
+    const int ctiles = (channels / 4 + 127) / 128, htiles = (a.heads + 31) / 32;
     const dim3 vgrid(ctiles + htiles, (s.T + CV_TOKENS - 1) / CV_TOKENS, s.n_seqs);
     cudaError_t e = a.taps == 4   ? skn_launch_pdl(skn_ssm_conv_kernel<4>, vgrid, dim3(128), 0, st, 1, a, s, (const float *)a.ring->d, a.ring->v_pitch, ctiles)
                     : a.taps == 2 ? skn_launch_pdl(skn_ssm_conv_kernel<2>, vgrid, dim3(128), 0, st, 1, a, s, (const float *)a.ring->d, a.ring->v_pitch, ctiles)
