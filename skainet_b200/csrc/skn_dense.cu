@@ -121,9 +121,31 @@ __device__ __forceinline__ void dense_store_run(const skn_epi &e, int64_t m, int
     }
 }
 
+// NC tokens of bf16 rows, the whole warp together (lane l: row n = (even base) + l): neighbouring lanes trade every other token, so that a
+// lane stores two columns at once.  y: column n of token m; `in` marks the rows that exist, in pairs.
+template <int NC>
+__device__ __forceinline__ void dense_put_packed(__nv_bfloat16 *y, int64_t ld, int64_t n, const float (&v)[NC], int count, bool in) {
+    const bool odd = n & 1;
+    uint32_t *p = reinterpret_cast<uint32_t *>(y - (odd ? 1 : 0)) + (odd ? ld / 2 : 0);
+#pragma unroll
+    for (int c = 0; c < NC; c += 2) {
+        const float got = __shfl_xor_sync(0xffffffffu, odd ? v[c] : v[c + 1], 1);
+        const uint32_t w = odd ? tc_pack_bf16(got, v[c + 1]) : tc_pack_bf16(v[c], got);
+        if (in && c + (odd ? 1 : 0) < count) *p = w;
+        p += ld;                                   // two tokens of ld / 2 words
+    }
+}
+// whether an epilogue's run may be stored that way
+template <int EPI>
+__device__ __forceinline__ bool dense_packs(const skn_epi &e, int N) {
+    if (EPI == SKN_EPI_STORE || EPI == SKN_EPI_ROTATE)
+        return N % 2 == 0 && !e.y32 && e.y16 && e.ld_y16 % 2 == 0 && (reinterpret_cast<uintptr_t>(e.y16) & 3) == 0;
+    return false;
+}
+
 // The same for the pair epilogues, the whole warp together: lane l holds row n = (even base) + l, `in` marks the rows that exist.
 template <int EPI, int NC>
-__device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count, bool in) {
+__device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count, bool in, bool packed) {
     const bool odd = n & 1;
     if (EPI == SKN_EPI_ROTATE) {
         // the angles of the run are loaded before its first store
@@ -136,6 +158,10 @@ __device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t 
         for (int c = 0; c < NC; ++c) {
             const float other = __shfl_xor_sync(0xffffffffu, v[c], 1);
             v[c] = odd ? v[c] * cs[c].x + other * cs[c].y : v[c] * cs[c].x - other * cs[c].y;
+        }
+        if (packed) {
+            dense_put_packed(e.y16 + m * e.ld_y16 + n, e.ld_y16, n, v, count, in);
+            return;
         }
 #pragma unroll
         for (int c = 0; c < NC; ++c)
@@ -892,6 +918,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     } else {
         // epilogue: TMEM lane = weight row, column = token; a warp's store covers 32 consecutive outputs of one token
         bool ok = true;
+        const bool packed = dense_packs<EPI>(e, N);
         int tile = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, ++tile) {
             const dtc_tile tl = tile_of(u);
@@ -917,7 +944,12 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                         float v[32];
 #pragma unroll
                         for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
-                        dense_store_run_pairs<EPI, 32>(e, m0 + c0, n, v, cols - c0, n < N && ok);
+                        dense_store_run_pairs<EPI, 32>(e, m0 + c0, n, v, cols - c0, n < N && ok, packed);
+                    } else if (EPI == SKN_EPI_STORE && packed) {
+                        float v[32];
+#pragma unroll
+                        for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
+                        dense_put_packed(e.y16 + (m0 + c0) * e.ld_y16 + n, e.ld_y16, n, v, cols - c0, n < N && ok);
                     } else if (n < N && ok) {
                         float v[32];
 #pragma unroll
@@ -949,7 +981,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                         for (int s = 0; s < splits; ++s)
 #pragma unroll
                             for (int c = 0; c < 16; ++c) v[c] += __ldcg(pbase + ((size_t)s * NT + c0 + c) * DTC_BM);
-                        if constexpr (skn_epi_pairs(EPI)) dense_store_run_pairs<EPI, 16>(e, m0 + c0, n, v, cols - c0, n < N && ok);
+                        if constexpr (skn_epi_pairs(EPI)) dense_store_run_pairs<EPI, 16>(e, m0 + c0, n, v, cols - c0, n < N && ok, packed);
                         else if (n < N && ok) dense_store_run<EPI, 16>(e, m0 + c0, n, v, cols - c0);
                     }
                     if (threadIdx.x == 0) tickets[tidx] = 0;

@@ -14,13 +14,15 @@ cudaError_t skn_launch_route(const skn_route_args &r, int M, cudaStream_t st) {
     return skn_launch_pdl(skn_route_kernel, dim3(M), dim3(32), skn_route_smem(r), st, 1, r);
 }
 
+constexpr int GP_THREADS = 1024;
+
 // CTA e reads every pair: those of lower experts count towards its offset, its own get consecutive places
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(GP_THREADS)
 skn_group_pairs_kernel(const int32_t *expert, int pairs, int experts, int32_t *offset, int32_t *place) {
-    __shared__ int below[256], own[256], base_s;
+    __shared__ int below[GP_THREADS], own[GP_THREADS], base_s;
     skn_pdl_launch_dependents();
     skn_pdl_wait();
-    const int e = blockIdx.x, tid = threadIdx.x, per = (pairs + 255) / 256, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
+    const int e = blockIdx.x, tid = threadIdx.x, per = (pairs + GP_THREADS - 1) / GP_THREADS, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
     int lo = 0, eq = 0;
 #pragma unroll 8
     for (int i = i0; i < i1; ++i) {
@@ -33,9 +35,9 @@ skn_group_pairs_kernel(const int32_t *expert, int pairs, int experts, int32_t *o
     __syncthreads();
     if (tid < 32) {
         int total = 0, run = 0;
-        for (int j = 0; j < 8; ++j) {
-            total += below[tid * 8 + j];
-            run += own[tid * 8 + j];
+        for (int j = 0; j < GP_THREADS / 32; ++j) {
+            total += below[tid * (GP_THREADS / 32) + j];
+            run += own[tid * (GP_THREADS / 32) + j];
         }
         int before = run;
 #pragma unroll
@@ -44,9 +46,9 @@ skn_group_pairs_kernel(const int32_t *expert, int pairs, int experts, int32_t *o
             if (tid >= o) before += y;
         }
         before -= run;
-        for (int j = 0; j < 8; ++j) {
-            const int n = own[tid * 8 + j];
-            own[tid * 8 + j] = before;
+        for (int j = 0; j < GP_THREADS / 32; ++j) {
+            const int n = own[tid * (GP_THREADS / 32) + j];
+            own[tid * (GP_THREADS / 32) + j] = before;
             before += n;
         }
 #pragma unroll
@@ -65,7 +67,7 @@ skn_group_pairs_kernel(const int32_t *expert, int pairs, int experts, int32_t *o
 }
 
 cudaError_t skn_launch_group_pairs(const int32_t *expert, int pairs, int experts, int32_t *offset, int32_t *place, cudaStream_t st) {
-    return skn_launch_pdl(skn_group_pairs_kernel, dim3(experts), dim3(256), 0, st, 1, expert, pairs, experts, offset, place);
+    return skn_launch_pdl(skn_group_pairs_kernel, dim3(experts), dim3(GP_THREADS), 0, st, 1, expert, pairs, experts, offset, place);
 }
 
 // rows in 16-byte pieces (pitches are multiples of 8 elements, padding included)
