@@ -261,19 +261,20 @@ struct mvd_norm {
     int cols, parts;                    // cols 0: the whole row
 };
 
-template <int MR, int UU, int PICK>
+template <int MR, int UU, int PICK, bool PAIRS, bool PIECES>
 __global__ void __launch_bounds__(MVD_THREADS, 2)
-skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_bytes, int pieces, int64_t pitch, int N, int K, int m0, const float *x,
+skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_bytes, int n_pieces, int64_t pitch, int N, int K, int m0, const float *x,
                         int64_t ldx, const float *xb, int64_t ldxb, int ka, mvd_norm nm, mvd_pick pk, int stages, skn_epi e, int32_t *status) {
     extern __shared__ __align__(128) uint8_t ring[];
     constexpr int GR = mvd_stage_rows(MR, UU);
     __shared__ uint64_t full_bar[MVD_MAX_STAGES], empty_bar[MVD_MAX_STAGES];
     __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS], psum[MR][MVD_WARPS][SKN_NORM_PARTS];
     const float *__restrict__ gain = nm.gain;
-    const bool pairs = skn_epi_pairs(e.kind), partial = gain && nm.cols > 0;
+    const bool partial = !PAIRS && gain && nm.cols > 0;
+    const int pieces = PIECES ? n_pieces : 1;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2;           // vectors of a piece (of the row, when there is one)
-    const int q_rows = pairs ? 2 : 1, nq = (N + q_rows - 1) / q_rows;     // pairs of rows stay together
+    const int q_rows = PAIRS ? 2 : 1, nq = (N + q_rows - 1) / q_rows;     // pairs of rows stay together
     const int r0 = min(N, q_rows * (int)((int64_t)nq * blockIdx.x / gridDim.x)), r1 = min(N, q_rows * (int)((int64_t)nq * (blockIdx.x + 1) / gridDim.x));
     const int steps = (r1 - r0 + GR - 1) / GR;
     const size_t stage_bytes = (size_t)GR * pitch;
@@ -576,14 +577,13 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_
                 for (int w8 = 0; w8 < MVD_WARPS; ++w8) t += part[buf][m][w8][r];
                 return t;
             };
-            if (pairs) {
+            if constexpr (PAIRS) {
                 const int np = (filled + 1) / 2;
                 for (int j = threadIdx.x; j < np * MR; j += MVD_WARPS * 32) {
                     const int m = j / np, r = j % np * 2;
                     const bool both = r + 1 < filled;
                     const float a = total(m, r), b = both ? total(m, r + 1) : 0.f;
-                    if (e.kind == SKN_EPI_ROTATE) dense_store_pair<SKN_EPI_ROTATE>(e, m0 + m, base + r, a, b, both);
-                    else dense_store_pair<SKN_EPI_SILU_TAIL>(e, m0 + m, base + r, a, b, both);
+                    dense_store_pair<SKN_EPI_SILU_TAIL>(e, m0 + m, base + r, a, b, both);
                 }
             } else for (int j = threadIdx.x; j < filled * MR; j += MVD_WARPS * 32) {
                 const int m = j / filled, r = j % filled;
@@ -603,9 +603,9 @@ static int mvd_uu(int64_t cols) { return (int)(((cols / 8 + MVD_WARPS - 1) / MVD
 constexpr int MVD_MAX_UU = 7;
 constexpr int64_t MVD_PIECE = (int64_t)MVD_MAX_UU * 32 * MVD_WARPS * 8;      // columns of x that the registers hold
 
-template <int MR, int UU, int PICK>
-static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int pieces, int64_t pitch, int m0, cudaStream_t st) {
-    auto kern = skn_dense_matvec_kernel<MR, UU, PICK>;
+template <int MR, int UU, int PICK, bool PAIRS, bool PIECES>
+static cudaError_t launch_mvd_kernel(skn_ctx *ctx, const skn_linear &l, int pieces, int64_t pitch, int m0, cudaStream_t st) {
+    auto kern = skn_dense_matvec_kernel<MR, UU, PICK, PAIRS, PIECES>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, mvd_smem(MR));
@@ -620,13 +620,27 @@ static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int pieces, int
     int stages = (int)(room / (rows * pitch));
     if (stages < 1) return cudaErrorNotSupported;
     if (stages > MVD_MAX_STAGES) stages = MVD_MAX_STAGES;
-    const int units = skn_epi_pairs(l.epi.kind) ? (N + 1) / 2 : N;
+    const int units = PAIRS ? (N + 1) / 2 : N;
     const int grid = units < ctx->sm_count ? units : ctx->sm_count;
     const mvd_norm nm = {l.gain, l.eps, l.gain ? l.norm_cols : 0, l.norm_parts > 0 ? l.norm_parts : 1};
     const mvd_pick pk = {l.pick.expert, PICK == SKN_PICK_COLS ? (const uint8_t *)l.pick.w2->d_blocks : nullptr, l.w->pitch,
                          PICK == SKN_PICK_COLS ? l.pick.w2->pitch : 0, l.pick.n, l.pick.rows_per};
     return skn_launch_pdl(kern, dim3(grid), dim3(MVD_THREADS), (size_t)stages * rows * pitch + xbytes, st, 1, (const uint8_t *)l.w->d_blocks, l.w->pitch,
                           row_bytes, pieces, pitch, N, K, m0, l.x32, l.ld_x32, l.x32b, l.ld_x32b, l.x32b ? (int)l.k_a : K, nm, pk, stages, l.epi, ctx->d_status);
+}
+
+template <int MR, int UU, int PICK>
+static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int pieces, int64_t pitch, int m0, cudaStream_t st) {
+    const bool pairs = l.epi.kind == SKN_EPI_SILU_TAIL;
+    if constexpr (PICK != SKN_PICK_COLS)
+        if (pairs) return launch_mvd_kernel<MR, UU, PICK, true, false>(ctx, l, 1, pitch, m0, st);
+    if (pairs) return cudaErrorInvalidValue;
+    if constexpr (PICK == SKN_PICK_ROWS) return cudaErrorInvalidValue;
+    else {
+        if constexpr (MR == 1 && UU >= 4)
+            if (pieces > 1) return launch_mvd_kernel<MR, UU, PICK, false, true>(ctx, l, pieces, pitch, m0, st);
+        return launch_mvd_kernel<MR, UU, PICK, false, false>(ctx, l, 1, pitch, m0, st);
+    }
 }
 
 // one activation row; more columns than the registers hold go in pieces where the kernel can (the norm within the first one, few rows per CTA)
@@ -656,7 +670,7 @@ static cudaError_t launch_mvd_row(skn_ctx *ctx, const skn_linear &l, int64_t col
 cudaError_t skn_launch_dense_matvec(skn_ctx *ctx, const skn_linear &l, cudaStream_t st) {
     const int64_t cols = l.pick.kind == SKN_PICK_COLS ? skn_linear_cols(l) : l.w->pitch / 2, pitch = cols * 2;
     if (l.gain && l.norm_cols > 0 && !skn_norm_folds(l.norm_cols, l.norm_parts)) return cudaErrorInvalidValue;
-    if (l.pick.kind && l.M != 1) return cudaErrorInvalidValue;
+    if ((l.pick.kind && l.M != 1) || l.epi.kind == SKN_EPI_ROTATE) return cudaErrorInvalidValue;
     if (l.pick.kind == SKN_PICK_ROWS) return launch_mvd_row<SKN_PICK_ROWS>(ctx, l, cols, 0, st);
     if (l.pick.kind == SKN_PICK_COLS) return launch_mvd_row<SKN_PICK_COLS>(ctx, l, cols, 0, st);
     if (pitch * 3 > mvd_smem(1)) return cudaErrorNotSupported;       // one stage and one activation row must fit
