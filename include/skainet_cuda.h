@@ -524,18 +524,18 @@ int32_t skn_lugasun_set_head(skn_decoder *m, const skn_tensor *embed, const floa
  * loop_step[t], and from the second pass on the embedding output again.
  *
  * Head and latent widths are padded to multiples of 8 with zero weights, written ~ below: ~n is n rounded up. */
-/* y_t = S_t^T C_t + D x_t, S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T per head, x, B, C out of a causal
- * convolution of `taps` taps with silu, dt_t = softplus; head h reads B and C of group h / (heads / groups).  y times
- * silu(z) is RMS-normed in norm_groups parts. */
+/* Per head a state S [state][vdim]: S <- exp(-exp(A_log) dt) S + dt B x^T, output S^T C + D x, where dt = softplus(raw + bias)
+ * and x, B, C are convolved over the last `taps` tokens (silu after).  Neighbouring heads, heads / groups of them, share B and
+ * C.  The outputs take a factor silu(z), then an RMS norm of norm_groups equal parts of all heads' columns. */
 typedef struct skn_ssm_spec {
     int32_t heads, vdim, state, groups, taps, norm_groups;
     float eps;
     int32_t reserved;
 } skn_ssm_spec;
 /* Queries and keys / values go through latents of q_rank and kv_rank (RMS-normed); a key is [dim from the latent |
- * rot_dim rotated, shared by the heads], adjacent dimensions of the rotated part forming pairs (the first rot_dims turn).  Only the
- * latent and the rotated key part are cached.  Query i sees keys j with 0 <= i - j < window (0: all earlier ones); one learned score
- * per head joins the softmax denominator; the heads are multiplied by a sigmoid gate. */
+ * rot_dim rotated, the same for every head], adjacent dimensions of the rotated part forming pairs (the first rot_dims turn).  The
+ * cache keeps one row per token: its latent and its rotated part.  A query sees the last `window` positions, its own included (0:
+ * every earlier one); one learned score per head joins the softmax denominator; a sigmoid gate multiplies the heads. */
 typedef struct skn_latent_spec {
     int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank, rot_dims, window;
     double rot_base;

@@ -28,7 +28,7 @@ def softplus(z):
 
 # ---- selective state space -------------------------------------------------------------------------------------
 def causal_conv(u, w, b):
-    """u [T, channels], w [channels, taps]: the last tap meets the current token, tokens before the start are zero."""
+    """u [T, channels], w [channels, taps]: y_t = b + sum over k of w_k u_(t - taps + 1 + k), with u = 0 ahead of the sequence."""
     T, taps = u.shape[0], w.shape[1]
     y = np.zeros_like(u)
     for t in range(T):

@@ -219,9 +219,11 @@ __device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 
 // CTA b owns the weight rows [b N / grid, (b + 1) N / grid): a producer warp streams them, a few rows per bulk copy, through
 // a ring of shared-memory stages and starts before the kernel waits for its predecessor; eight warps each take an eighth of
 // the columns of every row.  Their partial sums meet in shared memory, 128 rows at a time.  One activation row lives in
-// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).  Rows longer than the registers hold are taken in
-// column pieces, one after the other for all rows of the CTA (at most MVD_ROWS then), the partial sums waiting in shared memory.  PICK: the weight rows, or pieces of
-// them, belong to experts that a kernel before chose, so the stream of those starts after the dependency wait.
+// registers (UU vectors of eight columns per lane), more rows in shared memory (UU = 0).
+// EXT: a norm of a part of the columns, or rows longer than the registers hold, taken in column pieces: one piece after the other
+// for all rows of the CTA (at most MVD_ROWS), the partial sums waiting in shared memory.
+// PICK: the weight rows, or pieces of them, belong to experts that a kernel before chose, so the stream of those starts after
+// the dependency wait.
 constexpr int MVD_WARPS = 8, MVD_THREADS = (MVD_WARPS + 1) * 32, MVD_ROWS = 128;
 constexpr int MVD_RING = 96 * 1024, MVD_MAX_STAGES = 24;
 // dynamic shared memory beside the partial sums of MR rows
@@ -251,8 +253,7 @@ __device__ __forceinline__ int mvd_row(int lane) { return ((lane >> 4) & 1) * 4 
 struct mvd_pick {
     const int32_t *expert;
     const uint8_t *w2;                  // SKN_PICK_COLS
-    int64_t pitch1;                     // SKN_PICK_COLS: bytes that w (0: none of it) and each expert have in a joint row of `pitch` bytes
-    int64_t pitch2;
+    int64_t pitch1, pitch2;             // SKN_PICK_COLS: bytes that w and each expert have in a joint row
     int n, rows_per;
 };
 struct mvd_norm {
@@ -261,17 +262,17 @@ struct mvd_norm {
     int cols, parts;                    // cols 0: the whole row
 };
 
-template <int MR, int UU, int PICK, bool PAIRS, bool PIECES>
+template <int MR, int UU, int PICK, bool PAIRS, bool EXT>
 __global__ void __launch_bounds__(MVD_THREADS, 2)
 skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_bytes, int n_pieces, int64_t pitch, int N, int K, int m0, const float *x,
                         int64_t ldx, const float *xb, int64_t ldxb, int ka, mvd_norm nm, mvd_pick pk, int stages, skn_epi e, int32_t *status) {
     extern __shared__ __align__(128) uint8_t ring[];
     constexpr int GR = mvd_stage_rows(MR, UU);
     __shared__ uint64_t full_bar[MVD_MAX_STAGES], empty_bar[MVD_MAX_STAGES];
-    __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS], psum[MR][MVD_WARPS][SKN_NORM_PARTS];
+    __shared__ float red[MVD_WARPS][MR], part[2][MR][MVD_WARPS][MVD_ROWS], psum[EXT ? MR : 1][MVD_WARPS][EXT ? SKN_NORM_PARTS : 1];
     const float *__restrict__ gain = nm.gain;
-    const bool partial = !PAIRS && gain && nm.cols > 0;
-    const int pieces = PIECES ? n_pieces : 1;
+    const bool partial = EXT && gain && nm.cols > 0;
+    const int pieces = EXT ? n_pieces : 1;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int nv = (int)(pitch >> 4), K8 = nv * 8, half = K8 / 2;           // vectors of a piece (of the row, when there is one)
     const int q_rows = PAIRS ? 2 : 1, nq = (N + q_rows - 1) / q_rows;     // pairs of rows stay together
@@ -287,6 +288,28 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_
     }
     __syncthreads();
     if (warp == MVD_WARPS) {
+        if constexpr (PICK == SKN_PICK_NONE && !EXT) {
+            if (lane == 0) {
+                int s = 0;
+                uint32_t phase = 1;
+                for (int i = 0; i < steps; ++i) {
+                    const int row = r0 + i * GR;
+                    if (!skn_mbar_wait(&empty_bar[s], phase)) {
+                        atomicExch(status, SKN_ERR_TIMEOUT);
+                        break;
+                    }
+                    const uint32_t bytes = (uint32_t)(min(GR, r1 - row) * pitch);
+                    skn_mbar_expect_tx(&full_bar[s], bytes);
+                    skn_bulk_g2s(ring + s * stage_bytes, W + (int64_t)row * pitch, bytes, &full_bar[s]);
+                    if (++s == stages) {
+                        s = 0;
+                        phase ^= 1u;
+                    }
+                }
+            }
+            skn_pdl_wait();
+            return;
+        }
         // lane 0 keeps the ring; the copies of a stage are issued by as many lanes as there are pieces of rows in it
         int s = 0, early = 0;
         uint32_t phase = 1;
@@ -355,246 +378,246 @@ skn_dense_matvec_kernel(const uint8_t *__restrict__ W, int64_t wld, int64_t row_
     uint32_t phase = 0;
     const uint4 *w = reinterpret_cast<const uint4 *>(ring);
     for (int pc = 0; pc < pieces; ++pc) {
-    // this warp's columns: vectors v0 + lane + 32 u below v1 of the piece, which starts at vector vb of the row
-    const int vb = pc * nv, nvp = min(nv, (int)(row_bytes >> 4) - vb), per = (nvp + MVD_WARPS - 1) / MVD_WARPS, v0 = warp * per, v1 = min(nvp, v0 + per);
-    float4 xr[UU > 0 ? 2 * UU : 1];
-    float *xs = reinterpret_cast<float *>(ring + stages * stage_bytes);     // UU = 0: [MR][2 planes][K8 / 2]: quads 0 and 1 of every eight columns
-    float ss[MR];
-    auto fetch = [&](int m, int k) {
-        float v = 0.f;
-        if (k < K) v = __ldcg(k < ka ? x + (int64_t)(m0 + m) * ldx + k : xb + (int64_t)(m0 + m) * ldxb + k - ka);
-        return v;
-    };
-    if constexpr (UU > 0) {
-        // rows that are whole aligned vectors (the usual case) are read 16 bytes at a time
-        const bool vec = K % 8 == 0 && ka % 8 == 0 && ldx % 4 == 0 && ldxb % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xb)) & 15) == 0;
-        float q = 0.f, vsq[UU];
+        // this warp's columns: vectors v0 + lane + 32 u below v1 of the piece, which starts at vector vb of the row
+        const int vb = pc * nv, nvp = min(nv, (int)(row_bytes >> 4) - vb), per = (nvp + MVD_WARPS - 1) / MVD_WARPS, v0 = warp * per, v1 = min(nvp, v0 + per);
+        float4 xr[UU > 0 ? 2 * UU : 1];
+        float *xs = reinterpret_cast<float *>(ring + stages * stage_bytes);     // UU = 0: [MR][2 planes][K8 / 2]: quads 0 and 1 of every eight columns
+        float ss[MR];
+        auto fetch = [&](int m, int k) {
+            float v = 0.f;
+            if (k < K) v = __ldcg(k < ka ? x + (int64_t)(m0 + m) * ldx + k : xb + (int64_t)(m0 + m) * ldxb + k - ka);
+            return v;
+        };
+        if constexpr (UU > 0) {
+            // rows that are whole aligned vectors (the usual case) are read 16 bytes at a time
+            const bool vec = K % 8 == 0 && ka % 8 == 0 && ldx % 4 == 0 && ldxb % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xb)) & 15) == 0;
+            float q = 0.f, vsq[UU];
 #pragma unroll
-        for (int u = 0; u < UU; ++u) {
-            const int i = v0 + u * 32 + lane;
-            vsq[u] = 0.f;
-            float f[8];
-            const int k = (vb + i) * 8;
-            if (vec && i < v1) {
-                const float *p = k < ka ? x + (int64_t)m0 * ldx + k : xb + (int64_t)m0 * ldxb + k - ka;
-                *reinterpret_cast<float4 *>(f) = __ldcg(reinterpret_cast<const float4 *>(p));
-                *reinterpret_cast<float4 *>(f + 4) = __ldcg(reinterpret_cast<const float4 *>(p + 4));
-            } else {
-#pragma unroll
-                for (int j = 0; j < 8; ++j) f[j] = i < v1 ? fetch(0, k + j) : 0.f;
-            }
-#pragma unroll
-            for (int j = 0; j < 8; ++j) vsq[u] = fmaf(f[j], f[j], vsq[u]);
-            q += vsq[u];
-            if (gain && i < v1 && (!partial || k < nm.cols)) {
-                if (vec) {
-                    const float4 g0 = __ldg(reinterpret_cast<const float4 *>(gain + k)), g1 = __ldg(reinterpret_cast<const float4 *>(gain + k + 4));
-                    f[0] *= g0.x; f[1] *= g0.y; f[2] *= g0.z; f[3] *= g0.w;
-                    f[4] *= g1.x; f[5] *= g1.y; f[6] *= g1.z; f[7] *= g1.w;
+            for (int u = 0; u < UU; ++u) {
+                const int i = v0 + u * 32 + lane;
+                vsq[u] = 0.f;
+                float f[8];
+                const int k = (vb + i) * 8;
+                if (vec && i < v1) {
+                    const float *p = k < ka ? x + (int64_t)m0 * ldx + k : xb + (int64_t)m0 * ldxb + k - ka;
+                    *reinterpret_cast<float4 *>(f) = __ldcg(reinterpret_cast<const float4 *>(p));
+                    *reinterpret_cast<float4 *>(f + 4) = __ldcg(reinterpret_cast<const float4 *>(p + 4));
                 } else {
 #pragma unroll
-                    for (int j = 0; j < 8; ++j)
-                        if (k + j < K) f[j] *= __ldg(gain + k + j);
-                }
-            }
-            xr[2 * u] = make_float4(f[0], f[1], f[2], f[3]);
-            xr[2 * u + 1] = make_float4(f[4], f[5], f[6], f[7]);
-        }
-        ss[0] = q;
-        if (partial && pc == 0) {
-            const int pv = nm.cols / nm.parts / 8;                     // vectors of a part
-            for (int p = 0; p < nm.parts; ++p) {
-                float t = 0.f;
-#pragma unroll
-                for (int u = 0; u < UU; ++u) {
-                    const int i = v0 + u * 32 + lane;
-                    if (i < v1 && i / pv == p) t += vsq[u];
+                    for (int j = 0; j < 8; ++j) f[j] = i < v1 ? fetch(0, k + j) : 0.f;
                 }
 #pragma unroll
-                for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
-                if (lane == 0) psum[0][warp][p] = t;
-            }
-        }
-    } else {
+                for (int j = 0; j < 8; ++j) vsq[u] = fmaf(f[j], f[j], vsq[u]);
+                q += vsq[u];
+                if (gain && i < v1 && (!partial || k < nm.cols)) {
+                    if (vec) {
+                        const float4 g0 = __ldg(reinterpret_cast<const float4 *>(gain + k)), g1 = __ldg(reinterpret_cast<const float4 *>(gain + k + 4));
+                        f[0] *= g0.x; f[1] *= g0.y; f[2] *= g0.z; f[3] *= g0.w;
+                        f[4] *= g1.x; f[5] *= g1.y; f[6] *= g1.z; f[7] *= g1.w;
+                    } else {
 #pragma unroll
-        for (int m = 0; m < MR; ++m) {
-            ss[m] = 0.f;
-            for (int k = threadIdx.x; k < K8; k += MVD_WARPS * 32) {
-                float v = fetch(m, k);
-                ss[m] = fmaf(v, v, ss[m]);
-                if (gain && k < K && !partial) v *= __ldg(gain + k);
-                xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] = v;
+                        for (int j = 0; j < 8; ++j)
+                            if (k + j < K) f[j] *= __ldg(gain + k + j);
+                    }
+                }
+                xr[2 * u] = make_float4(f[0], f[1], f[2], f[3]);
+                xr[2 * u + 1] = make_float4(f[4], f[5], f[6], f[7]);
             }
-        }
-        if (partial) {
-            const int part_cols = nm.cols / nm.parts;
-            mvd_barrier();
-#pragma unroll
-            for (int m = 0; m < MR; ++m)
+            ss[0] = q;
+            if (EXT && partial && pc == 0) {
+                const int pv = nm.cols / nm.parts / 8;                     // vectors of a part
                 for (int p = 0; p < nm.parts; ++p) {
                     float t = 0.f;
-                    for (int k = p * part_cols + threadIdx.x; k < (p + 1) * part_cols; k += MVD_WARPS * 32) {
-                        const float v = xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)];
-                        t = fmaf(v, v, t);
+#pragma unroll
+                    for (int u = 0; u < UU; ++u) {
+                        const int i = v0 + u * 32 + lane;
+                        if (i < v1 && i / pv == p) t += vsq[u];
                     }
 #pragma unroll
                     for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
-                    if (lane == 0) psum[m][warp][p] = t;
-                }
-        }
-    }
-#pragma unroll
-    for (int m = 0; m < MR; ++m) {
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) ss[m] += __shfl_xor_sync(0xffffffffu, ss[m], o);
-        if (lane == 0) red[warp][m] = ss[m];
-    }
-    mvd_barrier();
-    float rs[MR];
-#pragma unroll
-    for (int m = 0; m < MR; ++m) {
-        rs[m] = 1.f;
-        if (gain && !partial) {
-            float t = 0.f;
-#pragma unroll
-            for (int w = 0; w < MVD_WARPS; ++w) t += red[w][m];
-            rs[m] = 1.f / sqrtf(t / (float)K + nm.eps);
-        }
-    }
-    if (partial && pc == 0) {                       // (the parts lie in the first piece)
-        const int part_cols = nm.cols / nm.parts;
-        auto scale = [&](int m, int p) {
-            float t = 0.f;
-#pragma unroll
-            for (int w = 0; w < MVD_WARPS; ++w) t += psum[m][w][p];
-            return 1.f / sqrtf(t / (float)part_cols + nm.eps);
-        };
-        if constexpr (UU > 0) {
-#pragma unroll
-            for (int u = 0; u < UU; ++u) {
-                const int k = (v0 + u * 32 + lane) * 8;
-                if (k < nm.cols) {
-                    const float f = scale(0, k / part_cols);
-                    xr[2 * u].x *= f; xr[2 * u].y *= f; xr[2 * u].z *= f; xr[2 * u].w *= f;
-                    xr[2 * u + 1].x *= f; xr[2 * u + 1].y *= f; xr[2 * u + 1].z *= f; xr[2 * u + 1].w *= f;
+                    if (lane == 0) psum[0][warp][p] = t;
                 }
             }
         } else {
 #pragma unroll
-            for (int m = 0; m < MR; ++m)
-                for (int p = 0; p < nm.parts; ++p) {
-                    const float f = scale(m, p);
-                    for (int k = p * part_cols + threadIdx.x; k < (p + 1) * part_cols; k += MVD_WARPS * 32)
-                        xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] *= f * __ldg(gain + k);
+            for (int m = 0; m < MR; ++m) {
+                ss[m] = 0.f;
+                for (int k = threadIdx.x; k < K8; k += MVD_WARPS * 32) {
+                    float v = fetch(m, k);
+                    ss[m] = fmaf(v, v, ss[m]);
+                    if (gain && k < K && !partial) v *= __ldg(gain + k);
+                    xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] = v;
                 }
-            mvd_barrier();
-        }
-    }
-
-    // eight rows at a time: their sums are reduced across the warp together (9 shuffles for 8 rows)
-    const bool last = pc + 1 == pieces;
-    filled = 0;
-    for (int g0 = 0; g0 < r1 - r0; g0 += 8) {
-        float acc[MR][8];
+            }
+            if (EXT && partial) {
+                const int part_cols = nm.cols / nm.parts;
+                mvd_barrier();
 #pragma unroll
-        for (int m = 0; m < MR; ++m)
-#pragma unroll
-            for (int j = 0; j < 8; ++j) acc[m][j] = 0.f;
-        const int rows = min(8, r1 - r0 - g0);
-        // the next launch comes in under the last rows: earlier, its own stream of weights delays this one's
-        if (last && g0 + 16 >= r1 - r0 && g0 + 8 < r1 - r0) skn_pdl_launch_dependents();
-#pragma unroll
-        for (int j0 = 0; j0 < 8; j0 += GR) {
-            if (j0 < rows) {
-                if (ok && !skn_mbar_wait(&full_bar[s], phase)) {
-                    if (lane == 0) atomicExch(status, SKN_ERR_TIMEOUT);
-                    ok = false;
-                }
-                // (rows past the CTA's last one are old bytes of the ring: multiplied, never stored)
-                if constexpr (UU > 0) {
-                    float odd[GR] = {};            // two chains
-#pragma unroll
-                    for (int u = 0; u < UU; ++u) {
-                        const int c = v0 + u * 32 + lane;
-                        if (c < v1) {
-#pragma unroll
-                            for (int j = 0; j < GR; ++j) {
-                                float &t = (u & 1) ? odd[j] : acc[0][j0 + j];
-                                t = mvd_dot8(w[j * nv + c], xr[2 * u], xr[2 * u + 1], t);
-                            }
+                for (int m = 0; m < MR; ++m)
+                    for (int p = 0; p < nm.parts; ++p) {
+                        float t = 0.f;
+                        for (int k = p * part_cols + threadIdx.x; k < (p + 1) * part_cols; k += MVD_WARPS * 32) {
+                            const float v = xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)];
+                            t = fmaf(v, v, t);
                         }
+#pragma unroll
+                        for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+                        if (lane == 0) psum[m][warp][p] = t;
                     }
-#pragma unroll
-                    for (int j = 0; j < GR; ++j) acc[0][j0 + j] += odd[j];
-                } else {
-                    for (int c = v0 + lane; c < v1; c += 32) {
-                        uint4 p[GR];
-#pragma unroll
-                        for (int j = 0; j < GR; ++j) p[j] = w[j * nv + c];
-#pragma unroll
-                        for (int m = 0; m < MR; ++m) {
-                            const float4 lo = *reinterpret_cast<const float4 *>(xs + m * K8 + c * 4), hi = *reinterpret_cast<const float4 *>(xs + m * K8 + half + c * 4);
-#pragma unroll
-                            for (int j = 0; j < GR; ++j) acc[m][j0 + j] = mvd_dot8(p[j], lo, hi, acc[m][j0 + j]);
-                        }
-                    }
-                }
-                __syncwarp();
-                if (lane == 0) skn_mbar_arrive(&empty_bar[s]);
-                if (++s == stages) {
-                    s = 0;
-                    phase ^= 1u;
-                    w = reinterpret_cast<const uint4 *>(ring);
-                } else {
-                    w += GR * nv;
-                }
             }
         }
 #pragma unroll
         for (int m = 0; m < MR; ++m) {
 #pragma unroll
-            for (int o = 16, n = 4; o >= 4; o >>= 1, n >>= 1)
-#pragma unroll
-                for (int j = 0; j < n; ++j) {
-                    const bool up = lane & o;
-                    const float mine = up ? acc[m][j + n] : acc[m][j], other = up ? acc[m][j] : acc[m][j + n];
-                    acc[m][j] = mine + __shfl_xor_sync(0xffffffffu, other, o);
-                }
-            float t = acc[m][0];
-            t += __shfl_xor_sync(0xffffffffu, t, 2);
-            t += __shfl_xor_sync(0xffffffffu, t, 1);
-            if ((lane & 3) == 0) {
-                float *p = &part[buf][m][warp][filled + mvd_row(lane)];
-                *p = pc > 0 ? *p + t : t * rs[m];
-            }
+            for (int o = 16; o > 0; o >>= 1) ss[m] += __shfl_xor_sync(0xffffffffu, ss[m], o);
+            if (lane == 0) red[warp][m] = ss[m];
         }
-        filled += rows;
-        if (last && (filled + 8 > MVD_ROWS || g0 + 8 >= r1 - r0)) {
-            mvd_barrier();
-            auto total = [&](int m, int r) {
+        mvd_barrier();
+        float rs[MR];
+#pragma unroll
+        for (int m = 0; m < MR; ++m) {
+            rs[m] = 1.f;
+            if (gain && !partial) {
                 float t = 0.f;
 #pragma unroll
-                for (int w8 = 0; w8 < MVD_WARPS; ++w8) t += part[buf][m][w8][r];
-                return t;
-            };
-            if constexpr (PAIRS) {
-                const int np = (filled + 1) / 2;
-                for (int j = threadIdx.x; j < np * MR; j += MVD_WARPS * 32) {
-                    const int m = j / np, r = j % np * 2;
-                    const bool both = r + 1 < filled;
-                    const float a = total(m, r), b = both ? total(m, r + 1) : 0.f;
-                    dense_store_pair<SKN_EPI_SILU_TAIL>(e, m0 + m, base + r, a, b, both);
-                }
-            } else for (int j = threadIdx.x; j < filled * MR; j += MVD_WARPS * 32) {
-                const int m = j / filled, r = j % filled;
-                dense_store_any(e, m0 + m, base + r, total(m, r));
+                for (int w = 0; w < MVD_WARPS; ++w) t += red[w][m];
+                rs[m] = 1.f / sqrtf(t / (float)K + nm.eps);
             }
-            base += filled;
-            filled = 0;
-            buf ^= 1;                              // the other half is free: every warp has passed the barrier of its readers
         }
-    }
-    if (!last) mvd_barrier();                      // (the sums of squares are written again)
+        if (EXT && partial && pc == 0) {                // (the parts lie in the first piece)
+            const int part_cols = nm.cols / nm.parts;
+            auto scale = [&](int m, int p) {
+                float t = 0.f;
+#pragma unroll
+                for (int w = 0; w < MVD_WARPS; ++w) t += psum[m][w][p];
+                return 1.f / sqrtf(t / (float)part_cols + nm.eps);
+            };
+            if constexpr (UU > 0) {
+#pragma unroll
+                for (int u = 0; u < UU; ++u) {
+                    const int k = (v0 + u * 32 + lane) * 8;
+                    if (k < nm.cols) {
+                        const float f = scale(0, k / part_cols);
+                        xr[2 * u].x *= f; xr[2 * u].y *= f; xr[2 * u].z *= f; xr[2 * u].w *= f;
+                        xr[2 * u + 1].x *= f; xr[2 * u + 1].y *= f; xr[2 * u + 1].z *= f; xr[2 * u + 1].w *= f;
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int m = 0; m < MR; ++m)
+                    for (int p = 0; p < nm.parts; ++p) {
+                        const float f = scale(m, p);
+                        for (int k = p * part_cols + threadIdx.x; k < (p + 1) * part_cols; k += MVD_WARPS * 32)
+                            xs[m * K8 + ((k >> 2) & 1) * half + (k >> 3) * 4 + (k & 3)] *= f * __ldg(gain + k);
+                    }
+                mvd_barrier();
+            }
+        }
+
+        // eight rows at a time: their sums are reduced across the warp together (9 shuffles for 8 rows)
+        const bool last = pc + 1 == pieces;
+        filled = 0;
+        for (int g0 = 0; g0 < r1 - r0; g0 += 8) {
+            float acc[MR][8];
+#pragma unroll
+            for (int m = 0; m < MR; ++m)
+#pragma unroll
+                for (int j = 0; j < 8; ++j) acc[m][j] = 0.f;
+            const int rows = min(8, r1 - r0 - g0);
+            // the next launch comes in under the last rows: earlier, its own stream of weights delays this one's
+            if (last && g0 + 16 >= r1 - r0 && g0 + 8 < r1 - r0) skn_pdl_launch_dependents();
+#pragma unroll
+            for (int j0 = 0; j0 < 8; j0 += GR) {
+                if (j0 < rows) {
+                    if (ok && !skn_mbar_wait(&full_bar[s], phase)) {
+                        if (lane == 0) atomicExch(status, SKN_ERR_TIMEOUT);
+                        ok = false;
+                    }
+                    // (rows past the CTA's last one are old bytes of the ring: multiplied, never stored)
+                    if constexpr (UU > 0) {
+                        float odd[GR] = {};            // two chains
+#pragma unroll
+                        for (int u = 0; u < UU; ++u) {
+                            const int c = v0 + u * 32 + lane;
+                            if (c < v1) {
+#pragma unroll
+                                for (int j = 0; j < GR; ++j) {
+                                    float &t = (u & 1) ? odd[j] : acc[0][j0 + j];
+                                    t = mvd_dot8(w[j * nv + c], xr[2 * u], xr[2 * u + 1], t);
+                                }
+                            }
+                        }
+#pragma unroll
+                        for (int j = 0; j < GR; ++j) acc[0][j0 + j] += odd[j];
+                    } else {
+                        for (int c = v0 + lane; c < v1; c += 32) {
+                            uint4 p[GR];
+#pragma unroll
+                            for (int j = 0; j < GR; ++j) p[j] = w[j * nv + c];
+#pragma unroll
+                            for (int m = 0; m < MR; ++m) {
+                                const float4 lo = *reinterpret_cast<const float4 *>(xs + m * K8 + c * 4), hi = *reinterpret_cast<const float4 *>(xs + m * K8 + half + c * 4);
+#pragma unroll
+                                for (int j = 0; j < GR; ++j) acc[m][j0 + j] = mvd_dot8(p[j], lo, hi, acc[m][j0 + j]);
+                            }
+                        }
+                    }
+                    __syncwarp();
+                    if (lane == 0) skn_mbar_arrive(&empty_bar[s]);
+                    if (++s == stages) {
+                        s = 0;
+                        phase ^= 1u;
+                        w = reinterpret_cast<const uint4 *>(ring);
+                    } else {
+                        w += GR * nv;
+                    }
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < MR; ++m) {
+#pragma unroll
+                for (int o = 16, n = 4; o >= 4; o >>= 1, n >>= 1)
+#pragma unroll
+                    for (int j = 0; j < n; ++j) {
+                        const bool up = lane & o;
+                        const float mine = up ? acc[m][j + n] : acc[m][j], other = up ? acc[m][j] : acc[m][j + n];
+                        acc[m][j] = mine + __shfl_xor_sync(0xffffffffu, other, o);
+                    }
+                float t = acc[m][0];
+                t += __shfl_xor_sync(0xffffffffu, t, 2);
+                t += __shfl_xor_sync(0xffffffffu, t, 1);
+                if ((lane & 3) == 0) {
+                    float *p = &part[buf][m][warp][filled + mvd_row(lane)];
+                    *p = pc > 0 ? *p + t : t * rs[m];
+                }
+            }
+            filled += rows;
+            if (last && (filled + 8 > MVD_ROWS || g0 + 8 >= r1 - r0)) {
+                mvd_barrier();
+                auto total = [&](int m, int r) {
+                    float t = 0.f;
+#pragma unroll
+                    for (int w8 = 0; w8 < MVD_WARPS; ++w8) t += part[buf][m][w8][r];
+                    return t;
+                };
+                if constexpr (PAIRS) {
+                    const int np = (filled + 1) / 2;
+                    for (int j = threadIdx.x; j < np * MR; j += MVD_WARPS * 32) {
+                        const int m = j / np, r = j % np * 2;
+                        const bool both = r + 1 < filled;
+                        const float a = total(m, r), b = both ? total(m, r + 1) : 0.f;
+                        dense_store_pair<SKN_EPI_SILU_TAIL>(e, m0 + m, base + r, a, b, both);
+                    }
+                } else for (int j = threadIdx.x; j < filled * MR; j += MVD_WARPS * 32) {
+                    const int m = j / filled, r = j % filled;
+                    dense_store_any(e, m0 + m, base + r, total(m, r));
+                }
+                base += filled;
+                filled = 0;
+                buf ^= 1;                              // the other half is free: every warp has passed the barrier of its readers
+            }
+        }
+        if (!last) mvd_barrier();                      // (the sums of squares are written again)
     }
 }
 
@@ -603,9 +626,9 @@ static int mvd_uu(int64_t cols) { return (int)(((cols / 8 + MVD_WARPS - 1) / MVD
 constexpr int MVD_MAX_UU = 7;
 constexpr int64_t MVD_PIECE = (int64_t)MVD_MAX_UU * 32 * MVD_WARPS * 8;      // columns of x that the registers hold
 
-template <int MR, int UU, int PICK, bool PAIRS, bool PIECES>
+template <int MR, int UU, int PICK, bool PAIRS, bool EXT>
 static cudaError_t launch_mvd_kernel(skn_ctx *ctx, const skn_linear &l, int pieces, int64_t pitch, int m0, cudaStream_t st) {
-    auto kern = skn_dense_matvec_kernel<MR, UU, PICK, PAIRS, PIECES>;
+    auto kern = skn_dense_matvec_kernel<MR, UU, PICK, PAIRS, EXT>;
     static bool attr_done[64] = {false};
     if (!attr_done[ctx->device & 63]) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, mvd_smem(MR));
@@ -637,9 +660,9 @@ static cudaError_t launch_mvd(skn_ctx *ctx, const skn_linear &l, int pieces, int
     if (pairs) return cudaErrorInvalidValue;
     if constexpr (PICK == SKN_PICK_ROWS) return cudaErrorInvalidValue;
     else {
-        if constexpr (MR == 1 && UU >= 4)
-            if (pieces > 1) return launch_mvd_kernel<MR, UU, PICK, false, true>(ctx, l, pieces, pitch, m0, st);
-        return launch_mvd_kernel<MR, UU, PICK, false, false>(ctx, l, 1, pitch, m0, st);
+        if (PICK == SKN_PICK_COLS || pieces > 1 || (l.gain && l.norm_cols > 0)) return launch_mvd_kernel<MR, UU, PICK, false, true>(ctx, l, pieces, pitch, m0, st);
+        if constexpr (PICK == SKN_PICK_NONE) return launch_mvd_kernel<MR, UU, PICK, false, false>(ctx, l, 1, pitch, m0, st);
+        return cudaErrorInvalidValue;
     }
 }
 

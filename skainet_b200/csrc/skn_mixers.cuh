@@ -1,6 +1,7 @@
 // Token mixers over position-addressed caches and recurrent states (declarations; kernels in skn_mixers.cu):
-//   chunked attention   per-head RMS norm of q and k, rotation of their first dimensions (half-split pairs), softmax
-//                       over the keys of the query's own chunk (or all earlier keys), optional tanh soft cap
+//   attention           per-head RMS norm of q and k, rotation of their first dimensions (half-split pairs), softmax
+//                       over the keys of the query's own chunk, of a sliding window, or all earlier keys, optional tanh
+//                       soft cap, optional sink in the denominator
 //   retention           linear attention with one fixed decay per head: S <- decay S + k v^T, o = S^T q; o divided by
 //                       its root mean square and multiplied by silu(gate)
 // Both read the raw fp32 rows of one joint projection and write the (scaled) concatenated heads that the output
