@@ -135,17 +135,35 @@ __device__ __forceinline__ void dense_put_packed(__nv_bfloat16 *y, int64_t ld, i
         p += ld;                                   // two tokens of ld / 2 words
     }
 }
-// whether an epilogue's run may be stored that way
-template <int EPI>
-__device__ __forceinline__ bool dense_packs(const skn_epi &e, int N) {
-    if (EPI == SKN_EPI_STORE || EPI == SKN_EPI_ROTATE)
-        return N % 2 == 0 && !e.y32 && e.y16 && e.ld_y16 % 2 == 0 && (reinterpret_cast<uintptr_t>(e.y16) & 3) == 0;
-    return false;
+__device__ __forceinline__ bool dense_packs(const __nv_bfloat16 *y16, int64_t ld, const float *y32, int N) {
+    return N % 4 == 0 && y16 && !y32 && ld % 2 == 0 && (reinterpret_cast<uintptr_t>(y16) & 3) == 0;
 }
 
-// The same for the pair epilogues, the whole warp together: lane l holds row n = (even base) + l, `in` marks the rows that exist.
+// NC tokens of rows (gate, up), a warp of activation rows only (n - n_act of its first lane is a multiple of 4).  The lanes of a pair take a
+// token each, then lanes two apart trade tokens, so that a lane stores two columns of every fourth token.
+template <int NC>
+__device__ __forceinline__ void dense_put_silu_packed(const skn_epi &e, int64_t m, int64_t n, const float (&v)[NC], int count, bool in) {
+    const bool odd = n & 1, high = (n >> 1) & 1;
+    const int t0 = (odd ? 1 : 0) + (high ? 2 : 0);
+    uint32_t *p = reinterpret_cast<uint32_t *>(e.act16 + (m + t0) * e.ld_act16 + (((n & ~(int64_t)3) - e.n_act) >> 1));
+#pragma unroll
+    for (int c = 0; c < NC; c += 4) {
+        float f[2];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            const float a = v[c + 2 * x], b = v[c + 2 * x + 1], got = __shfl_xor_sync(0xffffffffu, odd ? a : b, 1);
+            f[x] = odd ? dense_silu(got) * b : dense_silu(a) * got;
+        }
+        const float got = __shfl_xor_sync(0xffffffffu, high ? f[0] : f[1], 2);
+        const uint32_t w = high ? tc_pack_bf16(got, f[1]) : tc_pack_bf16(f[0], got);
+        if (in && c + t0 < count) *p = w;
+        p += e.ld_act16 * 2;                       // four tokens of ld / 2 words
+    }
+}
+
+// The pair epilogues in general, the whole warp together: lane l holds row n = (even base) + l, `in` marks the rows that exist.
 template <int EPI, int NC>
-__device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t m, int64_t n, float (&v)[NC], int count, bool in, bool packed) {
+__device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int N, int64_t m, int64_t n, float (&v)[NC], int count, bool in) {
     const bool odd = n & 1;
     if (EPI == SKN_EPI_ROTATE) {
         // the angles of the run are loaded before its first store
@@ -159,7 +177,7 @@ __device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t 
             const float other = __shfl_xor_sync(0xffffffffu, v[c], 1);
             v[c] = odd ? v[c] * cs[c].x + other * cs[c].y : v[c] * cs[c].x - other * cs[c].y;
         }
-        if (packed) {
+        if (dense_packs(e.y16, e.ld_y16, e.y32, N)) {
             dense_put_packed(e.y16 + m * e.ld_y16 + n, e.ld_y16, n, v, count, in);
             return;
         }
@@ -176,6 +194,47 @@ __device__ __forceinline__ void dense_store_run_pairs(const skn_epi &e, int64_t 
         if (!act) dense_put(e, m + c, n, v[c]);
         else if (!odd) dense_put_silu(e, m + c, n, v[c], other);
     }
+}
+
+// A run of NC tokens of the warp's 32 rows (lane l: row n, of N), in the quickest form that its destination allows
+template <int EPI, int NC>
+__device__ __forceinline__ void dense_store_warp(const skn_epi &e, int N, int64_t m, int64_t n, float (&v)[NC], int count, bool ok) {
+    const bool in = n < N && ok;
+    const int64_t first = n - (threadIdx.x & 31);
+    if constexpr (EPI == SKN_EPI_STORE || EPI == SKN_EPI_RELU2) {
+        if (dense_packs(e.y16, e.ld_y16, e.y32, N)) {
+            if (EPI == SKN_EPI_RELU2)
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    v[c] = fmaxf(v[c], 0.f);
+                    v[c] *= v[c];
+                }
+            dense_put_packed(e.y16 + m * e.ld_y16 + n, e.ld_y16, n, v, count, in);
+            return;
+        }
+    }
+    if constexpr (EPI == SKN_EPI_GELU_TAIL) {
+        if (first >= e.n_act && e.n_act % 2 == 0 && dense_packs(e.act16, e.ld_act16, e.act32, N)) {
+#pragma unroll
+            for (int c = 0; c < NC; ++c) v[c] = dense_gelu_exp(v[c]);
+            dense_put_packed(e.act16 + m * e.ld_act16 + n - e.n_act, e.ld_act16, n, v, count, in);
+            return;
+        }
+    }
+    if constexpr (EPI == SKN_EPI_SILU_TAIL) {
+        if (first >= e.n_act && e.n_act % 4 == 0 && !e.act_scale && dense_packs(e.act16, e.ld_act16, e.act32, N)) {
+            dense_put_silu_packed(e, m, n, v, count, in);
+            return;
+        }
+        if (first + 31 < e.n_act) {                // none of the rows is activated
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+                if (c < count && in) dense_put(e, m + c, n, v[c]);
+            return;
+        }
+    }
+    if constexpr (skn_epi_pairs(EPI)) dense_store_run_pairs<EPI, NC>(e, N, m, n, v, count, in);
+    else if (in) dense_store_run<EPI, NC>(e, m, n, v, count);
 }
 
 // experts as groups of rows: first tile of each in tiles of NT rows (start[E]: their number), by one warp
@@ -955,7 +1014,6 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
     } else {
         // epilogue: TMEM lane = weight row, column = token; a warp's store covers 32 consecutive outputs of one token
         bool ok = true;
-        const bool packed = dense_packs<EPI>(e, N);
         int tile = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, ++tile) {
             const dtc_tile tl = tile_of(u);
@@ -977,22 +1035,10 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 uint32_t acc[32];
                 tc_ld32(src + c0, acc);
                 if (splits == 1) {
-                    if constexpr (skn_epi_pairs(EPI)) {
-                        float v[32];
+                    float v[32];
 #pragma unroll
-                        for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
-                        dense_store_run_pairs<EPI, 32>(e, m0 + c0, n, v, cols - c0, n < N && ok, packed);
-                    } else if (EPI == SKN_EPI_STORE && packed) {
-                        float v[32];
-#pragma unroll
-                        for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
-                        dense_put_packed(e.y16 + (m0 + c0) * e.ld_y16 + n, e.ld_y16, n, v, cols - c0, n < N && ok);
-                    } else if (n < N && ok) {
-                        float v[32];
-#pragma unroll
-                        for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
-                        dense_store_run<EPI, 32>(e, m0 + c0, n, v, cols - c0);
-                    }
+                    for (int c = 0; c < 32; ++c) v[c] = __uint_as_float(acc[c]);
+                    dense_store_warp<EPI, 32>(e, N, m0 + c0, n, v, cols - c0, ok);
                 } else {
 #pragma unroll
                     for (int c = 0; c < 32; ++c)
@@ -1018,8 +1064,7 @@ skn_dense_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                         for (int s = 0; s < splits; ++s)
 #pragma unroll
                             for (int c = 0; c < 16; ++c) v[c] += __ldcg(pbase + ((size_t)s * NT + c0 + c) * DTC_BM);
-                        if constexpr (skn_epi_pairs(EPI)) dense_store_run_pairs<EPI, 16>(e, m0 + c0, n, v, cols - c0, n < N && ok, packed);
-                        else if (n < N && ok) dense_store_run<EPI, 16>(e, m0 + c0, n, v, cols - c0);
+                        dense_store_warp<EPI, 16>(e, N, m0 + c0, n, v, cols - c0, ok);
                     }
                     if (threadIdx.x == 0) tickets[tidx] = 0;
                 }
