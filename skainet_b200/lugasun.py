@@ -1,4 +1,4 @@
-"""Host side of the Lugasun decoder (skn_lugasun_*): configuration, weight loading and the step function.
+"""Host side of the Lugasun decoder (skn_lugasun_*): configuration and weight loading.
 
 A layer runs chunked softmax attention and retention side by side on one normalised input (`parallel` mixer), then an
 optional squared-relu feed-forward, then a token side input; a range of layers may be looped with a cache and a state
